@@ -13,6 +13,7 @@
 //
 //   maps_prep         bias, per-map RMS norm of q and k (a weight of dim values shared by heads and maps), rotation of the
 //                     first rdims values of every map of q and k, cache write of a step's tokens; q out
+//   maps_row_prep     the same with one norm over the whole projection of q (and of k), and a factor on q by its position
 //   maps_prefill      any number of new tokens per sequence (float and bfloat16, any sizes up to 256)
 //   maps_prefill_mma  bfloat16 prompts on the tensor cores
 //   maps_decode       one new token per sequence: runs of pages, one block of threads a run, then maps_merge, which also
@@ -92,6 +93,99 @@ __global__ void maps_prep_kernel(const float* __restrict__ qkv, const float* __r
     for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(rd > 0 ? maps_turned(buf, i, rd, cs, sn, interleaved) : buf[i]);
 }
 
+// ---------------------------------------------------------------------------------
+// prep with norms over whole projections: all H * maps * dim values of q (and all G * maps * dim of k) are divided by ONE
+// root mean square and multiplied by weights of that size, then turned as above; q is then multiplied by
+// 1 + t_coef * ln(floor((p + 1) / t_every) + 1), a factor that grows with the position p (t_coef 0: 1).
+// grid (T, 3): a block for a token's q, one for its k, one for its v.  FOURS: 4 values at a time (no rotation, all sizes
+// multiples of 4); a row of up to 16 values a thread then stays in registers between the sum and the result.
+// ---------------------------------------------------------------------------------
+template <typename T> __device__ __forceinline__ void maps_store4(T* dst, float4 v);
+template <> __device__ __forceinline__ void maps_store4<float>(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+template <> __device__ __forceinline__ void maps_store4<bf16>(bf16* dst, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+template <typename T, bool FOURS>
+__global__ void __launch_bounds__(256)
+maps_row_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ qw,
+                     const float* __restrict__ kw, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                     const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ page_table,
+                     int table_width, T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool, int H, int G, int maps,
+                     int dim, int vdim, int rdims, int interleaved, float eps, float t_coef, float t_every, int store_kv) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x, part = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
+    if (part > 0 && !store_kv) return;
+    const int kdim = maps * dim, nq = H * kdim, nk = G * kdim, nv = G * vdim;
+    const int n = part == 0 ? nq : (part == 1 ? nk : nv), col = part == 0 ? 0 : (part == 1 ? nq : nq + nk);
+    const int ld = nq + nk + nv, per = part == 2 ? vdim : kdim;
+    const float* src = qkv + (size_t)t * ld + col;
+    const float* bs = bias ? bias + col : nullptr;
+    const float* w = part == 0 ? qw : (part == 1 ? kw : nullptr);
+    const int p = tok_pos[t];
+    T* dst = q_out + (size_t)t * nq;                    // where value i of the row goes: dst + (i / per) * head_step + i % per
+    size_t head_step = per;
+    if (part > 0) {
+        const size_t page = page_table[(size_t)tok_seq[t] * table_width + p / QWB_MAPS_PAGE];
+        dst = (part == 1 ? k_pool : v_pool) + (page * G * QWB_MAPS_PAGE + p % QWB_MAPS_PAGE) * (size_t)per;
+        head_step = (size_t)QWB_MAPS_PAGE * per;
+    }
+    float factor = 1.f;
+    if (part == 0 && t_coef != 0.f) factor = 1.f + t_coef * logf((float)floor((double)(p + 1) / (double)t_every) + 1.f);
+
+    if constexpr (FOURS) {
+        constexpr int KEEP = 4;
+        float4 held[KEEP];
+        auto load = [&](int i) {
+            float4 v = *reinterpret_cast<const float4*>(src + 4 * i);
+            if (bs) { const float4 b = *reinterpret_cast<const float4*>(bs + 4 * i); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+            return v;
+        };
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const int i = tid + j * nt;
+            held[j] = i < n / 4 ? load(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss += held[j].x * held[j].x + held[j].y * held[j].y + held[j].z * held[j].z + held[j].w * held[j].w;
+        }
+        for (int i = tid + KEEP * nt; i < n / 4; i += nt) { const float4 v = load(i); ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+        float mul = factor;
+        if (w) mul *= rsqrtf(block_sum(ss, scratch) / (float)n + eps);
+        auto store = [&](int i, float4 v) {
+            float4 f = make_float4(mul, mul, mul, mul);
+            if (w) { const float4 a = *reinterpret_cast<const float4*>(w + 4 * i); f.x *= a.x; f.y *= a.y; f.z *= a.z; f.w *= a.w; }
+            const int head = 4 * i / per;
+            maps_store4<T>(dst + head * head_step + (4 * i - head * per), make_float4(v.x * f.x, v.y * f.y, v.z * f.z, v.w * f.w));
+        };
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) { const int i = tid + j * nt; if (i < n / 4) store(i, held[j]); }
+        for (int i = tid + KEEP * nt; i < n / 4; i += nt) store(i, load(i));
+    } else {
+        float ss = 0.f;
+        for (int i = tid; i < n; i += nt) { const float v = src[i] + (bs ? bs[i] : 0.f); ss += v * v; }
+        float mul = 1.f;
+        if (w) mul = rsqrtf(block_sum(ss, scratch) / (float)n + eps);
+        auto normed = [&](int i) { return (src[i] + (bs ? bs[i] : 0.f)) * mul * (w ? w[i] : 1.f); };
+        const int rd = part < 2 ? rdims : 0;
+        const float* cs = cos_t + (size_t)t * (rd >> 1);
+        const float* sn = sin_t + (size_t)t * (rd >> 1);
+        for (int i = tid; i < n; i += nt) {
+            const int head = i / per, in_map = part == 2 ? i - head * per : (i - head * per) % dim;
+            float v = normed(i);
+            if (in_map < rd) {
+                const int m = interleaved ? in_map >> 1 : (in_map < rd / 2 ? in_map : in_map - rd / 2);
+                const bool first = interleaved ? !(in_map & 1) : in_map < rd / 2;
+                const int other = interleaved ? (first ? i + 1 : i - 1) : (first ? i + rd / 2 : i - rd / 2);
+                v = first ? v * cs[m] - normed(other) * sn[m] : v * cs[m] + normed(other) * sn[m];
+            }
+            dst[head * head_step + (i - head * per)] = from_f32<T>(v * factor);
+        }
+    }
+}
+
 // `step`: 1 for the kernels that read value by value, 8 for those that copy 16 bytes at a time
 static int check_maps_sizes(const char* what, int H, int G, int maps, int dim, int vdim, int table_width, int chunk, int step) {
     if (H <= 0 || G <= 0 || H % G) return qwb_fail(QWB_ERR_ARG, "%s: %d query heads are not a multiple of %d key/value heads", what, H, G);
@@ -119,6 +213,34 @@ extern "C" int qwb_maps_prep(const float* qkv, const float* bias, const float* q
                    (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool, H, G, maps, dim, vdim, rdims, interleaved, eps, store_kv);
     else return qwb_fail(QWB_ERR_ARG, "maps_prep: unknown dtype %d", dtype);
     return qwb_check_launch("maps_prep");
+}
+
+// qw [H * maps * dim], kw [G * maps * dim] (either may be null); the rest as qwb_maps_prep.
+extern "C" int qwb_maps_row_prep(const float* qkv, const float* bias, const float* qw, const float* kw, const float* cos_t, const float* sin_t,
+                                 const int* tok_seq, const int* tok_pos, const int* page_table, int table_width, void* q_out, void* k_pool,
+                                 void* v_pool, int dtype, int T, int H, int G, int maps, int dim, int vdim, int rdims, int interleaved,
+                                 float eps, float t_coef, float t_every, int store_kv, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (int rc = check_maps_sizes("maps_row_prep", H, G, maps, dim, vdim, table_width, 0, 1)) return rc;
+    if (rdims < 0 || rdims > dim || rdims % 2) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a rotation of %d of %d values", rdims, dim);
+    if (rdims > 0 && (!cos_t || !sin_t)) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a rotation without its table");
+    if (t_coef != 0.f && !(t_every > 0.f)) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a query factor in steps of %g positions", t_every);
+    const bool fours = rdims == 0 && dim % 4 == 0 && vdim % 4 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 &&
+                       (uintptr_t)qw % 16 == 0 && (uintptr_t)kw % 16 == 0;
+    const int widest = H * maps * dim;
+    const dim3 grid(T, 3), block(widest >= 1024 ? 256 : 128);
+    auto go = [&](auto kernel, auto* q, auto* k, auto* v) {
+        qwb_launch(kernel, grid, block, 0, stream, qkv, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos, page_table, table_width, q, k, v, H, G, maps,
+                   dim, vdim, rdims, interleaved, eps, t_coef, t_every, store_kv);
+    };
+    if (dtype == QWB_DT_F32) {
+        if (fours) go(maps_row_prep_kernel<float, true>, (float*)q_out, (float*)k_pool, (float*)v_pool);
+        else go(maps_row_prep_kernel<float, false>, (float*)q_out, (float*)k_pool, (float*)v_pool);
+    } else if (dtype == QWB_DT_BF16) {
+        if (fours) go(maps_row_prep_kernel<bf16, true>, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool);
+        else go(maps_row_prep_kernel<bf16, false>, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool);
+    } else return qwb_fail(QWB_ERR_ARG, "maps_row_prep: unknown dtype %d", dtype);
+    return qwb_check_launch("maps_row_prep");
 }
 
 // ---------------------------------------------------------------------------------

@@ -135,6 +135,17 @@ template <typename T> __device__ __forceinline__ T from_f32(float x);
 template <> __device__ __forceinline__ float from_f32<float>(float x) { return x; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float x) { return __float2bfloat16_rn(x); }
 
+// The activations of an ungated product without numbers of their own: 0 none, 1 relu squared, 2 gelu (tanh form), 3 silu,
+// 5 gelu (v times the normal distribution's function).
+__host__ __device__ __forceinline__ bool qwb_activation_known(int act) { return act >= 0 && act <= 5 && act != 4; }
+__device__ __forceinline__ float qwb_activate(float v, int act) {
+    if (act == 1) { v = fmaxf(v, 0.f); return v * v; }
+    if (act == 2) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+    if (act == 3) return v / (1.f + expf(-v));
+    if (act == 5) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+    return v;
+}
+
 // 16-byte vectors of T: 4 floats or 8 bfloat16.
 template <typename T> struct Vec16;
 template <> struct Vec16<float> {

@@ -3,13 +3,14 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------------
-// h[t,:] = float(E[id_t,:]) * scale.  A row gather (the reference, which does not scale:
-// core/runtime.cpp:1001, ggml-cuda/getrows.cu:73-102).  An id outside [0, V) writes a
-// row of zeros and records the first such token in *bad_token (if given).
+// h[t,:] = float(E[id_t,:]) * scale (+ float(P[p_t,:]), p_t the token's position).  A row gather (the reference, which
+// neither scales nor adds: core/runtime.cpp:1001, ggml-cuda/getrows.cu:73-102).  An id outside [0, V) writes a row of
+// zeros and records the first such token in *bad_token (if given); a position outside [0, NP) adds nothing.
 // ---------------------------------------------------------------------------------
 template <typename T>
-__global__ void embed_gather_kernel(const int* __restrict__ ids, const T* __restrict__ table,
-                                    float* __restrict__ out, int D, int V, int* bad_token, float scale) {
+__global__ void embed_gather_kernel(const int* __restrict__ ids, const T* __restrict__ table, const int* __restrict__ pos,
+                                    const T* __restrict__ pos_table, float* __restrict__ out, int D, int V, int NP,
+                                    int* bad_token, float scale) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
@@ -21,31 +22,37 @@ __global__ void embed_gather_kernel(const int* __restrict__ ids, const T* __rest
         return;
     }
     const T* row = table + (size_t)id * D;
+    const int p = pos_table ? pos[t] : -1;
+    const T* prow = p >= 0 && p < NP ? pos_table + (size_t)p * D : nullptr;
     constexpr int VEC = Vec16<T>::N;
-    if (D % VEC == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)out % 16 == 0) {      // 16 bytes of the row a load
-        const Vec16<T>* src = reinterpret_cast<const Vec16<T>*>(row);
+    if (D % VEC == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)pos_table % 16 == 0) {
+        const Vec16<T>* src = reinterpret_cast<const Vec16<T>*>(row);                  // 16 bytes of the row a load
+        const Vec16<T>* psrc = reinterpret_cast<const Vec16<T>*>(prow);
         for (int i = threadIdx.x; i < D / VEC; i += blockDim.x) {
-            float v[VEC];
+            float v[VEC], w[VEC];
             src[i].get(v);
+            if (prow) psrc[i].get(w);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] = v[e] * scale + (prow ? w[e] : 0.f);
 #pragma unroll
             for (int e = 0; e < VEC; e += 4)
-                *reinterpret_cast<float4*>(o + (size_t)i * VEC + e) =
-                    make_float4(v[e] * scale, v[e + 1] * scale, v[e + 2] * scale, v[e + 3] * scale);
+                *reinterpret_cast<float4*>(o + (size_t)i * VEC + e) = make_float4(v[e], v[e + 1], v[e + 2], v[e + 3]);
         }
         return;
     }
-    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = to_f32(row[i]) * scale;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = to_f32(row[i]) * scale + (prow ? to_f32(prow[i]) : 0.f);
 }
 
-extern "C" int qwb_embed_gather(const int* ids, const void* table, int table_dtype, float* out,
-                                int T, int D, int V, int* bad_token, float scale, cudaStream_t stream) {
+extern "C" int qwb_embed_gather(const int* ids, const void* table, int table_dtype, const int* pos, const void* pos_table, float* out,
+                                int T, int D, int V, int NP, int* bad_token, float scale, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (D <= 0 || V <= 0) return qwb_fail(QWB_ERR_ARG, "embed_gather: bad sizes D=%d V=%d", D, V);
+    if (pos_table && (!pos || NP <= 0)) return qwb_fail(QWB_ERR_ARG, "embed_gather: a position table of %d rows without positions", NP);
     const int block = D >= 1024 ? 256 : 128;
     if (table_dtype == QWB_DT_F32)
-        qwb_launch(embed_gather_kernel<float>, T, block, 0, stream, ids, (const float*)table, out, D, V, bad_token, scale);
+        qwb_launch(embed_gather_kernel<float>, T, block, 0, stream, ids, (const float*)table, pos, (const float*)pos_table, out, D, V, NP, bad_token, scale);
     else if (table_dtype == QWB_DT_BF16)
-        qwb_launch(embed_gather_kernel<bf16>, T, block, 0, stream, ids, (const bf16*)table, out, D, V, bad_token, scale);
+        qwb_launch(embed_gather_kernel<bf16>, T, block, 0, stream, ids, (const bf16*)table, pos, (const bf16*)pos_table, out, D, V, NP, bad_token, scale);
     else
         return qwb_fail(QWB_ERR_ARG, "embed_gather: unknown dtype %d", table_dtype);
     return qwb_check_launch("embed_gather");
@@ -667,7 +674,8 @@ extern "C" int qwb_rmsnorm_mix(const float* y, const float* w, float* h, void* c
 // out[t, f] = act(x[t, f] + bias[f]) for F columns of a float matrix with rows of ld values (the caller offsets the
 // pointer to the first column); out [T, F] float or bfloat16 (may be x itself when float and ld = F).
 // act 0: none; 1: relu squared; 2: gelu (tanh form); 3: silu; 4: xIELU with two learned numbers p, q (`params`):
-// v > 0: softplus(p) v^2 + v / 2;  v <= 0: (1/2 + softplus(q)) (e^v - 1 - v) + v / 2.  bias may be null.
+// v > 0: softplus(p) v^2 + v / 2;  v <= 0: (1/2 + softplus(q)) (e^v - 1 - v) + v / 2; 5: gelu (v times the normal
+// distribution's function).  bias may be null.
 // ---------------------------------------------------------------------------------
 __device__ __forceinline__ float softplus32(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
@@ -681,10 +689,8 @@ __global__ void bias_act_kernel(const float* x, int ld, const float* __restrict_
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const size_t t = i / F, f = i - t * F;
         float v = x[t * ld + f] + (bias ? bias[f] : 0.f);
-        if (act == 1) { v = fmaxf(v, 0.f); v *= v; }
-        else if (act == 2) v = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
-        else if (act == 3) v = v / (1.f + expf(-v));
-        else if (act == 4) v = v > 0.f ? up * v * v + 0.5f * v : down * (expm1f(v) - v) + 0.5f * v;
+        if (act == 4) v = v > 0.f ? up * v * v + 0.5f * v : down * (expm1f(v) - v) + 0.5f * v;
+        else v = qwb_activate(v, act);
         out[i] = from_f32<TOut>(v);
     }
 }
@@ -693,7 +699,7 @@ extern "C" int qwb_bias_act(const float* x, int ld, const float* bias, void* out
                             const float* params, cudaStream_t stream) {
     if (T <= 0 || F <= 0) return 0;
     if (ld < F) return qwb_fail(QWB_ERR_ARG, "bias_act: rows of %d values hold no %d columns", ld, F);
-    if (act < 0 || act > 4) return qwb_fail(QWB_ERR_ARG, "bias_act: unknown activation %d", act);
+    if (act < 0 || act > 5) return qwb_fail(QWB_ERR_ARG, "bias_act: unknown activation %d", act);
     if (act == 4 && !params) return qwb_fail(QWB_ERR_ARG, "bias_act: this activation needs its two numbers");
     const size_t n = (size_t)T * F;
     const int block = 256;

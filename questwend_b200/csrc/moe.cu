@@ -1,178 +1,446 @@
-// Routed experts: the router's choice and the experts' gated feed-forward for the tokens that chose them.
+// Routed experts: the router's choice, and the experts' feed-forward for the tokens that chose them.
 //
-//   moe_route     scores = softmax(logits) over all experts (32-bit); the `top` largest, ties to the lower index;
-//                 weights = the chosen scores, divided by their sum only if `renorm`
-//   moe_gate_up   act[t, k, :] = silu(Wg[e] x_t) * (Wu[e] x_t), e = the k-th choice of token t
+//   moe_route     scores of all experts (softmax or sigmoid of the logits, 32-bit); a choice by score, or by score plus a
+//                 correction per expert, over all experts or inside the best groups of neighbours; the `top` largest,
+//                 ties to the lower index; weights from the scores alone
+//   moe_up        act[t, k, :] = silu(Wg[e] x_t) * (Wu[e] x_t) (gated) or f(Wu[e] x_t), e = the k-th choice of token t
 //   moe_down      out[t, :] = sum_k weight[t, k] * Wd[e_k] act[t, k, :]
+// A shared expert (ungated, a width of its own) that every token uses rides in the same two kernels; its output is
+// multiplied by a number per token.
 //
-// The products read each chosen expert's rows straight from the stacked weights (Wgu [E, 2F, D]: gate rows, then up
-// rows; Wd [E, D, F]): a warp per output feature, 32-bit sums.  This is the form for a step of few tokens, where every
+// The products read each chosen expert's rows straight from the stacked weights (Wu [E, F, D], gated: [E, 2F, D] with the
+// gate rows first; Wd [E, D, F]): a warp per few rows, 32-bit sums.  This is the form for a step of few tokens, where every
 // token's experts are streamed once, and for the 32-bit engine.  Many bfloat16 tokens are sorted by expert instead
-// and go through a library grouped product; moe_gated_act and moe_combine are the kernels around it.
+// and go through a library grouped product; moe_sort, moe_spread, moe_act and moe_combine are the kernels around it.
 #include "common.cuh"
 
 #define QWB_MOE_MAX_TOP 16
+#define QWB_MOE_MAX_EXPERTS 1024
+#define QWB_MOE_GATED 16        // activation code of the gated form, silu(gate) * up; others: qwb_activate's codes
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, int* __restrict__ chosen, float* __restrict__ weight,
-                                 int T, int E, int top, int renorm) {
+// ---------------------------------------------------------------------------------
+// route: a warp per token.  logits rows hold ld values: E experts and, with gate_out, the shared expert's gate after them.
+//   score[e]  softmax(z)[e] (sigmoid = 0) or 1 / (1 + exp(-z[e])) (sigmoid = 1)
+//   choice[e] score[e] + correction[e]; a group's score is the sum of its two largest choices (of one, if it has one
+//             expert), and the experts of all but the `keep` best groups (ties to the lower index) are out
+//   weight    score of a chosen expert, / (their sum + sum_eps) if `renorm`, * weight_scale
+//   gate_out  1 / (1 + exp(-z[E]))
+// ---------------------------------------------------------------------------------
+__global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int* __restrict__ chosen,
+                                 float* __restrict__ weight, float* __restrict__ gate_out, int T, int E, int top, int sigmoid,
+                                 int groups, int keep, int renorm, float sum_eps, float weight_scale) {
     pdl_wait();
     pdl_launch_dependents();
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    extern __shared__ float route_smem[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= T) return;
-    const float* z = logits + (size_t)t * E;
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
-    sum = warp_sum(sum);
+    float* choice = route_smem + warp * (E + groups);       // [E], then the groups' scores [groups]
+    float* gscore = choice + E;
+    const float* z = logits + (size_t)t * ld;
+    const unsigned full = 0xffffffffu;
+    float mx = 0.f, sum = 1.f;
+    if (!sigmoid) {
+        mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+        mx = warp_max(mx);
+        sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+        sum = warp_sum(sum);
+    }
+    auto score_of = [&](float v) { return sigmoid ? 1.f / (1.f + expf(-v)) : expf(v - mx) / sum; };
+    const bool by_logit = !sigmoid && !correction && groups == 1;       // a softmax keeps the logits' order
+    for (int e = lane; e < E; e += 32) choice[e] = by_logit ? z[e] : score_of(z[e]) + (correction ? correction[e] : 0.f);
+    __syncwarp();
+    // the largest of n values in shared memory (ties to the lower index), marked as taken
+    auto take_best = [&](float* v, int n) {
+        float best = -INFINITY;
+        int at = n;
+        for (int e = lane; e < n; e += 32)
+            if (v[e] > best) { best = v[e]; at = e; }
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(full, best, o);
+            const int oa = __shfl_xor_sync(full, at, o);
+            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+        }
+        __syncwarp();
+        if (lane == 0 && at < n) v[at] = -INFINITY;
+        __syncwarp();
+        return at;
+    };
+    if (keep < groups) {
+        const int size = E / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;             // the two largest
+            for (int e = g * size; e < (g + 1) * size; ++e) {
+                const float c = choice[e];
+                if (c > a) { b = a; a = c; }
+                else if (c > b) b = c;
+            }
+            gscore[g] = size > 1 ? a + b : a;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; ++k) take_best(gscore, groups);
+        for (int e = lane; e < E; e += 32)
+            if (gscore[e / size] != -INFINITY) choice[e] = -INFINITY;       // a group that was not taken
+        __syncwarp();
+    }
     int picked[QWB_MOE_MAX_TOP];
     float score[QWB_MOE_MAX_TOP];
     float total = 0.f;
-    for (int k = 0; k < top; ++k) {
-        float best = -INFINITY;
-        int at = E;
-        for (int e = lane; e < E; e += 32) {
-            bool taken = false;
-            for (int j = 0; j < k; ++j) taken |= picked[j] == e;
-            if (!taken && (z[e] > best)) { best = z[e]; at = e; }
-        }
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-        }
-        picked[k] = at;
-        score[k] = expf(best - mx) / sum;
+#pragma unroll
+    for (int k = 0; k < QWB_MOE_MAX_TOP; ++k) {
+        if (k >= top) break;
+        const int at = take_best(choice, E);
+        picked[k] = at < E ? at : k;                        // nothing comparable left (not-a-number logits): a valid index
+        score[k] = score_of(z[picked[k]]);
         total += score[k];
     }
-    if (lane == 0)
-        for (int k = 0; k < top; ++k) {
+    if (lane == 0) {
+        const float mul = weight_scale;
+#pragma unroll
+        for (int k = 0; k < QWB_MOE_MAX_TOP; ++k) {
+            if (k >= top) break;
             chosen[(size_t)t * top + k] = picked[k];
-            weight[(size_t)t * top + k] = renorm ? score[k] / total : score[k];
+            weight[(size_t)t * top + k] = (renorm ? score[k] / (total + sum_eps) : score[k]) * mul;
         }
+        if (gate_out) gate_out[t] = 1.f / (1.f + expf(-z[E]));
+    }
 }
 
-extern "C" int qwb_moe_route(const float* logits, int* chosen, float* weight, int T, int E, int top, int renorm, cudaStream_t stream) {
+extern "C" int qwb_moe_route(const float* logits, int ld, const float* correction, int* chosen, float* weight, float* gate_out, int T,
+                             int E, int top, int sigmoid, int groups, int keep, int renorm, float sum_eps, float weight_scale,
+                             cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || top > QWB_MOE_MAX_TOP)
-        return qwb_fail(QWB_ERR_ARG, "moe_route: %d of %d experts (at most %d)", top, E, QWB_MOE_MAX_TOP);
-    qwb_launch(moe_route_kernel, (T + 3) / 4, 128, 0, stream, logits, chosen, weight, T, E, top, renorm);
+    if (E <= 0 || E > QWB_MOE_MAX_EXPERTS || top <= 0 || top > E || top > QWB_MOE_MAX_TOP)
+        return qwb_fail(QWB_ERR_ARG, "moe_route: %d of %d experts (at most %d of %d)", top, E, QWB_MOE_MAX_TOP, QWB_MOE_MAX_EXPERTS);
+    if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups))
+        return qwb_fail(QWB_ERR_ARG, "moe_route: %d of %d experts from %d of %d groups", top, E, keep, groups);
+    if (ld < E + (gate_out ? 1 : 0)) return qwb_fail(QWB_ERR_ARG, "moe_route: rows of %d logits for %d experts", ld, E);
+    const int warps = T >= 592 ? 4 : 1;                     // few tokens: a block each, side by side on the SMs
+    const size_t smem = (size_t)warps * (E + groups) * sizeof(float);       // at most 32 KB
+    qwb_launch(moe_route_kernel, (T + warps - 1) / warps, 32 * warps, smem, stream, logits, ld, correction, chosen, weight, gate_out, T, E, top,
+               sigmoid, groups, keep, renorm, sum_eps, weight_scale);
     return qwb_check_launch("moe_route");
 }
 
-template <typename T>
-__device__ __forceinline__ float warp_dot(const T* __restrict__ w, const T* __restrict__ x, int n, int lane) {
+// ---------------------------------------------------------------------------------
+// Rows of a matrix times vectors, a warp each: acc[r * NX + v] = this lane's part of w_r . x_v; rows `ldw` values apart, of
+// which the first nr exist, vectors `ldx` apart, of which the first nx exist (a missing one repeats the last).
+// ---------------------------------------------------------------------------------
+template <typename T, int NR, int NX>
+__device__ __forceinline__ void lane_dots(const T* __restrict__ w, size_t ldw, int nr, const T* __restrict__ x, size_t ldx, int nx, int n,
+                                          int lane, float* acc) {
     constexpr int VEC = Vec16<T>::N;
-    float acc = 0.f;
-    if (n % VEC == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)x % 16 == 0) {
-        const Vec16<T>* w16 = reinterpret_cast<const Vec16<T>*>(w);
-        const Vec16<T>* x16 = reinterpret_cast<const Vec16<T>*>(x);
-        for (int i = lane; i < n / VEC; i += 32) {
-            float a[VEC], b[VEC];
-            w16[i].get(a);
-            x16[i].get(b);
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) acc += a[e] * b[e];
+    for (int i = 0; i < NR * NX; ++i) acc[i] = 0.f;
+    const T* wr[NR];
+    const T* xv[NX];
+#pragma unroll
+    for (int r = 0; r < NR; ++r) wr[r] = w + (size_t)(r < nr ? r : nr - 1) * ldw;
+#pragma unroll
+    for (int v = 0; v < NX; ++v) xv[v] = x + (size_t)(v < nx ? v : nx - 1) * ldx;
+    if (n % VEC == 0 && ldw % VEC == 0 && (NX == 1 || ldx % VEC == 0) && (uintptr_t)w % 16 == 0 && (uintptr_t)x % 16 == 0) {
+#pragma unroll 2
+        for (int i = lane; i < n / VEC; i += 32) {
+            float a[NR][VEC];
+#pragma unroll
+            for (int r = 0; r < NR; ++r) reinterpret_cast<const Vec16<T>*>(wr[r])[i].get(a[r]);
+#pragma unroll
+            for (int v = 0; v < NX; ++v) {
+                float b[VEC];
+                reinterpret_cast<const Vec16<T>*>(xv[v])[i].get(b);
+#pragma unroll
+                for (int r = 0; r < NR; ++r)
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) acc[r * NX + v] += a[r][e] * b[e];
+            }
         }
     } else {
-        for (int i = lane; i < n; i += 32) acc += to_f32(w[i]) * to_f32(x[i]);
+        for (int i = lane; i < n; i += 32)
+#pragma unroll
+            for (int v = 0; v < NX; ++v) {
+                const float b = to_f32(xv[v][i]);
+#pragma unroll
+                for (int r = 0; r < NR; ++r) acc[r * NX + v] += to_f32(wr[r][i]) * b;
+            }
     }
-    return warp_sum(acc);
 }
 
-// grid (ceil(F / 8), T * top); 8 warps, a feature each
-template <typename T>
-__global__ void moe_gate_up_kernel(const T* __restrict__ x, const T* __restrict__ wgu, const int* __restrict__ chosen,
-                                   T* __restrict__ act, int D, int F, int top) {
+// grid (ceil(rows / 8), T * top + ceil(T / NT)): the copies of the tokens, then the shared expert with NT tokens a warp.
+// A warp makes two features of a plain expert, one of a gated one (its gate and its up row), two of the shared expert.
+template <typename T, int NT>
+__global__ void __launch_bounds__(256)
+moe_up_kernel(const T* __restrict__ x, const T* __restrict__ wu, const int* __restrict__ chosen, T* __restrict__ act,
+              const T* __restrict__ wsu, T* __restrict__ act_s, int n_tok, int D, int F, int Fs, int top, int kind) {
     pdl_wait();
     pdl_launch_dependents();
-    const int slot = blockIdx.y, t = slot / top;
-    const int f = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (f >= F) return;
-    const T* w = wgu + (size_t)chosen[slot] * 2 * F * D;
-    const T* xr = x + (size_t)t * D;
-    const float g = warp_dot(w + (size_t)f * D, xr, D, lane);
-    const float u = warp_dot(w + (size_t)(F + f) * D, xr, D, lane);
-    if (lane == 0) act[(size_t)slot * F + f] = from_f32<T>(g / (1.f + expf(-g)) * u);
-}
-
-// grid (ceil(D / 8), T); 8 warps, an output each
-template <typename T>
-__global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__ wd, const int* __restrict__ chosen,
-                                const float* __restrict__ weight, float* __restrict__ out, int D, int F, int top) {
-    pdl_wait();
-    pdl_launch_dependents();
-    const int t = blockIdx.y;
-    const int d = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (d >= D) return;
-    float total = 0.f;
-    for (int k = 0; k < top; ++k) {
-        const size_t slot = (size_t)t * top + k;
-        const T* w = wd + ((size_t)chosen[slot] * D + d) * F;
-        total += weight[slot] * warp_dot(w, act + slot * F, F, lane);
-    }
-    if (lane == 0) out[(size_t)t * D + d] = total;
-}
-
-extern "C" int qwb_moe_experts(const void* x, const void* wgu, const void* wd, const int* chosen, const float* weight,
-                               void* act, float* out, int dtype, int T, int D, int F, int top, cudaStream_t stream) {
-    if (T <= 0) return 0;
-    if (D <= 0 || F <= 0 || top <= 0) return qwb_fail(QWB_ERR_ARG, "moe_experts: width %d, expert width %d, %d choices", D, F, top);
-    if ((long long)T * top > 65535 || T > 65535) return qwb_fail(QWB_ERR_ARG, "moe_experts: %d tokens x %d choices are too many for one launch", T, top);
-    const dim3 g1((F + 7) / 8, T * top), g2((D + 7) / 8, T);
-    if (dtype == QWB_DT_F32) {
-        qwb_launch(moe_gate_up_kernel<float>, g1, 256, 0, stream, (const float*)x, (const float*)wgu, chosen, (float*)act, D, F, top);
-        qwb_launch(moe_down_kernel<float>, g2, 256, 0, stream, (const float*)act, (const float*)wd, chosen, weight, out, D, F, top);
-    } else if (dtype == QWB_DT_BF16) {
-        qwb_launch(moe_gate_up_kernel<bf16>, g1, 256, 0, stream, (const bf16*)x, (const bf16*)wgu, chosen, (bf16*)act, D, F, top);
-        qwb_launch(moe_down_kernel<bf16>, g2, 256, 0, stream, (const bf16*)act, (const bf16*)wd, chosen, weight, out, D, F, top);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int slot = blockIdx.y, n_slots = n_tok * top;
+    const int item = blockIdx.x * 8 + warp;
+    if (slot < n_slots) {
+        const bool gated = kind == QWB_MOE_GATED;
+        const int f = gated ? item : 2 * item;
+        if (f >= F) return;
+        const size_t first = (size_t)chosen[slot] * (gated ? 2 * F : F) + f;
+        float acc[2];
+        lane_dots<T, 2, 1>(wu + first * D, gated ? (size_t)F * D : (size_t)D, gated ? 2 : min(2, F - f), x + (size_t)(slot / top) * D, 0, 1, D,
+                           lane, acc);
+        const float a = warp_sum(acc[0]), b = warp_sum(acc[1]);
+        T* o = act + (size_t)slot * F + f;
+        if (gated) { if (lane == 0) o[0] = from_f32<T>(a / (1.f + expf(-a)) * b); }
+        else if (lane < min(2, F - f)) o[lane] = from_f32<T>(qwb_activate(lane ? b : a, kind));
     } else {
-        return qwb_fail(QWB_ERR_ARG, "moe_experts: unknown dtype %d", dtype);
+        const int t0 = (slot - n_slots) * NT, f = 2 * item;
+        if (f >= Fs) return;
+        const int nt = min(NT, n_tok - t0), nf = min(2, Fs - f);
+        float acc[2 * NT];
+        lane_dots<T, 2, NT>(wsu + (size_t)f * D, D, nf, x + (size_t)t0 * D, D, nt, D, lane, acc);
+#pragma unroll
+        for (int i = 0; i < 2 * NT; ++i) {
+            const float v = warp_sum(acc[i]);
+            if (lane == i && i / NT < nf && i % NT < nt)
+                act_s[(size_t)(t0 + i % NT) * Fs + f + i / NT] = from_f32<T>(qwb_activate(v, kind == QWB_MOE_GATED ? 3 : kind));
+        }
     }
+}
+
+// grid (ceil(D / NR), T), a warp per choice and one for the shared expert: NR outputs of one token; the warps' products
+// are weighted and summed in the order of the choices, the shared expert last.  out may be added onto (`onto`).
+template <typename T, int NR>
+__global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__ wd, const int* __restrict__ chosen,
+                                const float* __restrict__ weight, const T* __restrict__ act_s, const T* __restrict__ wsd,
+                                const float* __restrict__ gate, float* out, int D, int F, int Fs, int top, int onto) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float part[QWB_MOE_MAX_TOP + 1][NR];
+    const int t = blockIdx.y, d = blockIdx.x * NR;
+    const int k = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int nr = min(NR, D - d);
+    float acc[NR], mul;
+    if (k < top) {
+        const size_t slot = (size_t)t * top + k;
+        lane_dots<T, NR, 1>(wd + ((size_t)chosen[slot] * D + d) * F, F, nr, act + slot * F, 0, 1, F, lane, acc);
+        mul = weight[slot];
+    } else {
+        lane_dots<T, NR, 1>(wsd + (size_t)d * Fs, Fs, nr, act_s + (size_t)t * Fs, 0, 1, Fs, lane, acc);
+        mul = gate ? gate[t] : 1.f;
+    }
+#pragma unroll
+    for (int r = 0; r < NR; ++r) {
+        const float v = warp_sum(acc[r]);
+        if (lane == 0) part[k][r] = mul * v;
+    }
+    __syncthreads();
+    if (threadIdx.x < nr) {
+        float total = 0.f;
+        for (int i = 0; i < (int)(blockDim.x >> 5); ++i) total += part[i][threadIdx.x];
+        float* o = out + (size_t)t * D + d + threadIdx.x;
+        *o = onto ? *o + total : total;
+    }
+}
+
+template <typename T>
+static void launch_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight, const void* wsu,
+                               const void* wsd, const float* gate, void* act, void* act_s, float* out, int n_tok, int D, int F, int Fs,
+                               int top, int kind, int onto, cudaStream_t stream) {
+    const int items = kind == QWB_MOE_GATED ? F : (F + 1) / 2, items_s = Fs > 0 ? (Fs + 1) / 2 : 0;
+    const int rows = items > items_s ? items : items_s;
+    const int nt = n_tok > 1 ? 4 : 1;
+    const dim3 g1((rows + 7) / 8, n_tok * top + (Fs > 0 ? (n_tok + nt - 1) / nt : 0)), g2((D + 3) / 4, n_tok);
+    if (nt == 1)
+        qwb_launch(moe_up_kernel<T, 1>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
+    else
+        qwb_launch(moe_up_kernel<T, 4>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
+    qwb_launch(moe_down_kernel<T, 4>, g2, 32 * (top + (Fs > 0 ? 1 : 0)), 0, stream, (const T*)act, (const T*)wd, chosen, weight, (const T*)act_s,
+               (const T*)wsd, gate, out, D, F, Fs, top, onto);
+}
+
+// wsu [Fs, D], wsd [D, Fs], gate [T] (or null: 1), act_s [T, Fs]: the shared expert, Fs = 0 for none.
+extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight, const void* wsu,
+                               const void* wsd, const float* gate, void* act, void* act_s, float* out, int dtype, int T, int D, int F,
+                               int Fs, int top, int kind, int onto, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (D <= 0 || F <= 0 || Fs < 0 || top <= 0 || top > QWB_MOE_MAX_TOP)
+        return qwb_fail(QWB_ERR_ARG, "moe_experts: width %d, expert width %d, shared %d, %d choices", D, F, Fs, top);
+    if (Fs > 0 && (!wsu || !wsd || !act_s)) return qwb_fail(QWB_ERR_ARG, "moe_experts: a shared expert without its matrices");
+    if (kind != QWB_MOE_GATED && !qwb_activation_known(kind)) return qwb_fail(QWB_ERR_ARG, "moe_experts: unknown activation %d", kind);
+    if ((long long)T * top + T > 65535) return qwb_fail(QWB_ERR_ARG, "moe_experts: %d tokens x %d choices are too many for one launch", T, top);
+    if (dtype == QWB_DT_F32)
+        launch_moe_experts<float>(x, wu, wd, chosen, weight, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
+    else if (dtype == QWB_DT_BF16)
+        launch_moe_experts<bf16>(x, wu, wd, chosen, weight, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
+    else return qwb_fail(QWB_ERR_ARG, "moe_experts: unknown dtype %d", dtype);
     return qwb_check_launch("moe_experts");
 }
 
 // ---------------------------------------------------------------------------------
-// Around a grouped product over token copies sorted by expert (bfloat16):
-//   moe_gated_act  act[s, f] = silu(gu[s, f]) * gu[s, F + f]           gu [S, 2F] -> act [S, F]
-//   moe_combine    out[t, :] = sum_k weight[t, k] * y[place[t, k], :]   y [S, D] -> out float [T, D]
-// place[t, k] is the row of token t's k-th copy in the sorted order.
+// Around a grouped product over token copies sorted by expert (bfloat16; D and F multiples of 8):
+//   moe_sort      place[c] = the row of copy c = t * top + k in the order (expert, copy); ends[e] = where expert e's run ends
+//   moe_spread    xs[place[t, k], :] = x[t, :]
+//   moe_act       act[s, f] = f(u[s, f]), u [S, F], or silu(u[s, f]) * u[s, F + f], u [S, 2F]
+//   moe_combine   out[t, :] (+)= sum_k weight[t, k] * y[place[t, k], :] + gate[t] * shared[t, :]
 // ---------------------------------------------------------------------------------
-__global__ void moe_gated_act_kernel(const bf16* __restrict__ gu, bf16* __restrict__ act, size_t n, int F) {
+// One block; each warp counts and then places a run of neighbouring copies, 32 at a time (lanes with the same expert find
+// their ranks by __match_any_sync), so that nothing depends on the order in which warps run.
+#define MOE_SORT_WARPS 32
+__global__ void __launch_bounds__(MOE_SORT_WARPS * 32)
+moe_sort_kernel(const int* __restrict__ chosen, int* __restrict__ place, int* __restrict__ ends, int S, int E) {
     pdl_wait();
     pdl_launch_dependents();
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t r = i / F, f = i - r * F;
-        const float g = to_f32(gu[r * 2 * F + f]), u = to_f32(gu[r * 2 * F + F + f]);
-        act[i] = from_f32<bf16>(g / (1.f + expf(-g)) * u);
+    extern __shared__ int sort_smem[];
+    int* hist = sort_smem;                              // [warps][E]: counts, then the next row of each (warp, expert)
+    int* base = hist + MOE_SORT_WARPS * E;              // [E]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const unsigned full = 0xffffffffu;
+    for (int i = threadIdx.x; i < MOE_SORT_WARPS * E; i += blockDim.x) hist[i] = 0;
+    __syncthreads();
+    const int per = ((S + MOE_SORT_WARPS - 1) / MOE_SORT_WARPS + 31) & ~31;
+    const int lo = min(S, warp * per), hi = min(S, lo + per);
+    int* mine = hist + warp * E;
+    for (int i0 = lo; i0 < hi; i0 += 32) {
+        const int i = i0 + lane;
+        const int e = i < hi ? min(max(chosen[i], 0), E - 1) : -1;
+        const unsigned same = __match_any_sync(full, e);
+        if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
+        __syncwarp();
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+        int run = 0;
+#pragma unroll 8
+        for (int w = 0; w < MOE_SORT_WARPS; ++w) { const int c = hist[w * E + e]; hist[w * E + e] = run; run += c; }
+        base[e] = run;
+    }
+    __syncthreads();
+    if (warp == 0) {
+        int run = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int c = e0 + lane < E ? base[e0 + lane] : 0;
+            int s = c;
+            for (int o = 1; o < 32; o <<= 1) { const int up = __shfl_up_sync(full, s, o); if (lane >= o) s += up; }
+            if (e0 + lane < E) { base[e0 + lane] = run + s - c; ends[e0 + lane] = run + s; }
+            run += __shfl_sync(full, s, 31);
+        }
+    }
+    __syncthreads();
+    for (int i0 = lo; i0 < hi; i0 += 32) {
+        const int i = i0 + lane;
+        const int e = i < hi ? min(max(chosen[i], 0), E - 1) : -1;
+        const unsigned same = __match_any_sync(full, e);
+        if (e >= 0) place[i] = base[e] + mine[e] + __popc(same & ((1u << lane) - 1u));
+        __syncwarp();
+        if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
+        __syncwarp();
     }
 }
 
-extern "C" int qwb_moe_gated_act(const void* gu, void* act, int S, int F, cudaStream_t stream) {
-    if (S <= 0 || F <= 0) return 0;
-    const size_t n = (size_t)S * F;
-    const int block = 256, grid = (int)((n + block - 1) / block < 148 * 16 ? (n + block - 1) / block : 148 * 16);
-    qwb_launch(moe_gated_act_kernel, grid, block, 0, stream, (const bf16*)gu, (bf16*)act, n, F);
-    return qwb_check_launch("moe_gated_act");
+extern "C" int qwb_moe_sort(const int* chosen, int* place, int* ends, int S, int E, cudaStream_t stream) {
+    if (S <= 0) return 0;
+    if (E <= 0 || E > QWB_MOE_MAX_EXPERTS) return qwb_fail(QWB_ERR_ARG, "moe_sort: %d experts (at most %d)", E, QWB_MOE_MAX_EXPERTS);
+    const size_t smem = (size_t)(MOE_SORT_WARPS + 1) * E * sizeof(int);
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "moe_sort: %s", cudaGetErrorString(e));
+    }
+    qwb_launch(moe_sort_kernel, 1, MOE_SORT_WARPS * 32, smem, stream, chosen, place, ends, S, E);
+    return qwb_check_launch("moe_sort");
 }
 
-__global__ void moe_combine_kernel(const bf16* __restrict__ y, const long long* __restrict__ place, const float* __restrict__ weight,
-                                   float* __restrict__ out, int D, int top) {
+__global__ void moe_spread_kernel(const uint4* __restrict__ x, const int* __restrict__ place, uint4* __restrict__ xs, int pieces, int top) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
-    for (int d = threadIdx.x; d < D; d += blockDim.x) {
-        float total = 0.f;
-        for (int k = 0; k < top; ++k)
-            total += weight[(size_t)t * top + k] * to_f32(y[(size_t)place[(size_t)t * top + k] * D + d]);
-        out[(size_t)t * D + d] = total;
+    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+        const uint4 v = x[(size_t)t * pieces + i];
+        for (int k = 0; k < top; ++k) xs[(size_t)place[(size_t)t * top + k] * pieces + i] = v;
     }
 }
 
-extern "C" int qwb_moe_combine(const void* y, const long long* place, const float* weight, float* out, int T, int D, int top,
-                               cudaStream_t stream) {
+extern "C" int qwb_moe_spread(const void* x, const int* place, void* xs, int T, int D, int top, cudaStream_t stream) {
     if (T <= 0 || D <= 0) return 0;
-    qwb_launch(moe_combine_kernel, T, D >= 1024 ? 256 : 128, 0, stream, (const bf16*)y, place, weight, out, D, top);
+    if (D % 8) return qwb_fail(QWB_ERR_ARG, "moe_spread: rows of %d values", D);
+    qwb_launch(moe_spread_kernel, T, D >= 2048 ? 256 : 128, 0, stream, (const uint4*)x, place, (uint4*)xs, D / 8, top);
+    return qwb_check_launch("moe_spread");
+}
+
+__device__ __forceinline__ uint4 pack_bf16x8(const float* v) {
+    uint4 o;
+    uint32_t* w = reinterpret_cast<uint32_t*>(&o);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __nv_bfloat162 p = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        w[i] = *reinterpret_cast<const uint32_t*>(&p);
+    }
+    return o;
+}
+
+// grid (S, ...): a block per row; 8 values a thread
+__global__ void moe_act_kernel(const Vec16<bf16>* __restrict__ u, uint4* __restrict__ act, int pieces, int kind) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t s = blockIdx.x;
+    const bool gated = kind == QWB_MOE_GATED;
+    const Vec16<bf16>* row = u + s * (gated ? 2 * pieces : pieces);
+    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+        float a[8], b[8];
+        row[i].get(a);
+        if (gated) {
+            row[pieces + i].get(b);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) a[e] = a[e] / (1.f + expf(-a[e])) * b[e];
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) a[e] = qwb_activate(a[e], kind);
+        }
+        act[s * pieces + i] = pack_bf16x8(a);
+    }
+}
+
+extern "C" int qwb_moe_act(const void* u, void* act, int S, int F, int kind, cudaStream_t stream) {
+    if (S <= 0 || F <= 0) return 0;
+    if (F % 8) return qwb_fail(QWB_ERR_ARG, "moe_act: rows of %d values", F);
+    if (kind != QWB_MOE_GATED && !qwb_activation_known(kind)) return qwb_fail(QWB_ERR_ARG, "moe_act: unknown activation %d", kind);
+    qwb_launch(moe_act_kernel, S, F >= 2048 ? 256 : 128, 0, stream, (const Vec16<bf16>*)u, (uint4*)act, F / 8, kind);
+    return qwb_check_launch("moe_act");
+}
+
+__global__ void moe_combine_kernel(const Vec16<bf16>* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weight,
+                                   const float* __restrict__ shared, const float* __restrict__ gate, float* out, int pieces, int top,
+                                   int onto) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const float g = gate ? gate[t] : 1.f;
+    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+        float total[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) total[e] = 0.f;
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) {
+            float v[8];
+            y[(size_t)place[(size_t)t * top + k] * pieces + i].get(v);
+            const float w = weight[(size_t)t * top + k];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) total[e] += w * v[e];
+        }
+        float4* o = reinterpret_cast<float4*>(out) + ((size_t)t * pieces + i) * 2;
+        const float4* sh = reinterpret_cast<const float4*>(shared) + ((size_t)t * pieces + i) * 2;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            float4 r = make_float4(total[4 * j], total[4 * j + 1], total[4 * j + 2], total[4 * j + 3]);
+            if (shared) { const float4 s = sh[j]; r.x += g * s.x; r.y += g * s.y; r.z += g * s.z; r.w += g * s.w; }
+            if (onto) { const float4 s = o[j]; r.x += s.x; r.y += s.y; r.z += s.z; r.w += s.w; }
+            o[j] = r;
+        }
+    }
+}
+
+// y [S, D] bfloat16; shared [T, D] float (or null) and gate [T] (or null: 1)
+extern "C" int qwb_moe_combine(const void* y, const int* place, const float* weight, const float* shared, const float* gate, float* out,
+                               int T, int D, int top, int onto, cudaStream_t stream) {
+    if (T <= 0 || D <= 0) return 0;
+    if (D % 8) return qwb_fail(QWB_ERR_ARG, "moe_combine: rows of %d values", D);
+    qwb_launch(moe_combine_kernel, T, D >= 2048 ? 256 : 128, 0, stream, (const Vec16<bf16>*)y, place, weight, shared, gate, out, D / 8, top, onto);
     return qwb_check_launch("moe_combine");
 }

@@ -142,6 +142,8 @@ class Engine:
             max_seq_len = max_tokens
             if self.plan.max_position:
                 max_seq_len = min(max_seq_len, self.plan.max_position)
+        if self.plan.position_limit and max_seq_len > self.plan.position_limit:
+            raise EngineError(f"max_seq_len {max_seq_len}: this model has {self.plan.position_limit} positions")
         max_seq_len = min(max_seq_len, pages_for(max_tokens) * PAGE_SIZE)
         if max_batch is None:
             max_batch = max(1, min(256, pages_for(max_tokens)))

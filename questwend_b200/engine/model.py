@@ -88,7 +88,7 @@ class Model:
         stands there (what is still to be added is added first: slower, for looking at a model layer by layer)."""
         for position in self._positions.values():       # the step's tables first: no layer's kernels find them half made
             position.prepare(ctx)
-        h = self.embedding.forward(ctx.token_ids)
+        h = self.embedding.forward(ctx.token_ids, ctx.tok_pos)
         delta = None
         for i, run in enumerate(self.schedule):
             if self.before[i] is not None:              # adds onto the stream; what is pending in ``delta`` stays pending

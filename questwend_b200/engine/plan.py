@@ -44,7 +44,8 @@ class ModelPlan:
     final_norm: PartSpec
     head: PartSpec
     stop_token_ids: tuple = ()
-    max_position: int | None = None
+    max_position: int | None = None     # the trained length: the default for an engine's longest sequence
+    position_limit: int | None = None   # no position at or above this exists (a learned table's rows): a hard limit
     extra: dict = field(default_factory=dict)
 
     def validate(self) -> None:

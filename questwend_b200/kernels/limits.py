@@ -18,6 +18,7 @@ SCAN_MAX_ROWS = 512         # rows of a recurrent state's column that one warp k
 LATENT_MAX_RANK = 512       # csrc/attention_latent.cu: QWB_LATENT_MAX_L
 LATENT_MAX_ROW = 1024       # ... QWB_LATENT_MAX_ROW
 MOE_MAX_TOP = 16            # csrc/moe.cu: QWB_MOE_MAX_TOP
+MOE_MAX_EXPERTS = 1024      # ... QWB_MOE_MAX_EXPERTS
 
 
 def conv_taps_refusal(taps: int) -> str | None:
@@ -41,9 +42,16 @@ def latent_refusal(rank: int, rot_dim: int) -> str | None:
     return None
 
 
-def moe_refusal(experts: int, top: int) -> str | None:
+def moe_refusal(experts: int, top: int, groups: int = 1, keep: int = 1) -> str | None:
+    """``groups`` equal groups of neighbouring experts, of which the router keeps ``keep``."""
     if experts <= 0 or not 1 <= top <= min(experts, MOE_MAX_TOP):
         return f"the router chooses 1 to {MOE_MAX_TOP} of its experts, not {top} of {experts}"
+    if experts > MOE_MAX_EXPERTS:
+        return f"the router takes up to {MOE_MAX_EXPERTS} experts, not {experts}"
+    if groups < 1 or experts % groups:
+        return f"{experts} experts do not form {groups} equal groups"
+    if not 1 <= keep <= groups or top > keep * (experts // groups):
+        return f"the router cannot choose {top} experts from {keep} of {groups} groups of {experts // groups}"
     return None
 
 

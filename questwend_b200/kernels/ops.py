@@ -82,14 +82,23 @@ _f = ctypes.c_float
 
 
 # ----------------------------------------------------------------------------- elementwise
-def embed_gather(ids: torch.Tensor, table: torch.Tensor, bad_token: torch.Tensor | None = None, scale: float = 1.0) -> torch.Tensor:
-    """Rows of ``table`` [V, D] for int32 ``ids`` [T], times ``scale``, as float32 [T, D]."""
+def embed_gather(ids: torch.Tensor, table: torch.Tensor, bad_token: torch.Tensor | None = None, scale: float = 1.0,
+                 pos_table: torch.Tensor | None = None, positions: torch.Tensor | None = None) -> torch.Tensor:
+    """Rows of ``table`` [V, D] for int32 ``ids`` [T], times ``scale``, as float32 [T, D]; with ``pos_table`` [P, D] (the
+    table's dtype) plus its row ``positions[t]`` (int32 [T])."""
     _need(ids, "ids", torch.int32, 1)
     _need(table, "table", ndim=2)
     T, (V, D) = ids.numel(), table.shape
+    NP = 0
+    if pos_table is not None:
+        _need(pos_table, "pos_table", table.dtype, 2)
+        _need(positions, "positions", torch.int32, 1)
+        NP = pos_table.shape[0]
+        if pos_table.shape[1] != D or positions.numel() != T:
+            raise KernelError(f"embed_gather: position table {tuple(pos_table.shape)}, {positions.numel()} positions for {T} rows of {D}")
     out = torch.empty((T, D), dtype=torch.float32, device=table.device)
-    _call("elementwise", "qwb_embed_gather", _ptr(ids), _ptr(table), _i(_dt(table.dtype)), _ptr(out),
-          _i(T), _i(D), _i(V), _ptr(bad_token), _f(scale), _stream())
+    _call("elementwise", "qwb_embed_gather", _ptr(ids), _ptr(table), _i(_dt(table.dtype)), _ptr(positions if NP else None),
+          _ptr(pos_table), _ptr(out), _i(T), _i(D), _i(V), _i(NP), _ptr(bad_token), _f(scale), _stream())
     return out
 
 
@@ -233,7 +242,7 @@ def rmsnorm_mix(h: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: flo
     return h if cast is None else cast
 
 
-ACTIVATIONS = {"none": 0, "relu2": 1, "gelu_tanh": 2, "silu": 3, "xielu": 4}
+ACTIVATIONS = {"none": 0, "relu2": 1, "gelu_tanh": 2, "silu": 3, "xielu": 4, "gelu": 5}     # gelu: the exact (erf) form
 ACTIVATION_PARAMS = {"xielu": 2}    # activations with learned numbers of their own, and how many
 
 
@@ -1137,7 +1146,8 @@ def pool_attention(q: torch.Tensor, k_pool, v_pool, pk_pool, pv_pool, page_table
                    scale: float, window: int, pool: int, interleaved: bool, impl: str = "auto") -> torch.Tensor:
     """Attention of a step's tokens over their window and the block rows before it.  ``q`` [T, H, dim] in the cache's
     dtype; returns [T, H * vdim] in that dtype, each head turned back by the query's position if ``cos_v`` is given.
-    Steps of one token per sequence take the kernel that cuts the keys into runs (sizes that are multiples of 8); other
+    Steps of one token per sequence take the kernels that cut the keys into runs (one uncapped map over all keys with keys
+    and values of 64 or 128: plain grouped-query attention's; other sizes that are multiples of 8: the one for maps); other
     steps the tensor-core kernel where it fits (``impl`` "auto" or "mma"), else the plain one ("plain")."""
     _need(q, "q", k_pool.dtype, 3)
     T, H, dim = q.shape
@@ -1180,11 +1190,13 @@ MAPS_FAST_STEP = 8          # key and value sizes that are multiples of this tak
 
 def maps_prep(qkv: torch.Tensor, bias, q_weight, k_weight, cos, sin, ctx, page_table, k_pool, v_pool, n_heads: int,
               n_kv_heads: int, maps: int, dim: int, vdim: int, rotary_dim: int, interleaved: bool, eps: float,
-              store_kv: bool = True) -> torch.Tensor:
+              store_kv: bool = True, whole_norm: bool = False, temp_coef: float = 0.0, temp_every: float = 1.0) -> torch.Tensor:
     """Bias (float32 over all columns, or None), per-map RMS norm of q and k (weights [dim] shared by heads and maps, or
     None), rotation of the first ``rotary_dim`` values of every map of q and k, cache write.  ``qkv`` float32
     [T, (H + G) * maps * dim + G * vdim]; the pools [pages, G, 64, maps * dim] / [pages, G, 64, vdim].  Returns q
-    [T, H, maps * dim] in the cache's dtype."""
+    [T, H, maps * dim] in the cache's dtype.  ``whole_norm``: one norm over all of q (weights [H * maps * dim]) and one over
+    all of k ([G * maps * dim]) instead; with it q is multiplied by 1 + ``temp_coef`` ln(floor((p + 1) / ``temp_every``) + 1)
+    at position p."""
     _need(qkv, "qkv", torch.float32, 2)
     T = qkv.shape[0]
     ld = (n_heads + n_kv_heads) * maps * dim + n_kv_heads * vdim
@@ -1192,11 +1204,14 @@ def maps_prep(qkv: torch.Tensor, bias, q_weight, k_weight, cos, sin, ctx, page_t
         raise KernelError(f"maps_prep: qkv {tuple(qkv.shape)} for {n_heads}+{n_kv_heads} heads of {maps} x {dim}, values of {vdim}")
     if tuple(k_pool.shape[1:]) != (n_kv_heads, PAGE_SIZE, maps * dim) or tuple(v_pool.shape[1:]) != (n_kv_heads, PAGE_SIZE, vdim):
         raise KernelError(f"maps_prep: pools {tuple(k_pool.shape)}, {tuple(v_pool.shape)} do not fit")
-    for name, t, n in (("bias", bias, ld), ("q_weight", q_weight, dim), ("k_weight", k_weight, dim)):
+    norm_sizes = (n_heads * maps * dim, n_kv_heads * maps * dim) if whole_norm else (dim, dim)
+    for name, t, n in (("bias", bias, ld), ("q_weight", q_weight, norm_sizes[0]), ("k_weight", k_weight, norm_sizes[1])):
         if t is not None:
             _need(t, name, torch.float32, 1)
             if t.numel() != n:
                 raise KernelError(f"maps_prep: {name} of {t.numel()}, wanted {n}")
+    if temp_coef and not whole_norm:
+        raise KernelError("maps_prep: the factor on q by its position goes with norms over whole projections")
     if cos is None:
         rotary_dim = 0
     for name, t in (("cos", cos), ("sin", sin)):
@@ -1205,6 +1220,12 @@ def maps_prep(qkv: torch.Tensor, bias, q_weight, k_weight, cos, sin, ctx, page_t
             if tuple(t.shape) != (T, rotary_dim // 2):
                 raise KernelError(f"maps_prep: table {name} {tuple(t.shape)} for {T} tokens and {rotary_dim} turned values")
     q = torch.empty((T, n_heads, maps * dim), dtype=k_pool.dtype, device=qkv.device)
+    if whole_norm:
+        _call("attention_maps", "qwb_maps_row_prep", _ptr(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos), _ptr(sin),
+              _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(page_table), _i(page_table.shape[1]), _ptr(q), _ptr(k_pool), _ptr(v_pool),
+              _i(_dt(k_pool.dtype)), _i(T), _i(n_heads), _i(n_kv_heads), _i(maps), _i(dim), _i(vdim), _i(rotary_dim),
+              _i(1 if interleaved else 0), _f(eps), _f(temp_coef), _f(temp_every), _i(1 if store_kv else 0), _stream())
+        return q
     _call("attention_maps", "qwb_maps_prep", _ptr(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos), _ptr(sin),
           _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(page_table), _i(page_table.shape[1]), _ptr(q), _ptr(k_pool), _ptr(v_pool),
           _i(_dt(k_pool.dtype)), _i(T), _i(n_heads), _i(n_kv_heads), _i(maps), _i(dim), _i(vdim), _i(rotary_dim),
@@ -1237,6 +1258,9 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
     dim = kdim // maps
     out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
     width = page_table.shape[1]
+    plain = maps == 1 and softcap <= 0.0 and not norm_out and out_scale == 1.0 and dim == vdim
+    if ctx.single_token and impl == "auto" and plain and chunk == 0 and mma_attention_fits(q.dtype, dim, k_pool.shape[2]):
+        return attn_decode(q, k_pool, v_pool, page_table, ctx.seq_len, scale, ctx.max_len)
     if ctx.single_token and dim % MAPS_FAST_STEP == 0 and vdim % MAPS_FAST_STEP == 0:
         lib = _lookup("attention_maps", "qwb_maps_decode_runs")[0]
         n_runs = lib.qwb_maps_decode_runs(_i(ctx.max_len), _i(chunk))
@@ -1248,7 +1272,7 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
               _f(softcap), _i(chunk), _i(n_runs), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), _stream(), kernels=2)
         return out
     # one map, no cap, keys and values of one size: the prompt kernel of plain grouped-query attention, with the chunk mask
-    if (impl in ("auto", "tc") and maps == 1 and softcap <= 0.0 and dim == vdim and q.dtype == torch.bfloat16
+    if (impl in ("auto", "tc") and plain and q.dtype == torch.bfloat16
             and ctx.max_new * (H // G) >= 64 and tc_attention_fits(q.dtype, dim, k_pool.shape[2], H // G)):
         return attn_prefill(q, k_pool, v_pool, page_table, ctx.cu_seqlens, ctx.pos0, ctx.max_new, scale, impl="tc", chunk=chunk)
     if impl == "mma" or (impl == "auto" and maps_prefill_mma_fits(q.dtype, maps, dim, vdim)):
@@ -1521,84 +1545,137 @@ def latent_attention(q_abs: torch.Tensor, q_rot: torch.Tensor, pool: torch.Tenso
 
 # ----------------------------------------------------------------------------- routed experts
 MOE_MAX_TOP = 16            # csrc/moe.cu: QWB_MOE_MAX_TOP
+MOE_ACTIVATIONS = {"gated_silu": 16, **{k: v for k, v in ACTIVATIONS.items() if k not in ACTIVATION_PARAMS}}
+MOE_SCORES = ("softmax", "sigmoid")
 _MOE_SLOTS_PER_LAUNCH = 65535
 
 
-def moe_route(logits: torch.Tensor, top: int, renormalize: bool = False):
-    """softmax over float32 ``logits`` [T, E]; the ``top`` largest per row (ties to the lower index).  Returns
-    (chosen int32 [T, top], weight float32 [T, top]): the chosen scores, divided by their sum if ``renormalize``."""
+def moe_route(logits: torch.Tensor, top: int, renormalize: bool = False, experts: int | None = None, scores: str = "softmax",
+              correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1, sum_eps: float = 0.0,
+              weight_scale: float = 1.0, gate: bool = False):
+    """The router's choice from float32 ``logits`` [T, >= experts] (default: all columns).  Scores are the softmax or the
+    sigmoid of the logits; chosen are the ``top`` largest scores (ties to the lower index), plus ``correction`` [experts]
+    if given, inside the ``keep`` of ``groups`` equal groups of neighbours whose two largest choice scores sum highest.
+    Returns (chosen int32 [T, top], weight float32 [T, top]): the chosen scores, divided by their sum + ``sum_eps`` if
+    ``renormalize``, times ``weight_scale``; with ``gate`` also float32 [T], the sigmoid of the column after the experts'."""
     _need(logits, "logits", torch.float32, 2)
-    T, E = logits.shape
+    T, ld = logits.shape
+    E = ld if experts is None else experts
+    if scores not in MOE_SCORES:
+        raise KernelError(f"moe_route: unknown scores '{scores}'")
+    if correction is not None:
+        _need(correction, "correction", torch.float32, 1)
+        if correction.numel() != E:
+            raise KernelError(f"moe_route: correction of {correction.numel()} for {E} experts")
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weight = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    _call("moe", "qwb_moe_route", _ptr(logits), _ptr(chosen), _ptr(weight), _i(T), _i(E), _i(top),
-          _i(1 if renormalize else 0), _stream())
-    return chosen, weight
+    gate_out = torch.empty((T,), dtype=torch.float32, device=logits.device) if gate else None
+    _call("moe", "qwb_moe_route", _ptr(logits), _i(ld), _ptr(correction), _ptr(chosen), _ptr(weight), _ptr(gate_out), _i(T), _i(E),
+          _i(top), _i(MOE_SCORES.index(scores)), _i(groups), _i(keep), _i(1 if renormalize else 0), _f(sum_eps), _f(weight_scale), _stream())
+    return (chosen, weight, gate_out) if gate else (chosen, weight)
 
 
-def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor,
-                weight: torch.Tensor) -> torch.Tensor:
-    """sum_k weight[t, k] * down_e(silu(gate_e x_t) * up_e x_t), e = chosen[t, k].  ``x`` [T, D] and the stacked
-    weights (``w_gate_up`` [E, 2F, D]: gate rows, then up rows; ``w_down`` [E, D, F]) in one dtype.  Returns float32 [T, D]."""
-    _need(x, "x", w_gate_up.dtype, 2)
-    _need(w_gate_up, "w_gate_up", ndim=3)
-    _need(w_down, "w_down", w_gate_up.dtype, 3)
+def _moe_sizes(what, x, w_up, w_down, chosen, weight, kind):
+    _need(x, "x", w_up.dtype, 2)
+    _need(w_up, "w_up", ndim=3)
+    _need(w_down, "w_down", w_up.dtype, 3)
     _need(chosen, "chosen", torch.int32, 2)
     _need(weight, "weight", torch.float32, 2)
+    if kind not in MOE_ACTIVATIONS:
+        raise KernelError(f"{what}: unknown activation '{kind}'")
     T, D = x.shape
-    E, F2, _ = w_gate_up.shape
-    F, top = F2 // 2, chosen.shape[1]
-    if w_gate_up.shape[2] != D or tuple(w_down.shape) != (E, D, F) or tuple(chosen.shape) != (T, top) or weight.shape != chosen.shape:
-        raise KernelError(f"moe_experts: x {tuple(x.shape)}, gate/up {tuple(w_gate_up.shape)}, down {tuple(w_down.shape)}, "
+    E, rows, _ = w_up.shape
+    F, top = (rows // 2 if kind == "gated_silu" else rows), chosen.shape[1]
+    if w_up.shape[2] != D or tuple(w_down.shape) != (E, D, F) or tuple(chosen.shape) != (T, top) or weight.shape != chosen.shape:
+        raise KernelError(f"{what}: x {tuple(x.shape)}, up {tuple(w_up.shape)}, down {tuple(w_down.shape)}, "
                           f"chosen {tuple(chosen.shape)}")
+    return T, D, E, F, top
+
+
+def moe_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor, weight: torch.Tensor,
+                activation: str = "gated_silu", shared_up: torch.Tensor | None = None, shared_down: torch.Tensor | None = None,
+                gate: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """sum_k weight[t, k] * down_e(act(up_e x_t)), e = chosen[t, k].  ``x`` [T, D] and the stacked weights (``w_up``
+    [E, F, D]; "gated_silu": [E, 2F, D], gate rows, then up rows, silu(gate x) * up x; ``w_down`` [E, D, F]) in one dtype.
+    A shared expert (``shared_up`` [Fs, D], ``shared_down`` [D, Fs], the same activation, plain) is added for every token,
+    times ``gate`` [T] if given.  Returns float32 [T, D], or adds onto ``out`` if that is given."""
+    T, D, E, F, top = _moe_sizes("moe_experts", x, w_up, w_down, chosen, weight, activation)
+    Fs = 0
+    if shared_up is not None:
+        _need(shared_up, "shared_up", x.dtype, 2)
+        _need(shared_down, "shared_down", x.dtype, 2)
+        Fs = shared_up.shape[0]
+        if activation == "gated_silu" or shared_up.shape[1] != D or tuple(shared_down.shape) != (D, Fs):
+            raise KernelError(f"moe_experts: shared expert {tuple(shared_up.shape)}, {tuple(shared_down.shape)} ({activation})")
+    if gate is not None:
+        _need(gate, "gate", torch.float32, 1)
+    onto = out is not None
+    if onto:
+        _need(out, "out", torch.float32, 2)
+        if tuple(out.shape) != (T, D):
+            raise KernelError(f"moe_experts: out {tuple(out.shape)} for {T} x {D}")
+    else:
+        out = torch.empty((T, D), dtype=torch.float32, device=x.device)
     act = torch.empty((T * top, F), dtype=x.dtype, device=x.device)
-    out = torch.empty((T, D), dtype=torch.float32, device=x.device)
-    per = max(1, _MOE_SLOTS_PER_LAUNCH // top)
+    act_s = torch.empty((T, Fs), dtype=x.dtype, device=x.device) if Fs else None
+    per = max(1, _MOE_SLOTS_PER_LAUNCH // (top + 1))
     for t0 in range(0, T, per):
         n = min(per, T - t0)
-        _call("moe", "qwb_moe_experts", _ptr(x[t0:t0 + n]), _ptr(w_gate_up), _ptr(w_down), _ptr(chosen[t0:t0 + n]),
-              _ptr(weight[t0:t0 + n]), _ptr(act[t0 * top:(t0 + n) * top]), _ptr(out[t0:t0 + n]), _i(_dt(x.dtype)), _i(n),
-              _i(D), _i(F), _i(top), _stream(), kernels=2)
+        cut = (lambda t: None if t is None else t[t0:t0 + n])
+        _call("moe", "qwb_moe_experts", _ptr(cut(x)), _ptr(w_up), _ptr(w_down), _ptr(cut(chosen)), _ptr(cut(weight)), _ptr(shared_up),
+              _ptr(shared_down), _ptr(cut(gate)), _ptr(act[t0 * top:(t0 + n) * top]), _ptr(cut(act_s)), _ptr(cut(out)), _i(_dt(x.dtype)),
+              _i(n), _i(D), _i(F), _i(Fs), _i(top), _i(MOE_ACTIVATIONS[activation]), _i(1 if onto else 0), _stream(), kernels=2)
     return out
 
 
 MOE_GROUPED_MIN_TOKENS = 17     # from here on bfloat16 tokens are sorted by expert and go through the library's grouped product
 
 
-def moe_grouped_fits(x: torch.Tensor, w_gate_up: torch.Tensor) -> bool:
+def moe_grouped_fits(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor) -> bool:
     """Whether a step's tokens take the sorted, grouped form (else the expert-streaming kernels do)."""
-    D, F = w_gate_up.shape[2], w_gate_up.shape[1] // 2
+    D, F = w_down.shape[1], w_down.shape[2]
     return (x.dtype == torch.bfloat16 and x.shape[0] >= MOE_GROUPED_MIN_TOKENS and D % 8 == 0 and F % 8 == 0
             and hasattr(torch, "_grouped_mm"))
 
 
-def moe_experts_grouped(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor,
-                        weight: torch.Tensor) -> torch.Tensor:
-    """``moe_experts`` for many bfloat16 tokens: the tokens' copies are sorted by expert (a stable sort: nothing depends
-    on the order in which blocks finish), each expert's run goes through the library's grouped matrix product (32-bit
-    sums, bfloat16 results) for gate/up and for down, with the gated SiLU between them and the weighted sum of every
-    token's copies after them in kernels of this library.  No value is read on the host."""
-    _need(x, "x", torch.bfloat16, 2)
-    _need(w_gate_up, "w_gate_up", torch.bfloat16, 3)
-    _need(w_down, "w_down", torch.bfloat16, 3)
+def moe_sort(chosen: torch.Tensor, experts: int):
+    """Copies of tokens in the order (expert, copy): (place int32 [T, top], the row of each copy; ends int32 [experts],
+    where each expert's run ends)."""
     _need(chosen, "chosen", torch.int32, 2)
-    _need(weight, "weight", torch.float32, 2)
-    T, D = x.shape
-    E, F2, _ = w_gate_up.shape
-    F, top = F2 // 2, chosen.shape[1]
-    flat = chosen.view(-1)
-    order = torch.argsort(flat, stable=True)                        # sorted row -> copy (t * top + k)
-    ends = torch.searchsorted(flat.index_select(0, order), torch.arange(E, dtype=torch.int32, device=x.device),
-                              right=True).to(torch.int32)           # where each expert's run ends (no value read on the host)
-    place = torch.empty_like(order)
-    place[order] = torch.arange(order.numel(), device=x.device)     # copy -> sorted row
-    xs = x.index_select(0, order // top)
-    gu = torch._grouped_mm(xs, w_gate_up.transpose(1, 2), offs=ends).contiguous()
+    place = torch.empty_like(chosen)
+    ends = torch.empty((experts,), dtype=torch.int32, device=chosen.device)
+    _call("moe", "qwb_moe_sort", _ptr(chosen), _ptr(place), _ptr(ends), _i(chosen.numel()), _i(experts), _stream())
+    return place, ends
+
+
+def moe_experts_grouped(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor, weight: torch.Tensor,
+                        activation: str = "gated_silu", shared: torch.Tensor | None = None, gate: torch.Tensor | None = None,
+                        out: torch.Tensor | None = None) -> torch.Tensor:
+    """``moe_experts`` for many bfloat16 tokens: the tokens' copies are sorted by expert (in an order that does not depend
+    on which blocks finish first), each expert's run goes through the library's grouped matrix product (32-bit sums,
+    bfloat16 results) for up and for down, with the activation between them and the weighted sum of every token's copies
+    after them in kernels of this library.  No value is read on the host.  ``shared``: the shared expert's output float32
+    [T, D], added times ``gate`` [T] in the last kernel."""
+    T, D, E, F, top = _moe_sizes("moe_experts_grouped", x, w_up, w_down, chosen, weight, activation)
+    if x.dtype != torch.bfloat16:
+        raise KernelError(f"moe_experts_grouped: takes bfloat16, not {x.dtype}")
+    for name, t, shape in (("shared", shared, (T, D)), ("gate", gate, (T,)), ("out", out, (T, D))):
+        if t is not None:
+            _need(t, name, torch.float32, len(shape))
+            if tuple(t.shape) != shape:
+                raise KernelError(f"moe_experts_grouped: {name} {tuple(t.shape)}, wanted {shape}")
+    place, ends = moe_sort(chosen, E)
+    xs = torch.empty((T * top, D), dtype=torch.bfloat16, device=x.device)
+    _call("moe", "qwb_moe_spread", _ptr(x), _ptr(place), _ptr(xs), _i(T), _i(D), _i(top), _stream())
+    u = torch._grouped_mm(xs, w_up.transpose(1, 2), offs=ends).contiguous()
     act = torch.empty((T * top, F), dtype=torch.bfloat16, device=x.device)
-    _call("moe", "qwb_moe_gated_act", _ptr(gu), _ptr(act), _i(T * top), _i(F), _stream())
+    _call("moe", "qwb_moe_act", _ptr(u), _ptr(act), _i(T * top), _i(F), _i(MOE_ACTIVATIONS[activation]), _stream())
     y = torch._grouped_mm(act, w_down.transpose(1, 2), offs=ends).contiguous()
-    out = torch.empty((T, D), dtype=torch.float32, device=x.device)
-    _call("moe", "qwb_moe_combine", _ptr(y), _ptr(place), _ptr(weight), _ptr(out), _i(T), _i(D), _i(top), _stream())
+    onto = out is not None
+    if not onto:
+        out = torch.empty((T, D), dtype=torch.float32, device=x.device)
+    _call("moe", "qwb_moe_combine", _ptr(y), _ptr(place), _ptr(weight), _ptr(shared), _ptr(gate), _ptr(out), _i(T), _i(D), _i(top),
+          _i(1 if onto else 0), _stream())
     return out
 
 

@@ -227,11 +227,13 @@ class ScoreMapsAttention(Mixer):
     square over the value size (eps inside the root) and multiplied by 1 - ``diff``.  In front of the scores, in this
     order and each optional: biases on q, k and v, a short causal convolution over time on every channel of q, k and v
     (``conv`` taps, no activation; its last inputs are per-sequence state), an RMS norm of every map of q and k with a
-    weight shared by heads and maps, and a rotation of the first part of every map.
+    weight shared by heads and maps (``qk_norm_over`` "head") or of the whole projections of q and of k with weights of
+    their sizes ("projection"), a rotation of the first part of every map, and (with "projection") a factor on q that
+    grows with its position p, 1 + ``q_temp_coef`` ln(floor((p + 1) / ``q_temp_every``) + 1).
 
     params: hidden_size, n_heads, n_kv_heads, head_dim, value_dim, maps (default 1), biases (q, k, v), out_bias, conv
-    (0: none), qk_norm, norm_eps, scale (default 1/sqrt(head_dim)), softcap (0: none), chunk (0: plain causal), diff,
-    layout ("halves": pairs (i, i + n/2); "interleaved": (2i, 2i + 1)), names (optional overrides).  ``position``: an
+    (0: none), qk_norm, qk_norm_over (default "head"), norm_eps, q_temp_coef (0: none), q_temp_every, scale (default
+    1/sqrt(head_dim)), softcap (0: none), chunk (0: plain causal), diff, layout ("halves": pairs (i, i + n/2); "interleaved": (2i, 2i + 1)), names (optional overrides).  ``position``: an
     encoding that gives cos and sin [T, n/2].
     The cache: keys (all maps of a head in one row) and values per token; with a convolution also its tail."""
 
@@ -239,6 +241,7 @@ class ScoreMapsAttention(Mixer):
              "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "q_norm": "q.norm", "k_norm": "k.norm",
              "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2"}
     LAYOUTS = ("halves", "interleaved")
+    NORMS = ("head", "projection")
 
     def __init__(self, spec, runtime, position=None):
         super().__init__(spec, runtime)
@@ -251,6 +254,8 @@ class ScoreMapsAttention(Mixer):
         self.biases, self.out_bias = bool(p.get("biases", False)), bool(p.get("out_bias", False))
         self.taps = int(p.get("conv", 0) or 0)
         self.qk_norm = bool(p.get("qk_norm", False))
+        self.norm_over = str(p.get("qk_norm_over", "head"))
+        self.temp_coef, self.temp_every = float(p.get("q_temp_coef", 0.0)), float(p.get("q_temp_every", 1.0))
         self.eps = float(p.get("norm_eps", 0.0))
         self.scale = float(p.get("scale", 1.0 / math.sqrt(self.head_dim)))
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
@@ -264,6 +269,11 @@ class ScoreMapsAttention(Mixer):
             raise ValueError(f"{self.n_heads} heads are not a multiple of {self.n_kv_heads} key/value heads")
         if self.layout not in self.LAYOUTS:
             raise ValueError(f"attention '{self.prefix}': layout '{self.layout}' is not one of {', '.join(self.LAYOUTS)}")
+        if self.norm_over not in self.NORMS:
+            raise ValueError(f"attention '{self.prefix}': qk_norm_over '{self.norm_over}' is not one of {', '.join(self.NORMS)}")
+        if self.temp_coef and (self.norm_over != "projection" or not self.temp_every > 0):
+            raise ValueError(f"attention '{self.prefix}': a factor on q by its position goes with norms over the whole projection "
+                             f"and a positive step, not '{self.norm_over}' and {self.temp_every}")
         for refusal in (maps_attention_refusal(self.maps, self.head_dim, self.value_dim),
                         conv_taps_refusal(self.taps) if self.taps else None):
             if refusal:
@@ -288,8 +298,9 @@ class ScoreMapsAttention(Mixer):
         if self.taps:
             out += [TensorSpec(px + n[x + "_conv"], (sizes[x], self.taps), VECTOR) for x in "qkv"]
         if self.qk_norm:
-            out += [TensorSpec(px + n["q_norm"], (self.head_dim,), VECTOR, NORM_WEIGHT),
-                    TensorSpec(px + n["k_norm"], (self.head_dim,), VECTOR, NORM_WEIGHT)]
+            whole = self.norm_over == "projection"
+            out += [TensorSpec(px + n["q_norm"], (self.n_q if whole else self.head_dim,), VECTOR, NORM_WEIGHT),
+                    TensorSpec(px + n["k_norm"], (self.n_k if whole else self.head_dim,), VECTOR, NORM_WEIGHT)]
         if self.maps == 2:
             out += [TensorSpec(px + n[x], (self.head_dim,), VECTOR) for x in ("lq1", "lk1", "lq2", "lk2")]
         return out
@@ -315,7 +326,9 @@ class ScoreMapsAttention(Mixer):
         mods = ["attention_maps", "rope_kv", "elementwise", *(("recurrent",) if self.taps else ()), *linear_modules(self.runtime.dtype)]
         if (self.maps == 1 and self.softcap <= 0.0 and self.head_dim == self.value_dim
                 and ops.tc_attention_fits(self.runtime.dtype, self.head_dim, ops.PAGE_SIZE, self.n_heads // self.n_kv_heads)):
-            mods.append("attention_tc")         # prompts of one uncapped map with keys and values of 64 or 128
+            mods.append("attention_tc")         # prompts of one uncapped map with keys and values of 64 or 128 ...
+            if self.chunk == 0:
+                mods.append("attention_mma")    # ... and its single tokens over all keys
         return tuple(mods)
 
     def kv_spec(self):
@@ -338,7 +351,8 @@ class ScoreMapsAttention(Mixer):
         table = ctx.page_tables[cache.group_id]
         q = ops.maps_prep(qkv, bias, self.q_norm_w, self.k_norm_w, cos, sin, ctx, table, cache.k_pool, cache.v_pool,
                           self.n_heads, self.n_kv_heads, self.maps, self.head_dim, self.value_dim, self.rotary_dim,
-                          self.layout == "interleaved", self.eps, store_kv=cache.writable)
+                          self.layout == "interleaved", self.eps, store_kv=cache.writable,
+                          whole_norm=self.norm_over == "projection", temp_coef=self.temp_coef, temp_every=self.temp_every)
         two = self.maps == 2
         att = ops.maps_attention(q, cache.k_pool, cache.v_pool, table, ctx, self.maps, self.scale, softcap=self.softcap,
                                  chunk=self.chunk, lam=self.lam, norm_out=two, eps=self.eps,

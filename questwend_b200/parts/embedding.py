@@ -13,7 +13,9 @@ from .registry import register_embedding, register_head, register_stream_step
 
 class TokenEmbedding(Part):
     """params: vocab_size, hidden_size, name, scale (the rows are multiplied by it; default 1), norm (the tensor name of
-    an RMS norm's weight that the rows pass right after the gather; default none) with norm_eps."""
+    an RMS norm's weight that the rows pass right after the gather; default none) with norm_eps, positions (the tensor
+    name of a table of learned position vectors [max_positions, hidden_size]: row p is added, unscaled, to the embedding of
+    a token at position p; default none) with max_positions."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -23,24 +25,32 @@ class TokenEmbedding(Part):
         self.scale = float(spec.params.get("scale", 1.0))
         self.norm = None if spec.params.get("norm") is None else self.prefix + str(spec.params["norm"])
         self.norm_eps = float(spec.params.get("norm_eps", 0.0))
-        self.table = self.norm_w = None
+        self.positions = None if spec.params.get("positions") is None else self.prefix + str(spec.params["positions"])
+        self.max_positions = int(spec.params.get("max_positions", 0))
+        self.table = self.norm_w = self.pos_table = None
 
     def tensors(self):
         out = [TensorSpec(self.name, (self.vocab, self.hidden), MATRIX)]
+        if self.positions is not None:
+            out.append(TensorSpec(self.positions, (self.max_positions, self.hidden), MATRIX))
         if self.norm is not None:
             out.append(TensorSpec(self.norm, (self.hidden,), VECTOR, NORM_WEIGHT))
         return out
 
     def bind(self, weights):
         self.table = weights[self.name]
+        if self.positions is not None:
+            self.pos_table = weights[self.positions]
         if self.norm is not None:
             self.norm_w = weights[self.norm].to(torch.float32).contiguous()
 
     def kernel_modules(self):
         return ("elementwise",)
 
-    def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
-        h = ops.embed_gather(token_ids, self.table, scale=self.scale)
+    def forward(self, token_ids: torch.Tensor, positions: torch.Tensor | None = None) -> torch.Tensor:
+        if self.pos_table is not None and positions is None:
+            raise ValueError(f"embedding '{self.name}': learned positions need the tokens' positions")
+        h = ops.embed_gather(token_ids, self.table, scale=self.scale, pos_table=self.pos_table, positions=positions)
         return h if self.norm_w is None else ops.rmsnorm(h, self.norm_w, self.norm_eps, torch.float32)
 
 

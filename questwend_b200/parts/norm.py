@@ -5,26 +5,29 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from ..weights.manifest import NORM_WEIGHT, VECTOR, TensorSpec
+from ..weights.manifest import NORM_DELTA, NORM_WEIGHT, VECTOR, TensorSpec
 from .base import Norm, NormedSum, ScaledSum
 from .registry import register_norm
 
 
 class RMSNorm(Norm):
-    """params: dim, eps, name (default "weight"); tensor: <prefix><name> [dim]."""
+    """params: dim, eps, name (default "weight"), about_one (default False: the stored weight is the factor; True: it is
+    the factor's difference from 1); tensor: <prefix><name> [dim]."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         self.dim = int(spec.params["dim"])
         self.eps = float(spec.params["eps"])
         self.name = self.prefix + str(spec.params.get("name", "weight"))
+        self.about_one = bool(spec.params.get("about_one", False))
         self.weight = None
 
     def tensors(self):
-        return [TensorSpec(self.name, (self.dim,), VECTOR, NORM_WEIGHT)]
+        return [TensorSpec(self.name, (self.dim,), VECTOR, NORM_DELTA if self.about_one else NORM_WEIGHT)]
 
     def bind(self, weights):
-        self.weight = weights[self.name].to(torch.float32).contiguous()
+        w = weights[self.name].to(torch.float32)
+        self.weight = (w + 1.0 if self.about_one else w).contiguous()      # the sum in 32-bit, once
 
     def kernel_modules(self):
         return ("elementwise",)

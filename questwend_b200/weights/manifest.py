@@ -9,6 +9,7 @@ TABLE = "table"        # integer tables: held as int32
 
 NORMAL = "normal"            # random mode: N(0, 0.02)
 NORM_WEIGHT = "norm_weight"  # random mode: 1 + U(-0.1, 0.1)
+NORM_DELTA = "norm_delta"    # a norm weight stored as its difference from 1; random mode: U(-0.1, 0.1)
 
 
 @dataclass(frozen=True)

@@ -1,7 +1,8 @@
 """Random weights from a configuration and a seed.
 
 The reference has no such mode.  Matrices and the embedding are drawn from
-N(0, 0.02) and every norm weight from 1 + U(-0.1, 0.1).  Each tensor has its
+N(0, 0.02) and every norm weight from 1 + U(-0.1, 0.1) (one that is stored as its
+difference from 1: from U(-0.1, 0.1)).  Each tensor has its
 own generator, seeded by the seed and the tensor's place in the manifest, so
 the values do not depend on the order of generation; drawn on the CPU they are
 the same on every machine.
@@ -13,7 +14,7 @@ import os
 
 import torch
 
-from .manifest import MATRIX, NORM_WEIGHT, NORMAL, TABLE, TensorSpec
+from .manifest import MATRIX, NORM_DELTA, NORM_WEIGHT, NORMAL, TABLE, TensorSpec
 from .safetensors_io import write_safetensors
 
 INIT_STD = 0.02
@@ -29,10 +30,10 @@ def _draw(spec: TensorSpec, seed: int, index: int, device) -> torch.Tensor:
         t = torch.empty(spec.shape, dtype=torch.float32, device=device)
         t.normal_(0.0, INIT_STD, generator=gen)
         return t
-    if spec.init == NORM_WEIGHT:
+    if spec.init in (NORM_WEIGHT, NORM_DELTA):
         t = torch.empty(spec.shape, dtype=torch.float32, device=device)
         t.uniform_(-NORM_SPREAD, NORM_SPREAD, generator=gen)
-        return t.add_(1.0)
+        return t.add_(1.0) if spec.init == NORM_WEIGHT else t
     raise ValueError(f"tensor '{spec.name}': unknown init '{spec.init}'")
 
 
