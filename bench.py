@@ -129,6 +129,27 @@ def sagupel_sizes(width=2048, repeats=2, window=1024, vocab=32768):
             "postln_alpha": 1.5, "vocab": vocab, "width": width}
 
 
+def tufadra_sizes(width=2048, layers=6, vdim=128, vocab=32768, runs=1):
+    """A Tufadra configuration at sizes that resemble real layers: attention with 16 heads of 128 over 4 key/value heads
+    (values of ``vdim``), 64 ungated experts of 1,408 in 8 groups of which a token uses 6 from the best 3, a shared expert
+    of 2,816 and 4,096 positions.  ``runs`` 2: half as many layers of tensors, each run twice."""
+    mlp = {"kind": "moe", "expert": {"ff": 1408}, "shared": {"ff": 2816},
+           "router": {"experts": 64, "top": 6, "scale": 2.5, "groups": {"count": 8, "keep": 3}}}
+    layer = {"type": "attention", "mlp": mlp,
+             "mixer": {"dim": 128, "heads": width // 128, "kv_heads": width // 512, "vdim": vdim, "scale": 128 ** -0.5,
+                       "q_temp": {"coef": 0.1, "every": 1024}}}
+    own = layers // runs
+    return {"architecture": "Tufadra", "layers": [layer if i < own else {**layer, "weights_of": i % own} for i in range(layers)],
+            "max_positions": 4096, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+
+
+def movudra_experts_beside(width=2048, layers=6, vocab=32768):
+    """The closest model the library had for the feed-forward: Movudra's latent attention layers (16 heads of 128 + 64) with
+    its routed experts, 64 gated ones of 1,408 of which a token uses 6, at the same width, depth and vocabulary."""
+    latent = next(layer for layer in movudra_sizes(width)["layers"] if layer["type"] == "latent_attention")
+    return {"architecture": "Movudra", "layers": [latent] * layers, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+
+
 def qwen3_beside(width=2048, layers=6, vocab=32768):
     """The closest model the library had, at the same width, depth and vocabulary: Qwen3 layers with 16 heads of 128
     (8 key/value heads) and a gated feed-forward of 3 x width."""
@@ -386,8 +407,10 @@ def step_weight_bytes(engine, batch: int) -> int:
         if ffn is None:
             continue
         if hasattr(ffn, "experts"):
-            per_expert = (ffn.w_gate_up[0].numel() + ffn.w_down[0].numel()) * ffn.w_down.element_size()
+            per_expert = (ffn.w_up[0].numel() + ffn.w_down[0].numel()) * ffn.w_down.element_size()
             total += min(ffn.experts, batch * ffn.top) * per_expert + ffn.w_router.numel() * ffn.w_router.element_size()
+            if ffn.shared:
+                total += (ffn.w_shared_up.numel() + ffn.w_shared_down.numel()) * ffn.w_shared_up.element_size()
         else:
             total += _tensor_bytes(ffn, seen)
     return total + engine.model.head.weight.numel() * engine.model.head.weight.element_size()
@@ -824,6 +847,115 @@ def sagupel_kernels(torch, np, peaks) -> dict:
     return out
 
 
+def tufadra_kernels(torch, np, peaks) -> dict:
+    """The Tufadra design's kernels alone at the sizes of ``tufadra_sizes``, each beside the like kernel of a model the
+    library had, with the bytes or FLOPs it must move and the share of the measured peak that this comes to: the embedding
+    with its positions (beside the plain gather), the preparation of q and k with norms over whole projections (beside the
+    per-head norms), attention with values of 128 (Qwen3's kernels) and of 64 (beside Qwen3's), the router with groups
+    (beside Movudra's), and the experts with a shared one (beside Movudra's gated experts)."""
+    from questwend_b200.cache.manager import CacheManager
+    from questwend_b200.engine.engine import StepEntry, build_step_context
+    from questwend_b200.kernels import ops
+    from questwend_b200.parts.base import KVSpec
+    from questwend_b200.parts.linear import linear, linear_act
+    dev, bf = torch.device("cuda:0"), torch.bfloat16
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def timed(fn, reps=7):
+        times = []
+        for _ in range(reps + 3):
+            flush.zero_()                                         # L2 holds nothing of the last run
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            times.append(a.elapsed_time(b) * 1e3)
+        return statistics.median(times[3:])
+
+    def point(us, n_bytes=0, flops=0):
+        p = {"us": round(us, 1)}
+        if n_bytes:
+            p.update(gb_s=round(n_bytes / us / 1e3, 1), hbm_frac=round(n_bytes / (us * 1e-6) / hbm, 3))
+        if flops:
+            p.update(tflops=round(flops / us / 1e6, 1), tensor_frac=round(flops / (us * 1e-6) / tf, 3))
+        return p
+
+    out = {}
+    H, G, D = 16, 4, 2048
+    for label, n_new, B, prompt in (("prefill_2048", 2048, 1, 0), ("prefill_8192", 8192, 1, 0), ("decode_b8_at_4096", 1, 8, 4095),
+                                    ("decode_b8_at_32768", 1, 8, 32767)):
+        n_ctx, rows = prompt + n_new, B * n_new
+        for vdim in (128, 64):
+            cache = CacheManager([(KVSpec(G, 128, 0, value_dim=vdim), None, None)], B * n_ctx + 64 * B, B, n_ctx + 64, bf, dev)
+            slots = cache.open(B)
+            if prompt:
+                build_step_context(cache, [StepEntry(s, [0] * prompt, []) for s in slots], 10, dev)
+                for s in slots:
+                    cache.advance(s, prompt)
+            u = cache.unit_cache(0)
+            u.k_pool.normal_()
+            u.v_pool.normal_()
+            ctx = build_step_context(cache, [StepEntry(s, [0] * n_new, []) for s in slots], 10, dev)[0]
+            table = ctx.page_tables[u.group_id]
+            q = torch.randn(rows, H, 128, device=dev).to(bf)
+            run = lambda: ops.maps_attention(q, u.k_pool, u.v_pool, table, ctx, 1, 0.09)
+            full = n_new * (n_new + 1) // 2
+            work = {"flops": H * full * 2 * (128 + vdim)} if n_new > 1 else {"n_bytes": B * G * n_ctx * (128 + vdim) * 2}
+            out[f"attention_values_{vdim}_{label}"] = point(timed(run, reps=3), **work)
+            if vdim == 128:
+                for impl in (("tc", "mma") if n_new > 1 else ("auto",)):
+                    like = ((lambda: ops.attn_prefill(q, u.k_pool, u.v_pool, table, ctx.cu_seqlens, ctx.pos0, ctx.max_new, 0.09, impl=impl)) if n_new > 1
+                            else (lambda: ops.attn_decode(q, u.k_pool, u.v_pool, table, ctx.seq_len, 0.09, ctx.max_len)))
+                    out[f"qwen3_attention_{impl}_{label}"] = point(timed(like, reps=3), **work)
+            n_cols = (H + G) * 128 + G * vdim
+            qkv, w = torch.randn(rows, n_cols, device=dev), torch.ones(H * 128, device=dev)
+            out[f"prep_whole_norm_values_{vdim}_{label}"] = point(
+                timed(lambda: ops.maps_prep(qkv, None, w, w[:G * 128], None, None, ctx, table, u.k_pool, u.v_pool, H, G, 1, 128, vdim, 0, False, 1e-5,
+                                            whole_norm=True, temp_coef=0.1, temp_every=1024)), rows * n_cols * 6)
+            if vdim == 128:
+                cs = torch.ones(rows, 64, device=dev)
+                out[f"punolix_maps_prep_{label}"] = point(
+                    timed(lambda: ops.maps_prep(qkv, None, w[:128], w[:128], cs, cs, ctx, table, u.k_pool, u.v_pool, H, G, 1, 128, 128, 128, False, 1e-5)), rows * n_cols * 6)
+                out[f"qwen3_qk_norm_rope_store_{label}"] = point(
+                    timed(lambda: ops.qk_norm_rope_store(qkv, w[:128], w[:128], cs, cs, ctx.tok_seq, ctx.tok_pos, table, u.k_pool, u.v_pool, H, G, 128, 128, 1e-5)), rows * n_cols * 6)
+            del cache, u
+            torch.cuda.empty_cache()
+    E, top, F, Fs = 64, 6, 1408, 2816
+    w_up, w_gu = torch.randn(E, F, D, device=dev).to(bf) * 0.02, torch.randn(E, 2 * F, D, device=dev).to(bf) * 0.02
+    w_down = torch.randn(E, D, F, device=dev).to(bf) * 0.02
+    s_up, s_down = torch.randn(Fs, D, device=dev).to(bf) * 0.02, torch.randn(D, Fs, device=dev).to(bf) * 0.02
+    table, ptable = torch.randn(32768, D, device=dev).to(bf), torch.randn(4096, D, device=dev).to(bf)
+    for T in (2048, 16, 8, 1):
+        x = torch.randn(T, D, device=dev).to(bf)
+        ids = torch.randint(0, 32768, (T,), device=dev).int()
+        pos = torch.arange(T, device=dev).int()
+        out[f"embedding_with_positions_{T}"] = point(timed(lambda: ops.embed_gather(ids, table, pos_table=ptable, positions=pos)), T * D * 8)
+        out[f"embedding_{T}"] = point(timed(lambda: ops.embed_gather(ids, table)), T * D * 6)
+        z = torch.randn(T, 72, device=dev)
+        z64 = z[:, :E].contiguous()
+        corr = torch.randn(E, device=dev) * 0.1
+        route = lambda: ops.moe_route(z, top, True, experts=E, scores="sigmoid", correction=corr, groups=8, keep=3, sum_eps=1e-20, weight_scale=2.5, gate=True)
+        out[f"router_groups_{T}"] = point(timed(route), T * (E * 4 + top * 8))
+        out[f"router_movudra_{T}"] = point(timed(lambda: ops.moe_route(z64, top)), T * (E * 4 + top * 8))
+        chosen, weight, gate = route()
+        used = len(torch.unique(chosen))
+        if T > 16:
+            for name, up, act, k in (("experts_grouped", w_up, "gelu", 1), ("experts_grouped_movudra", w_gu, "gated_silu", 2)):
+                out[f"{name}_{T}"] = point(timed(lambda: ops.moe_experts_grouped(x, up, w_down, chosen, weight, act)), flops=T * top * 2 * D * F * (k + 1))
+            shared = linear(linear_act(x, s_up, None, "gelu", bf), s_down)
+            out[f"shared_expert_{T}"] = point(timed(lambda: linear(linear_act(x, s_up, None, "gelu", bf), s_down)), flops=T * 4 * D * Fs)
+            out[f"experts_grouped_with_shared_sum_{T}"] = point(timed(lambda: ops.moe_experts_grouped(x, w_up, w_down, chosen, weight, "gelu", shared=shared, gate=gate)),
+                                                                flops=T * top * 4 * D * F)
+            out[f"experts_sort_{T}"] = point(timed(lambda: ops.moe_sort(chosen, E)))
+        else:
+            out[f"experts_with_shared_{T}"] = point(timed(lambda: ops.moe_experts(x, w_up, w_down, chosen, weight, "gelu", s_up, s_down, gate)), (used * 2 * D * F + 2 * D * Fs) * 2)
+            out[f"experts_{T}"] = point(timed(lambda: ops.moe_experts(x, w_up, w_down, chosen, weight, "gelu")), used * 2 * D * F * 2)
+            out[f"experts_movudra_{T}"] = point(timed(lambda: ops.moe_experts(x, w_gu, w_down, chosen, weight)), used * 3 * D * F * 2)
+    return out
+
+
 def reference_arm(args) -> int:
     """kishida/questwend itself, unmodified, through its own public classes (baseline/ref_bench.cpp), on the same sizes.
     Nothing of questwend_b200 is imported on this path."""
@@ -916,9 +1048,9 @@ def main() -> int:
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--model", default="8b", choices=sorted(MODELS) + ["movudra", "roritar", "roritar-kernels", "punolix", "punolix-kernels", "sagupel", "sagupel-kernels"],
-                    help="8b: the benchmark; 0.6b, 32b: its other workloads alone; movudra, roritar, punolix, sagupel: that design at real layer "
-                         "sizes beside Qwen3 layers of the same width and depth; roritar-kernels, punolix-kernels, sagupel-kernels: its own kernels alone, each "
+    ap.add_argument("--model", default="8b", choices=sorted(MODELS) + ["movudra", "roritar", "roritar-kernels", "punolix", "punolix-kernels", "sagupel", "sagupel-kernels", "tufadra", "tufadra-kernels"],
+                    help="8b: the benchmark; 0.6b, 32b: its other workloads alone; movudra, roritar, punolix, sagupel, tufadra: that design at real layer "
+                         "sizes beside Qwen3 layers of the same width and depth; roritar-kernels, punolix-kernels, sagupel-kernels, tufadra-kernels: its own kernels alone, each "
                          "beside the like kernel of a model the library had")
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the model has (named in config)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
@@ -980,6 +1112,18 @@ def main() -> int:
         print(json.dumps({"metric": "Sagupel's kernels alone, each beside the like kernel of an earlier model", "n_gpus": 1,
                           "dtype": "bf16", "data": "synthetic: random tensors of the sizes of sagupel_sizes; L2 flushed between runs",
                           "peaks": peak_source, "points": sagupel_kernels(torch, np, peaks)}))
+        return 0
+    if args.model == "tufadra":
+        designs = (("tufadra", tufadra_sizes()), ("tufadra_values_64_two_runs", tufadra_sizes(vdim=64, runs=2)), ("tufadra_width_1024", tufadra_sizes(width=1024)),
+                   ("movudra_experts_same_size", movudra_experts_beside()), ("qwen3_same_size", qwen3_beside()))
+        print(json.dumps({"metric": "Tufadra at real layer sizes beside Movudra's routed experts and Qwen3 layers of equal width and depth", "n_gpus": 1,
+                          "dtype": "bf16", "data": "synthetic: seeded random weights and uniform random token ids",
+                          "peaks": peak_source, "points": movudra_workload(torch, np, peaks, steps, warmup, designs)}))
+        return 0
+    if args.model == "tufadra-kernels":
+        print(json.dumps({"metric": "Tufadra's kernels alone, each beside the like kernel of an earlier model", "n_gpus": 1,
+                          "dtype": "bf16", "data": "synthetic: random tensors of the sizes of tufadra_sizes; L2 flushed between runs",
+                          "peaks": peak_source, "points": tufadra_kernels(torch, np, peaks)}))
         return 0
     if args.model != "8b":                      # one of the other workloads alone, as a line of its own
         points = small_model_workload(torch, np, peaks) if args.model == "0.6b" else large_model_workload(torch, np, peaks)

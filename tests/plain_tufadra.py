@@ -35,7 +35,8 @@ _erf = np.frompyfunc(math.erf, 1, 1)
 
 def gelu_exact(z):
     """z times the normal distribution's function at z."""
-    return 0.5 * z * (1.0 + _erf(np.asarray(z) / math.sqrt(2.0)).astype(np.float64))
+    z = np.asarray(z, dtype=np.float64)
+    return 0.5 * z * (1.0 + _erf(z / math.sqrt(2.0)).astype(np.float64))
 
 
 def unit_rms(x, eps):
