@@ -1,4 +1,5 @@
-// Tensor-core attention over the paged bfloat16 cache, for head sizes 64 and 128.
+// Tensor-core attention over the paged bfloat16 cache, for head sizes 64 and 128; single tokens also for other key and
+// value sizes up to 128 (multiples of 8, equal or not), which are filled up with zeros to 64 or 128 in shared memory.
 //
 // Same contract as attention.cu (causal, grouped heads, optional window, pages of 64 keys);
 // those kernels stay the path for float32 and for other head sizes.  Here the scores
@@ -65,6 +66,29 @@ __device__ __forceinline__ void load_tile(bf16* tile, const bf16* src, int n_val
     }
 }
 
+// The same for rows of n values (a multiple of 8, at most HD) whose tile rows are HD values apart.  What lies beyond n in a
+// tile row is written by clear_tail, once: no copy touches it again.
+template <int HD>
+__device__ __forceinline__ void load_tile_part(bf16* tile, const bf16* src, int n, int n_valid, int tid, int nthreads) {
+    constexpr int CPR = HD / 8;
+    for (int i = tid; i < AM_TILE * CPR; i += nthreads) {
+        const int row = i / CPR, c = i % CPR;
+        if (8 * c >= n) continue;
+        bf16* dst = tile + row * HD + ((c ^ (row & 7)) << 3);
+        if (row < n_valid) cp_async16(dst, src + row * n + (c << 3));
+        else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+    }
+}
+template <int HD>
+__device__ __forceinline__ void clear_tail(bf16* tile, int n, int tid, int nthreads) {
+    constexpr int CPR = HD / 8;
+    if (n >= HD) return;
+    for (int i = tid; i < AM_TILE * CPR; i += nthreads) {
+        const int row = i / CPR, c = i % CPR;
+        if (8 * c >= n) *reinterpret_cast<uint4*>(tile + row * HD + ((c ^ (row & 7)) << 3)) = make_uint4(0u, 0u, 0u, 0u);
+    }
+}
+
 // One warp, 16 rows, one tile of 64 keys: S = Q K^T, mask, online softmax, O += P V, in two halves so that a caller
 // can wait for K and for V separately and start the next tile's copies in between.
 //   qf     Q fragments of the warp's 16 rows: [HD/16][4]
@@ -73,11 +97,11 @@ __device__ __forceinline__ void load_tile(bf16* tile, const bf16* src, int n_val
 //   m, l   running maximum and (this thread's share of the) sum for rows g and g + 8;  o: [HD/8][4]
 //   KEYS, key_off: the warp takes the KEYS keys (a multiple of 16) of the tile that start at key_off
 //   s, base: the masked scores and the rows' new maxima (scaled), handed from the first half to the second
-template <int HD, int KEYS>
+template <int HD, int KEYS, int VD = HD>
 __device__ __forceinline__ void tile_scores(const uint32_t (*qf)[4], const bf16* Kt, int key0, const int* row_pos, int len,
                                             int window, float sl2, float* m, float* l, float (*o)[4], int lane, int key_off,
                                             float (*s)[4], float* base) {
-    constexpr int KS = HD / 16, NT = KEYS / 8, DT = HD / 8;
+    constexpr int KS = HD / 16, NT = KEYS / 8, DT = VD / 8;
     const int t = lane & 3;
 #pragma unroll
     for (int j = 0; j < NT; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
@@ -165,17 +189,18 @@ __device__ __forceinline__ void tile_step(const uint32_t (*qf)[4], const bf16* K
     tile_pv<HD, AM_TILE>(Vt, s, base, sl2, l, o, lane, 0);
 }
 
-// Q fragments of rows (g, g + 8) of a warp; q_lo / q_hi point at the rows' hd values (or null).
+// Q fragments of rows (g, g + 8) of a warp; q_lo / q_hi point at the rows' n values (a multiple of 8; or null).
 template <int HD>
-__device__ __forceinline__ void load_q_frags(uint32_t (*qf)[4], const bf16* q_lo, const bf16* q_hi, int lane) {
+__device__ __forceinline__ void load_q_frags(uint32_t (*qf)[4], const bf16* q_lo, const bf16* q_hi, int lane, int n = HD) {
     const int t = lane & 3;
 #pragma unroll
     for (int ks = 0; ks < HD / 16; ++ks) {
         const int d = 16 * ks + 2 * t;
-        qf[ks][0] = q_lo ? *reinterpret_cast<const uint32_t*>(q_lo + d) : 0u;
-        qf[ks][1] = q_hi ? *reinterpret_cast<const uint32_t*>(q_hi + d) : 0u;
-        qf[ks][2] = q_lo ? *reinterpret_cast<const uint32_t*>(q_lo + d + 8) : 0u;
-        qf[ks][3] = q_hi ? *reinterpret_cast<const uint32_t*>(q_hi + d + 8) : 0u;
+        const bool a = 16 * ks < n, b = 16 * ks + 8 < n;
+        qf[ks][0] = q_lo && a ? *reinterpret_cast<const uint32_t*>(q_lo + d) : 0u;
+        qf[ks][1] = q_hi && a ? *reinterpret_cast<const uint32_t*>(q_hi + d) : 0u;
+        qf[ks][2] = q_lo && b ? *reinterpret_cast<const uint32_t*>(q_lo + d + 8) : 0u;
+        qf[ks][3] = q_hi && b ? *reinterpret_cast<const uint32_t*>(q_hi + d + 8) : 0u;
     }
 }
 
@@ -393,13 +418,16 @@ __device__ __forceinline__ void fused_new_row(const FusedQKV& f, const float* sr
     }
 }
 
-template <int HD, bool FUSED, bool K_TWO>
+// HD, VD: key and value sizes, with PART filled up from hd_given and vd_given to 64 or 128 (only not FUSED).
+template <int HD, int VD, bool FUSED, bool K_TWO, bool PART>
 __global__ void __launch_bounds__(32)
 attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, const bf16* v_pool,
                        const int* __restrict__ page_table, const int* __restrict__ seq_len, float* __restrict__ part_acc,
                        float* __restrict__ part_m, float* __restrict__ part_l, bf16* __restrict__ out, int Hq, int Hkv,
                        int table_width, float scale, int window, int runs_target, int run_pages_max, int max_runs, int Gc,
-                       int chunks) {
+                       int chunks, int hd_given, int vd_given) {
+    static_assert(!FUSED || (HD == VD && !PART), "the fused form takes one size of 64 or 128");
+    const int hd = PART ? hd_given : HD, vd = PART ? vd_given : VD;
     constexpr bool k_two = K_TWO;
     // Launched with programmatic stream serialization, the block may start while the kernel before it still runs.
     // FUSED, that kernel is the q/k/v projection, and what the block needs first does not come from it: the sequences'
@@ -434,20 +462,31 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
     // k_two (the host gives the block a third tile when all blocks still find room on the SMs): K has two buffers, so
     // that the next page's K is asked for a page ahead - the second page's with the first, before anything else - and
     // only V waits for its buffer.  The arithmetic is the same either way.
-    bf16* k_tiles[2] = {my_tiles, k_two ? my_tiles + 2 * AM_TILE * HD : my_tiles};
+    bf16* k_tiles[2] = {my_tiles, k_two ? my_tiles + AM_TILE * (HD + VD) : my_tiles};
     bf16* v_tile = my_tiles + AM_TILE * HD;
+    auto load_k = [&](bf16* tile, const bf16* src, int n_valid) {
+        if (PART) load_tile_part<HD>(tile, src, hd, n_valid, lane, 32); else load_tile<HD>(tile, src, n_valid, lane, 32);
+    };
+    auto load_v = [&](const bf16* src, int n_valid) {
+        if (PART) load_tile_part<VD>(v_tile, src, vd, n_valid, lane, 32); else load_tile<VD>(v_tile, src, n_valid, lane, 32);
+    };
+    if (PART) {
+        clear_tail<HD>(k_tiles[0], hd, lane, 32);
+        if (k_two) clear_tail<HD>(k_tiles[1], hd, lane, 32);
+        clear_tail<VD>(v_tile, vd, lane, 32);
+    }
     int base_tok = max(tok_begin, (k_lo / AM_TILE) * AM_TILE);                 // pages wholly before the window are skipped
     if (base_tok < tok_end) {
-        const size_t src = ((size_t)pages[base_tok / AM_TILE] * Hkv + kvh) * AM_TILE * HD;
+        const size_t src = ((size_t)pages[base_tok / AM_TILE] * Hkv + kvh) * AM_TILE;
         const int n_valid = min(AM_TILE, len - base_tok);
-        load_tile<HD>(k_tiles[0], k_pool + src, n_valid, lane, 32);
+        load_k(k_tiles[0], k_pool + src * hd, n_valid);
         cp_async_commit();
-        load_tile<HD>(v_tile, v_pool + src, n_valid, lane, 32);
+        load_v(v_pool + src * vd, n_valid);
         cp_async_commit();
         if (k_two && base_tok + AM_TILE < tok_end) {
             const int next_tok = base_tok + AM_TILE;
-            const size_t src1 = ((size_t)pages[next_tok / AM_TILE] * Hkv + kvh) * AM_TILE * HD;
-            load_tile<HD>(k_tiles[1], k_pool + src1, min(AM_TILE, len - next_tok), lane, 32);
+            const size_t src1 = ((size_t)pages[next_tok / AM_TILE] * Hkv + kvh) * AM_TILE;
+            load_k(k_tiles[1], k_pool + src1 * hd, min(AM_TILE, len - next_tok));
             cp_async_commit();
         }
     }
@@ -464,11 +503,11 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
             const int r = g + 8 * h, head_in = chunk * Gc + r;
             const bool ok = r < Gc && head_in < G;
             row_pos[h] = ok ? len - 1 : -1;
-            qrow[h] = ok && !FUSED ? q + ((size_t)b * Hq + kvh * G + head_in) * HD : nullptr;
+            qrow[h] = ok && !FUSED ? q + ((size_t)b * Hq + kvh * G + head_in) * hd : nullptr;
             frow[h] = ok && FUSED ? fused.qkv + ((size_t)b * n_all + kvh * G + head_in) * HD : nullptr;
         }
-        if (FUSED) fused_q_frags<HD>(qf, fused, frow[0], frow[1], b, lane);
-        else load_q_frags<HD>(qf, qrow[0], qrow[1], lane);
+        if constexpr (FUSED) fused_q_frags<HD>(qf, fused, frow[0], frow[1], b, lane);
+        else load_q_frags<HD>(qf, qrow[0], qrow[1], lane, hd);
     }
     // FUSED: the new token's key and value, if its place lies in this run: into the cache (one block per key/value head
     // writes) and, below, into the shared tiles of its page
@@ -495,9 +534,9 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
 #pragma unroll
         for (int e = 0; e < HD / 32; e += 2) *reinterpret_cast<uint32_t*>(dst + e) = pack_bf16(y[e], y[e + 1]);
     };
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[HD / 8][4];
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[VD / 8][4];
 #pragma unroll
-    for (int d = 0; d < HD / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+    for (int d = 0; d < VD / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
     if constexpr (!K_TWO) {
     for (; base_tok < tok_end; base_tok += AM_TILE) {
         bf16* k_tile = k_tiles[0];
@@ -506,7 +545,7 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
         size_t src = 0;
         int n_valid = 0;
         if (more) {
-            src = ((size_t)pages[next_tok / AM_TILE] * Hkv + kvh) * AM_TILE * HD;
+            src = ((size_t)pages[next_tok / AM_TILE] * Hkv + kvh) * AM_TILE;
             n_valid = min(AM_TILE, len - next_tok);
         }
         float s[AM_TILE / 8][4], sbase[2];
@@ -514,10 +553,10 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
         __syncwarp();
         const bool new_here = has_new && new_pos >= base_tok && new_pos < base_tok + AM_TILE;
         if (new_here) { patch(k_tile, new_k); __syncwarp(); }
-        tile_scores<HD, AM_TILE>(qf, k_tile, base_tok, row_pos, len, window, sl2, m, l, o, lane, 0, s, sbase);
+        tile_scores<HD, AM_TILE, VD>(qf, k_tile, base_tok, row_pos, len, window, sl2, m, l, o, lane, 0, s, sbase);
         __syncwarp();                                                           // every lane is done reading K
         if (more) {
-            load_tile<HD>(k_tile, k_pool + src, n_valid, lane, 32);
+            load_k(k_tile, k_pool + src * hd, n_valid);
             cp_async_commit();
             cp_async_wait<1>();                                                 // all but the copy just started: this page's V
         } else {
@@ -525,10 +564,10 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
         }
         __syncwarp();
         if (new_here) { patch(v_tile, new_v); __syncwarp(); }
-        tile_pv<HD, AM_TILE>(v_tile, s, sbase, sl2, l, o, lane, 0);
+        tile_pv<VD, AM_TILE>(v_tile, s, sbase, sl2, l, o, lane, 0);
         __syncwarp();                                                           // every lane is done reading V
         if (more) {
-            load_tile<HD>(v_tile, v_pool + src, n_valid, lane, 32);
+            load_v(v_pool + src * vd, n_valid);
             cp_async_commit();
         }
     }
@@ -540,7 +579,7 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
         size_t src = 0;
         int n_valid = 0;
         if (more) {
-            src = ((size_t)pages[next_tok / AM_TILE] * Hkv + kvh) * AM_TILE * HD;
+            src = ((size_t)pages[next_tok / AM_TILE] * Hkv + kvh) * AM_TILE;
             n_valid = min(AM_TILE, len - next_tok);
         }
         float s[AM_TILE / 8][4], sbase[2];
@@ -549,29 +588,29 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
         __syncwarp();
         const bool new_here = has_new && new_pos >= base_tok && new_pos < base_tok + AM_TILE;
         if (new_here) { patch(k_tile, new_k); __syncwarp(); }
-        tile_scores<HD, AM_TILE>(qf, k_tile, base_tok, row_pos, len, window, sl2, m, l, o, lane, 0, s, sbase);
+        tile_scores<HD, AM_TILE, VD>(qf, k_tile, base_tok, row_pos, len, window, sl2, m, l, o, lane, 0, s, sbase);
         __syncwarp();                                                           // every lane is done reading K
         bool started = false;                                                   // a copy of K started just now
         if (k_two) {
             if (more2) {                                                        // the page after the next into this page's buffer
                 const int tok2 = next_tok + AM_TILE;
-                const size_t src2 = ((size_t)pages[tok2 / AM_TILE] * Hkv + kvh) * AM_TILE * HD;
-                load_tile<HD>(k_tile, k_pool + src2, min(AM_TILE, len - tok2), lane, 32);
+                const size_t src2 = ((size_t)pages[tok2 / AM_TILE] * Hkv + kvh) * AM_TILE;
+                load_k(k_tile, k_pool + src2 * hd, min(AM_TILE, len - tok2));
                 cp_async_commit();
                 started = true;
             }
         } else if (more) {
-            load_tile<HD>(k_tile, k_pool + src, n_valid, lane, 32);
+            load_k(k_tile, k_pool + src * hd, n_valid);
             cp_async_commit();
             started = true;
         }
         if (started) cp_async_wait<1>(); else cp_async_wait<0>();               // all but the copy just started: this page's V
         __syncwarp();
         if (new_here) { patch(v_tile, new_v); __syncwarp(); }
-        tile_pv<HD, AM_TILE>(v_tile, s, sbase, sl2, l, o, lane, 0);
+        tile_pv<VD, AM_TILE>(v_tile, s, sbase, sl2, l, o, lane, 0);
         __syncwarp();                                                           // every lane is done reading V
         if (more) {
-            load_tile<HD>(v_tile, v_pool + src, n_valid, lane, 32);
+            load_v(v_pool + src * vd, n_valid);
             cp_async_commit();
         }
     }
@@ -590,15 +629,15 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
         const int head = kvh * G + head_in;
         if (single) {
             const float inv = 1.f / l[h];
-            bf16* dst = out + ((size_t)b * Hq + head) * HD;
+            bf16* dst = out + ((size_t)b * Hq + head) * vd;
 #pragma unroll
-            for (int d = 0; d < HD / 8; ++d)
-                *reinterpret_cast<uint32_t*>(dst + 8 * d + 2 * t) = pack_bf16(o[d][2 * h] * inv, o[d][2 * h + 1] * inv);
+            for (int d = 0; d < VD / 8; ++d)
+                if (!PART || 8 * d < vd) *reinterpret_cast<uint32_t*>(dst + 8 * d + 2 * t) = pack_bf16(o[d][2 * h] * inv, o[d][2 * h + 1] * inv);
         } else {
             const size_t at = ((size_t)b * Hq + head) * max_runs + run;
-            float* dst = part_acc + at * HD;
+            float* dst = part_acc + at * VD;                // (filled-up columns hold zeros)
 #pragma unroll
-            for (int d = 0; d < HD / 8; ++d)
+            for (int d = 0; d < VD / 8; ++d)
                 *reinterpret_cast<float2*>(dst + 8 * d + 2 * t) = make_float2(o[d][2 * h], o[d][2 * h + 1]);
             if (t == 0) { part_m[at] = m[h] * scale; part_l[at] = l[h]; }   // the combine kernel works with scaled scores
         }
@@ -611,10 +650,10 @@ attn_mma_decode_kernel(const FusedQKV fused, const bf16* q, const bf16* k_pool, 
 // first is used.  (One block of 128 threads per (head, sequence), a column a thread, took 3.7 us at 8 sequences and 8.0
 // at 64, where this takes 3.6 and 4.5; a decode step of 8 sequences got 1.3 % faster, one of 64 2 %.)
 #define AM_COMBINE_THREADS 128
-template <int VEC>                     // columns per lane: hd = 32 * VEC
+template <int VEC>                     // columns per lane: partial results of hd = 32 * VEC values, of which the first vd are written
 __global__ void __launch_bounds__(AM_COMBINE_THREADS)
 attn_mma_combine_warp_kernel(const float* part_acc, const float* part_m, const float* part_l, const int* __restrict__ seq_len,
-                             bf16* __restrict__ out, int Hq, int window, int runs_target, int run_pages_max, int max_runs) {
+                             bf16* __restrict__ out, int Hq, int window, int runs_target, int run_pages_max, int max_runs, int vd) {
     pdl_launch_dependents();            // the trigger first: the kernel after this one may start while attention still runs
     pdl_wait();
     constexpr int hd = 32 * VEC;
@@ -674,7 +713,8 @@ attn_mma_combine_warp_kernel(const float* part_acc, const float* part_m, const f
             }
         }
     }
-    bf16* dst = out + ((size_t)b * Hq + h) * hd + lane * VEC;
+    if (lane * VEC >= vd) return;       // vd is a multiple of 8
+    bf16* dst = out + ((size_t)b * Hq + h) * vd + lane * VEC;
 #pragma unroll
     for (int v = 0; v < VEC; v += 2) *reinterpret_cast<uint32_t*>(dst + v) = pack_bf16(a[v] / L, a[v + 1] / L);
 }
@@ -725,9 +765,9 @@ static int am_sm_count() {
     return n_sm;
 }
 
-template <int HD, bool FUSED>
+template <int HD, int VD, bool FUSED, bool PART>
 static int launch_decode(const FusedQKV& fused, const void* q, const void* k_pool, const void* v_pool, const int* page_table,
-                         const int* seq_len, float* scratch, void* out, int B, int Hq, int Hkv, int table_width, float scale,
+                         const int* seq_len, float* scratch, void* out, int B, int Hq, int Hkv, int hd, int vd, int table_width, float scale,
                          int window, int runs_target, int run_pages_max, int max_runs, cudaStream_t stream) {
     const int G = Hq / Hkv, Gc = group_chunk(G), chunks = (G + Gc - 1) / Gc;
     // A third tile (two for K) while every block of the grid still finds room: 4 blocks of 48 KB an SM.  Decode steps at
@@ -739,9 +779,9 @@ static int launch_decode(const FusedQKV& fused, const void* q, const void* k_poo
     // QWB200_ATTN_K2=0 switches it off, for measurements.
     static const bool k_two_allowed = [] { const char* e = getenv("QWB200_ATTN_K2"); return !(e && e[0] == '0'); }();
     const bool k_two = k_two_allowed && (long long)Hkv * chunks * B * max_runs <= 4LL * am_sm_count();
-    const size_t smem = (size_t)(k_two ? 3 : 2) * AM_TILE * HD * sizeof(bf16);
+    const size_t smem = (size_t)AM_TILE * ((k_two ? 2 : 1) * HD + VD) * sizeof(bf16);
     float* part_acc = scratch;
-    float* part_m = scratch + (size_t)B * Hq * max_runs * HD;
+    float* part_m = scratch + (size_t)B * Hq * max_runs * VD;
     float* part_l = part_m + (size_t)B * Hq * max_runs;
     dim3 grid(Hkv * chunks, B, max_runs);
     // early: see the kernel's first lines
@@ -750,15 +790,15 @@ static int launch_decode(const FusedQKV& fused, const void* q, const void* k_poo
         if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "attn_mma_decode: %s", cudaGetErrorString(e));
         qwb_launch_early(kernel, grid, 32, smem, stream, fused, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, page_table, seq_len,
                          part_acc, part_m, part_l, (bf16*)out, Hq, Hkv, table_width, scale, window, runs_target, run_pages_max, max_runs,
-                         Gc, chunks);
+                         Gc, chunks, hd, vd);
         return 0;
     };
-    if (int rc = k_two ? go(attn_mma_decode_kernel<HD, FUSED, true>) : go(attn_mma_decode_kernel<HD, FUSED, false>)) return rc;
+    if (int rc = k_two ? go(attn_mma_decode_kernel<HD, VD, FUSED, true, PART>) : go(attn_mma_decode_kernel<HD, VD, FUSED, false, PART>)) return rc;
     if (int rc = qwb_check_launch("attn_mma_decode")) return rc;
     if (max_runs > 1) {
         // (launched early with more sequences, even with its trigger after its wait, a step of 8 got 1 % slower)
-        qwb_launch_link(B, QWB_LINK_ROWS_MERGE, attn_mma_combine_warp_kernel<HD / 32>, dim3((Hq + AM_COMBINE_THREADS / 32 - 1) / (AM_COMBINE_THREADS / 32), B),
-                        AM_COMBINE_THREADS, 0, stream, part_acc, part_m, part_l, seq_len, (bf16*)out, Hq, window, runs_target, run_pages_max, max_runs);
+        qwb_launch_link(B, QWB_LINK_ROWS_MERGE, attn_mma_combine_warp_kernel<VD / 32>, dim3((Hq + AM_COMBINE_THREADS / 32 - 1) / (AM_COMBINE_THREADS / 32), B),
+                        AM_COMBINE_THREADS, 0, stream, part_acc, part_m, part_l, seq_len, (bf16*)out, Hq, window, runs_target, run_pages_max, max_runs, vd);
         return qwb_check_launch("attn_mma_combine");
     }
     return 0;
@@ -771,9 +811,11 @@ extern "C" int qwb_attn_mma_decode_runs(int max_len, int runs_target, int run_pa
     return max_runs_for(max_len, runs_target, run_pages_max);
 }
 
-static int check_decode(int B, int Hq, int Hkv, int hd, int page_size, int runs_target, int run_pages_max, int max_len,
+static int check_decode(int B, int Hq, int Hkv, int hd, int vd, int page_size, int runs_target, int run_pages_max, int max_len,
                         const float* scratch, int* max_runs) {
-    if (int rc = check_sizes("attn_mma_decode", Hq, Hkv, hd, page_size, B)) return rc;
+    if (hd <= 0 || hd > 128 || hd % 8 || vd <= 0 || vd > 128 || vd % 8)
+        return qwb_fail(QWB_ERR_ARG, "attn_mma_decode: key size %d or value size %d is not a multiple of 8 up to 128", hd, vd);
+    if (int rc = check_sizes("attn_mma_decode", Hq, Hkv, 64, page_size, B)) return rc;
     if (runs_target <= 0 || run_pages_max <= 0 || max_len <= 0)
         return qwb_fail(QWB_ERR_ARG, "attn_mma_decode: %d runs of up to %d pages for up to %d keys", runs_target, run_pages_max, max_len);
     *max_runs = max_runs_for(max_len, runs_target, run_pages_max);
@@ -783,24 +825,36 @@ static int check_decode(int B, int Hq, int Hkv, int hd, int page_size, int runs_
     return 0;
 }
 
-// bfloat16 only.  Arguments as qwb_attn_decode, but for how the keys are cut into runs: a sequence of p pages is cut into
-// runs of clamp(ceil(p / runs_target), 1, run_pages_max) pages (runs_target 1 gives runs of exactly run_pages_max pages);
-// max_len bounds every entry of seq_len.  scratch: B * Hq * runs(max_len) * (hd + 2) floats, unused with a single run.
+// bfloat16 only.  Arguments as qwb_attn_decode, but for the values' own size vd (out [B, Hq * vd]) and for how the keys are
+// cut into runs: a sequence of p pages is cut into runs of clamp(ceil(p / runs_target), 1, run_pages_max) pages
+// (runs_target 1 gives runs of exactly run_pages_max pages); max_len bounds every entry of seq_len.  scratch:
+// B * Hq * runs(max_len) * (vd filled up to 64 or 128, + 2) floats, unused with a single run.
 extern "C" int qwb_attn_mma_decode(const void* q, const void* k_pool, const void* v_pool, const int* page_table,
-                                   const int* seq_len, float* scratch, void* out, int B, int Hq, int Hkv, int hd, int page_size,
+                                   const int* seq_len, float* scratch, void* out, int B, int Hq, int Hkv, int hd, int vd, int page_size,
                                    int table_width, float scale, int window, int runs_target, int run_pages_max, int max_len,
                                    cudaStream_t stream) {
     if (B <= 0) return 0;
     int max_runs = 0;
-    if (int rc = check_decode(B, Hq, Hkv, hd, page_size, runs_target, run_pages_max, max_len, scratch, &max_runs)) return rc;
+    if (int rc = check_decode(B, Hq, Hkv, hd, vd, page_size, runs_target, run_pages_max, max_len, scratch, &max_runs)) return rc;
     FusedQKV none = {};
-    if (hd == 64) return launch_decode<64, false>(none, q, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, table_width, scale, window, runs_target, run_pages_max, max_runs, stream);
-    return launch_decode<128, false>(none, q, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, table_width, scale, window, runs_target, run_pages_max, max_runs, stream);
+#define QWB_AM_DECODE(HD, VD, PART)                                                                                              \
+    return launch_decode<HD, VD, false, PART>(none, q, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, hd, vd,    \
+                                              table_width, scale, window, runs_target, run_pages_max, max_runs, stream)
+    if (hd == vd && hd == 64) QWB_AM_DECODE(64, 64, false);
+    if (hd == vd && hd == 128) QWB_AM_DECODE(128, 128, false);
+    if (hd <= 64) {
+        if (vd <= 64) QWB_AM_DECODE(64, 64, true);
+        QWB_AM_DECODE(64, 128, true);
+    }
+    if (vd <= 64) QWB_AM_DECODE(128, 64, true);
+    QWB_AM_DECODE(128, 128, true);
+#undef QWB_AM_DECODE
 }
 
-// The same with the step's q, k and v taken from the q/k/v projection's 32-bit output qkv [B, (Hq + 2 Hkv) * hd]: per-head
-// norm of q and k (weights [hd], or null), rotation of all hd values by cos/sin [B, hd / 2] (or null), and, with store_kv,
-// the new key and value written into the cache at each sequence's position seq_len - 1, all inside the attention kernel.
+// The same with the step's q, k and v taken from the q/k/v projection's 32-bit output qkv [B, (Hq + 2 Hkv) * hd] (values of
+// the keys' size, 64 or 128): per-head norm of q and k (weights [hd], or null), rotation of all hd values by cos/sin
+// [B, hd / 2] (or null), and, with store_kv, the new key and value written into the cache at each sequence's position
+// seq_len - 1, all inside the attention kernel.
 extern "C" int qwb_attn_mma_decode_fused(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_t,
                                          const float* sin_t, float eps, int store_kv, void* k_pool, void* v_pool,
                                          const int* page_table, const int* seq_len, float* scratch, void* out, int B, int Hq,
@@ -808,11 +862,12 @@ extern "C" int qwb_attn_mma_decode_fused(const float* qkv, const float* q_weight
                                          int runs_target, int run_pages_max, int max_len, cudaStream_t stream) {
     if (B <= 0) return 0;
     int max_runs = 0;
-    if (int rc = check_decode(B, Hq, Hkv, hd, page_size, runs_target, run_pages_max, max_len, scratch, &max_runs)) return rc;
+    if (hd != 64 && hd != 128) return qwb_fail(QWB_ERR_ARG, "attn_mma_decode_fused: head size %d is not 64 or 128", hd);
+    if (int rc = check_decode(B, Hq, Hkv, hd, hd, page_size, runs_target, run_pages_max, max_len, scratch, &max_runs)) return rc;
     if (!qkv || (uintptr_t)qkv % 8 || (q_weight && (uintptr_t)q_weight % 8) || (cos_t && ((uintptr_t)cos_t % 8 || (uintptr_t)sin_t % 8)))
         return qwb_fail(QWB_ERR_ARG, "attn_mma_decode_fused: qkv, norm weights and cos/sin must be 8-byte aligned");
     if ((cos_t == nullptr) != (sin_t == nullptr)) return qwb_fail(QWB_ERR_ARG, "attn_mma_decode_fused: cos and sin come together");
     FusedQKV f = {qkv, q_weight, k_weight, cos_t, sin_t, (bf16*)k_pool, (bf16*)v_pool, eps, store_kv};
-    if (hd == 64) return launch_decode<64, true>(f, nullptr, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, table_width, scale, window, runs_target, run_pages_max, max_runs, stream);
-    return launch_decode<128, true>(f, nullptr, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, table_width, scale, window, runs_target, run_pages_max, max_runs, stream);
+    if (hd == 64) return launch_decode<64, 64, true, false>(f, nullptr, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, hd, hd, table_width, scale, window, runs_target, run_pages_max, max_runs, stream);
+    return launch_decode<128, 128, true, false>(f, nullptr, k_pool, v_pool, page_table, seq_len, scratch, out, B, Hq, Hkv, hd, hd, table_width, scale, window, runs_target, run_pages_max, max_runs, stream);
 }

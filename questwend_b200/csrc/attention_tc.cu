@@ -1,5 +1,8 @@
-// Prefill attention on the fifth-generation tensor cores (tcgen05), bfloat16, head sizes 64 and 128, groups of
-// up to 64 query heads per key/value head, pages of 64 keys.  Same contract as attn_prefill in attention.cu.
+// Prefill attention on the fifth-generation tensor cores (tcgen05), bfloat16, key and value sizes of up to 128 (multiples
+// of 8, equal or not), groups of up to 64 query heads per key/value head, pages of 64 keys.  Same contract as attn_prefill
+// in attention.cu.  Keys and values of other sizes than 64 and 128 are filled up to the next of the two by the TMA loads:
+// a box that reaches beyond a row's last value reads zeros there, which add nothing to a score and give outputs that are
+// not written.
 //
 // A block serves (128 / G tokens, rounded down) x (the G query heads of one key/value head) rows, up to 128; with a
 // G that does not divide 128 the last rows of the 128 stay unused.  Per tile of 64 keys (one cache page of that head):
@@ -7,7 +10,7 @@
 //                    buffers: the tensor core is up to two tiles ahead of the softmax)
 //     P = softmax    four warps, one thread per row: read S, mask, running maximum and sum in 32-bit, write P as
 //                    bfloat16 into shared memory in the layout the tensor core reads
-//     O += P V       tcgen05.mma, P and V from shared memory, O accumulates in tensor memory (HD columns).  V is read as
+//     O += P V       tcgen05.mma, P and V from shared memory, O accumulates in tensor memory (VD columns).  V is read as
 //                    it lies in the cache ([key][d], d contiguous): the "MN-major" operand form.
 // O lives in tensor memory across the tiles.  It carries a reference maximum per row; when a tile raises a row's
 // maximum by more than 2^8 the row's O and sum are rescaled (read, scale, write back), else the old reference stays
@@ -114,25 +117,27 @@ __host__ __device__ constexpr uint32_t at_idesc(int m, int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((b_mn ? 1u : 0u) << 16) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
 }
 
-template <int HD>
+template <int HD, int VD>
 struct AtSmem {
-    static constexpr int ATOMS = HD / 64;                                  // 128-byte pieces of a row of Q, K or V
-    static constexpr size_t Q_BYTES = (size_t)AT_ROWS * HD * 2;            // ATOMS blocks of [128 rows][128 bytes]
-    static constexpr size_t KV_BYTES = (size_t)AT_KEYS * HD * 2;           // ATOMS blocks of [64 keys][128 bytes]
+    static constexpr int K_ATOMS = HD / 64, V_ATOMS = VD / 64;             // 128-byte pieces of a row of Q and K, of V
+    static constexpr size_t Q_BYTES = (size_t)AT_ROWS * HD * 2;            // K_ATOMS blocks of [128 rows][128 bytes]
+    static constexpr size_t K_BYTES = (size_t)AT_KEYS * HD * 2;            // K_ATOMS blocks of [64 keys][128 bytes]
+    static constexpr size_t V_BYTES = (size_t)AT_KEYS * VD * 2;            // V_ATOMS such blocks
     static constexpr size_t P_BYTES = (size_t)AT_ROWS * AT_KEYS * 2;       // [128 rows][128 bytes]
-    static constexpr size_t BYTES = Q_BYTES + 2 * AT_KV_STAGES * KV_BYTES + P_BYTES + 128;   // 128: barriers, tensor-memory slot
+    static constexpr size_t BYTES = Q_BYTES + AT_KV_STAGES * (K_BYTES + V_BYTES) + P_BYTES + 128;   // 128: barriers, tensor-memory slot
 };
 
-template <int HD, bool SHAPED>      // SHAPED: the softmax also takes a distance bias per head and a sink (else the kernel is as it was)
+// HD, VD: key and value sizes filled up to 64 or 128; vd: the value size itself.
+template <int HD, int VD, bool SHAPED>      // SHAPED: the softmax also takes a distance bias per head and a sink (else the kernel is as it was)
 __global__ void __launch_bounds__(AT_THREADS)
 attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const int* __restrict__ page_table,
                        const int* __restrict__ cu_seqlens, const int* __restrict__ pos0, bf16* __restrict__ out, int Hq, int Hkv,
-                       int table_width, float scale, int window, int chunk, int G, int* error,
+                       int vd, int table_width, float scale, int window, int chunk, int G, int* error,
                        const float* __restrict__ slopes, const float* __restrict__ sinks) {
-    constexpr int ATOMS = AtSmem<HD>::ATOMS;
-    constexpr uint32_t KV_BYTES = AtSmem<HD>::KV_BYTES;
-    constexpr uint32_t TMEM_COLS = 256;                                     // S: 2 x 64 columns, O: HD columns
+    using Smem = AtSmem<HD, VD>;
+    constexpr uint32_t K_BYTES = Smem::K_BYTES, V_BYTES = Smem::V_BYTES;
+    constexpr uint32_t TMEM_COLS = 256;                                     // S: 2 x 64 columns, O: VD columns
     // The tiles need 1024-byte alignment (128-byte swizzle).  No padding to reach it: at head size 128 the block's
     // 113 KB then leave room for a second block on the SM, whose products run while this block's softmax does.
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -141,10 +146,10 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         return;
     }
     unsigned char* q_tile = smem_raw;
-    unsigned char* k_tiles = q_tile + AtSmem<HD>::Q_BYTES;
-    unsigned char* v_tiles = k_tiles + AT_KV_STAGES * KV_BYTES;
-    unsigned char* p_tile = v_tiles + AT_KV_STAGES * KV_BYTES;
-    uint64_t* q_full = reinterpret_cast<uint64_t*>(p_tile + AtSmem<HD>::P_BYTES);
+    unsigned char* k_tiles = q_tile + Smem::Q_BYTES;
+    unsigned char* v_tiles = k_tiles + AT_KV_STAGES * K_BYTES;
+    unsigned char* p_tile = v_tiles + AT_KV_STAGES * V_BYTES;
+    uint64_t* q_full = reinterpret_cast<uint64_t*>(p_tile + Smem::P_BYTES);
     uint64_t* k_full = q_full + 1;                       // K and V have barriers of their own: a K buffer is free as soon
     uint64_t* k_empty = k_full + AT_KV_STAGES;           // as its scores are formed, long before its tile's V buffer is
     uint64_t* v_full = k_empty + AT_KV_STAGES;
@@ -193,7 +198,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     __syncthreads();
     at_fence_after();
     const uint32_t tmem_s = *tmem_slot;                 // S: two buffers, columns [0, 64) and [64, 128)
-    const uint32_t tmem_o = tmem_s + 128;               // O: columns [128, 128 + HD)
+    const uint32_t tmem_o = tmem_s + 128;               // O: columns [128, 128 + VD)
 
     pdl_wait();
     pdl_launch_dependents();
@@ -201,7 +206,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     if (warp == 0) {
         if (lane == 0) {
             at_expect_tx(q_full, (uint32_t)(tok_per_block * G * HD * 2));      // the box's bytes: with G no divisor of 128, fewer than 128 rows
-            for (int a = 0; a < ATOMS; ++a)             // rows (token, head of the group): a box of [128 / G tokens][G heads][64 d]
+            for (int a = 0; a < Smem::K_ATOMS; ++a)     // rows (token, head of the group): a box of [128 / G tokens][G heads][64 d]
                 at_tma_3d(q_tile + (size_t)a * AT_ROWS * 128, &map_q, q_full, a * 64, kvh * G, t0 + q0);
             // K of tile j + 1 goes out before V of tile j: its buffer is free earlier (after the scores of tile j - 1,
             // not after the product of tile j - 2), and the tensor core wants it earlier (the scores run two tiles ahead).
@@ -213,9 +218,10 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 uint64_t* full = is_k ? &k_full[s] : &v_full[s];
                 if (j >= AT_KV_STAGES && !at_wait(empty, ((j / AT_KV_STAGES) - 1) & 1)) return false;
                 const int row0 = (pages[tile_first + j] * Hkv + kvh) * AT_KEYS;        // the (page, head) block's first row
-                unsigned char* dst = (is_k ? k_tiles : v_tiles) + (size_t)s * KV_BYTES;
-                at_expect_tx(full, KV_BYTES);
-                for (int a = 0; a < ATOMS; ++a)
+                const uint32_t bytes = is_k ? K_BYTES : V_BYTES;
+                unsigned char* dst = (is_k ? k_tiles : v_tiles) + (size_t)s * bytes;
+                at_expect_tx(full, bytes);
+                for (int a = 0; a < (is_k ? Smem::K_ATOMS : Smem::V_ATOMS); ++a)
                     at_tma_2d(dst + (size_t)a * AT_KEYS * 128, is_k ? &map_k : &map_v, full, a * 64, row0);
                 if (is_k) k_issued = j + 1; else v_issued = j + 1;
                 return true;
@@ -235,7 +241,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     } else if (warp == 1) {
         if (lane == 0) {
             constexpr uint32_t idesc_s = at_idesc(AT_ROWS, AT_KEYS, false);           // S [128 x 64] = Q [128 x HD] K[64 x HD]^T
-            constexpr uint32_t idesc_o = at_idesc(AT_ROWS, HD, true);                  // O [128 x HD] += P [128 x 64] V [64 x HD]
+            constexpr uint32_t idesc_o = at_idesc(AT_ROWS, VD, true);                  // O [128 x VD] += P [128 x 64] V [64 x VD]
             bool ok = at_wait(q_full, 0);
             // S runs two tiles ahead of P V: while the softmax warps work on one S buffer the tensor core fills the other.
             auto issue_s = [&](int j) -> bool {
@@ -243,7 +249,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 if (!at_wait(&k_full[s], (j / AT_KV_STAGES) & 1)) return false;
                 if (j >= 2 && !at_wait(&s_empty[j & 1], ((j >> 1) - 1) & 1)) return false;
                 at_fence_after();
-                const unsigned char* kt = k_tiles + (size_t)s * KV_BYTES;
+                const unsigned char* kt = k_tiles + (size_t)s * K_BYTES;
 #pragma unroll
                 for (int k = 0; k < HD / 16; ++k) {                                    // 16 values of d per product
                     const uint64_t da = at_desc_kmajor(q_tile + (size_t)(k / 4) * AT_ROWS * 128) + 2 * (k % 4);
@@ -261,7 +267,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 ok = at_wait(&v_full[s], (j / AT_KV_STAGES) & 1) && at_wait(p_full, j & 1);   // V has landed; P is in shared memory
                 if (!ok) break;
                 at_fence_after();
-                const unsigned char* vt = v_tiles + (size_t)s * KV_BYTES;
+                const unsigned char* vt = v_tiles + (size_t)s * V_BYTES;
 #pragma unroll
                 for (int k = 0; k < AT_KEYS / 16; ++k) {                               // 16 keys per product
                     const uint64_t da = at_desc_kmajor(p_tile) + 2 * k;
@@ -361,7 +367,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 if (!ok) { if (lane == 0) atomicExch(error, 4); break; }
                 if (__any_sync(0xffffffffu, rescale)) {                                 // some row of this warp moves its reference: rescale O
 #pragma unroll 1
-                    for (int c = 0; c < HD; c += 32) {
+                    for (int c = 0; c < VD; c += 32) {
                         uint32_t ov[32];
                         at_ld32(tmem_o + lane_off + c, ov);
 #pragma unroll
@@ -389,9 +395,9 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             // a sink: one more term of the denominator, exp(sink), relative to the row's reference
             if (SHAPED && sinks && row_ok) l += at_exp2(sinks[head] * 1.4426950408889634f - (m_ref == -INFINITY ? 0.f : m_ref * sl2));
             const float inv = l > 0.f ? 1.f / l : 0.f;
-            bf16* dst = out + ((size_t)(t0 + tok) * Hq + head) * HD;
+            bf16* dst = out + ((size_t)(t0 + tok) * Hq + head) * vd;
 #pragma unroll 1
-            for (int c = 0; c < HD; c += 32) {
+            for (int c = 0; c < VD; c += 32) {
                 uint32_t ov[32];
                 at_ld32(tmem_o + lane_off + c, ov);
                 if (row_ok) {
@@ -403,7 +409,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                             __nv_bfloat162 v = __floats2bfloat162_rn(__uint_as_float(ov[i + 2 * u]) * inv, __uint_as_float(ov[i + 2 * u + 1]) * inv);
                             pk[u] = *reinterpret_cast<uint32_t*>(&v);
                         }
-                        *reinterpret_cast<uint4*>(dst + c + i) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                        if (c + i < vd) *reinterpret_cast<uint4*>(dst + c + i) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                     }
                 }
             }
@@ -433,17 +439,17 @@ static AtEncodeFn at_encode() {
     return fn;
 }
 
-template <int HD>
+template <int HD, int VD>
 static int launch_attn_tc(const void* q, const void* k_pool, const void* v_pool, const int* page_table, const int* cu_seqlens,
-                          const int* pos0, void* out, int B, int T, int max_new, int n_pages, int Hq, int Hkv, int table_width,
+                          const int* pos0, void* out, int B, int T, int max_new, int n_pages, int Hq, int Hkv, int hd, int vd, int table_width,
                           float scale, int window, int chunk, int* error, const float* slopes, const float* sinks, cudaStream_t stream) {
     AtEncodeFn enc = at_encode();
     if (!enc) return qwb_fail(QWB_ERR_CUDA, "attn_tc_prefill: cuTensorMapEncodeTiled is not available from this driver");
     const int G = Hq / Hkv;
     CUtensorMap map_q, map_k, map_v;
-    {   // q [T, Hq, HD]: boxes of [128 / G tokens][G heads][64 d]
-        cuuint64_t dims[3] = {(cuuint64_t)HD, (cuuint64_t)Hq, (cuuint64_t)T};
-        cuuint64_t strides[2] = {(cuuint64_t)HD * 2, (cuuint64_t)Hq * HD * 2};
+    {   // q [T, Hq, hd]: boxes of [128 / G tokens][G heads][64 d]
+        cuuint64_t dims[3] = {(cuuint64_t)hd, (cuuint64_t)Hq, (cuuint64_t)T};
+        cuuint64_t strides[2] = {(cuuint64_t)hd * 2, (cuuint64_t)Hq * hd * 2};
         cuuint32_t box[3] = {64, (cuuint32_t)G, (cuuint32_t)(AT_ROWS / G)};
         cuuint32_t elem[3] = {1, 1, 1};
         CUresult r = enc(&map_q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), dims, strides, box, elem,
@@ -453,9 +459,10 @@ static int launch_attn_tc(const void* q, const void* k_pool, const void* v_pool,
     }
     const void* pools[2] = {k_pool, v_pool};
     CUtensorMap* maps[2] = {&map_k, &map_v};
-    for (int i = 0; i < 2; ++i) {   // a pool [pages, Hkv, 64, HD] as rows of HD: boxes of [64 keys][64 d]
-        cuuint64_t dims[2] = {(cuuint64_t)HD, (cuuint64_t)n_pages * Hkv * AT_KEYS};
-        cuuint64_t strides[1] = {(cuuint64_t)HD * 2};
+    for (int i = 0; i < 2; ++i) {   // a pool [pages, Hkv, 64, size] as rows of `size` values: boxes of [64 keys][64 d]
+        const int size = i == 0 ? hd : vd;
+        cuuint64_t dims[2] = {(cuuint64_t)size, (cuuint64_t)n_pages * Hkv * AT_KEYS};
+        cuuint64_t strides[1] = {(cuuint64_t)size * 2};
         cuuint32_t box[2] = {64, AT_KEYS};
         cuuint32_t elem[2] = {1, 1};
         CUresult r = enc(maps[i], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(pools[i]), dims, strides, box, elem,
@@ -463,33 +470,36 @@ static int launch_attn_tc(const void* q, const void* k_pool, const void* v_pool,
                          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) return qwb_fail(QWB_ERR_CUDA, "attn_tc_prefill: cuTensorMapEncodeTiled(cache) failed with %d", (int)r);
     }
-    const size_t smem = AtSmem<HD>::BYTES;
-    const bool shaped = slopes || sinks;
-    cudaError_t e = shaped ? cudaFuncSetAttribute(attn_tc_prefill_kernel<HD, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
-                           : cudaFuncSetAttribute(attn_tc_prefill_kernel<HD, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "attn_tc_prefill: %s", cudaGetErrorString(e));
+    const size_t smem = AtSmem<HD, VD>::BYTES;
     const int tok_per_block = AT_ROWS / G;
     dim3 grid(Hkv, (max_new + tok_per_block - 1) / tok_per_block, B);
-    if (shaped)
-        e = qwb_launch(attn_tc_prefill_kernel<HD, true>, grid, AT_THREADS, smem, stream, map_q, map_k, map_v, page_table, cu_seqlens, pos0,
-                       (bf16*)out, Hq, Hkv, table_width, scale, window, chunk, G, error, slopes, sinks);
-    else
-        e = qwb_launch(attn_tc_prefill_kernel<HD, false>, grid, AT_THREADS, smem, stream, map_q, map_k, map_v, page_table, cu_seqlens, pos0,
-                       (bf16*)out, Hq, Hkv, table_width, scale, window, chunk, G, error, slopes, sinks);
-    if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "attn_tc_prefill: launch failed: %s", cudaGetErrorString(e));
-    return qwb_check_launch("attn_tc_prefill");
+    auto go = [&](auto kernel) -> int {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "attn_tc_prefill: %s", cudaGetErrorString(e));
+        e = qwb_launch(kernel, grid, AT_THREADS, smem, stream, map_q, map_k, map_v, page_table, cu_seqlens, pos0,
+                       (bf16*)out, Hq, Hkv, vd, table_width, scale, window, chunk, G, error, slopes, sinks);
+        if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "attn_tc_prefill: launch failed: %s", cudaGetErrorString(e));
+        return qwb_check_launch("attn_tc_prefill");
+    };
+    if (slopes || sinks) {
+        if constexpr (HD == VD) return go(attn_tc_prefill_kernel<HD, VD, true>);
+        else return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: a distance bias or a sink goes with keys and values of about one size, not %d and %d", hd, vd);
+    }
+    return go(attn_tc_prefill_kernel<HD, VD, false>);
 }
 
-// bfloat16.  q [T, Hq, hd] with T the packed tokens of all B sequences; pools of n_pages pages; `error` as for qwb_gemm_tc.
+// bfloat16.  q [T, Hq, hd] with T the packed tokens of all B sequences; pools of n_pages pages, keys of hd and values of vd
+// values; out [T, Hq * vd]; `error` as for qwb_gemm_tc.
 // `chunk` > 0: a query sees the keys of its own block of `chunk` positions only (beside the causal mask and the window).
 // `slopes` [Hq] (or null): slopes[h] * (query position - key position) is taken off the scaled score; `sinks` [Hq] (or
 // null): exp(sinks[h]) joins the softmax's denominator.
-extern "C" int qwb_attn_tc_prefill_shaped(const void* q, const void* k_pool, const void* v_pool, const int* page_table,
-                                          const int* cu_seqlens, const int* pos0, void* out, int B, int T, int max_new, int n_pages,
-                                          int Hq, int Hkv, int hd, int page_size, int table_width, float scale, int window,
-                                          int chunk, const float* slopes, const float* sinks, int* error, cudaStream_t stream) {
+extern "C" int qwb_attn_tc_prefill(const void* q, const void* k_pool, const void* v_pool, const int* page_table,
+                                   const int* cu_seqlens, const int* pos0, void* out, int B, int T, int max_new, int n_pages,
+                                   int Hq, int Hkv, int hd, int vd, int page_size, int table_width, float scale, int window,
+                                   int chunk, const float* slopes, const float* sinks, int* error, cudaStream_t stream) {
     if (B <= 0 || max_new <= 0 || T <= 0) return 0;
-    if (hd != 64 && hd != 128) return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: head size %d is not 64 or 128", hd);
+    if (hd <= 0 || hd > 128 || hd % 8 || vd <= 0 || vd > 128 || vd % 8)
+        return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: key size %d or value size %d is not a multiple of 8 up to 128", hd, vd);
     if (page_size != AT_KEYS) return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: page size %d is not %d", page_size, AT_KEYS);
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv) return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: %d query heads are not a multiple of %d key/value heads", Hq, Hkv);
     const int G = Hq / Hkv;
@@ -501,22 +511,14 @@ extern "C" int qwb_attn_tc_prefill_shaped(const void* q, const void* k_pool, con
     if ((uintptr_t)q % 16 || (uintptr_t)k_pool % 16 || (uintptr_t)v_pool % 16 || (uintptr_t)out % 16)
         return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: operands must be 16-byte aligned");
     if (!(scale > 0.f) && slopes) return qwb_fail(QWB_ERR_ARG, "attn_tc_prefill: a distance bias needs a positive scale, got %g", (double)scale);
-    if (hd == 64) return launch_attn_tc<64>(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, T, max_new, n_pages, Hq, Hkv, table_width, scale, window, chunk, error, slopes, sinks, stream);
-    return launch_attn_tc<128>(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, T, max_new, n_pages, Hq, Hkv, table_width, scale, window, chunk, error, slopes, sinks, stream);
-}
-
-extern "C" int qwb_attn_tc_prefill_chunked(const void* q, const void* k_pool, const void* v_pool, const int* page_table,
-                                           const int* cu_seqlens, const int* pos0, void* out, int B, int T, int max_new, int n_pages,
-                                           int Hq, int Hkv, int hd, int page_size, int table_width, float scale, int window,
-                                           int chunk, int* error, cudaStream_t stream) {
-    return qwb_attn_tc_prefill_shaped(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, T, max_new, n_pages, Hq, Hkv, hd,
-                                      page_size, table_width, scale, window, chunk, nullptr, nullptr, error, stream);
-}
-
-extern "C" int qwb_attn_tc_prefill(const void* q, const void* k_pool, const void* v_pool, const int* page_table,
-                                   const int* cu_seqlens, const int* pos0, void* out, int B, int T, int max_new, int n_pages,
-                                   int Hq, int Hkv, int hd, int page_size, int table_width, float scale, int window, int* error,
-                                   cudaStream_t stream) {
-    return qwb_attn_tc_prefill_chunked(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, T, max_new, n_pages, Hq, Hkv, hd,
-                                       page_size, table_width, scale, window, 0, error, stream);
+#define QWB_AT_LAUNCH(HD, VD)                                                                                                       \
+    return launch_attn_tc<HD, VD>(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, T, max_new, n_pages, Hq, Hkv, hd, vd,   \
+                                  table_width, scale, window, chunk, error, slopes, sinks, stream)
+    if (hd <= 64) {
+        if (vd <= 64) QWB_AT_LAUNCH(64, 64);
+        QWB_AT_LAUNCH(64, 128);
+    }
+    if (vd <= 64) QWB_AT_LAUNCH(128, 64);
+    QWB_AT_LAUNCH(128, 128);
+#undef QWB_AT_LAUNCH
 }

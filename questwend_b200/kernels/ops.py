@@ -384,9 +384,20 @@ def tc_attention_fits(dtype: torch.dtype, head_dim: int, page_size: int, group: 
     return mma_attention_fits(dtype, head_dim, page_size) and 1 <= group <= 64
 
 
+PART_ATTN_MAX_DIM = 128     # key and value sizes, multiples of 8 up to this, that the tcgen05 prompt kernel and the tensor-core
+                            # decode kernel take, each of its own size (filled up to 64 or 128 on the chip)
+
+
+def part_attention_fits(dtype: torch.dtype, dim: int, vdim: int, page_size: int, group: int) -> bool:
+    """Whether both of these kernels take keys of ``dim`` and values of ``vdim``."""
+    return (dtype == torch.bfloat16 and page_size == 64 and 1 <= group <= 64
+            and all(0 < n <= PART_ATTN_MAX_DIM and n % 8 == 0 for n in (dim, vdim)))
+
+
 def attn_prefill(q, k_pool, v_pool, page_table, cu_seqlens, pos0, max_new: int, scale: float,
                  window: int = 0, impl: str = "auto", chunk: int = 0, slopes=None, sinks=None) -> torch.Tensor:
-    """Causal attention of new tokens over the cache.  q [T, Hq, hd]; returns [T, Hq * hd].
+    """Causal attention of new tokens over the cache.  q [T, Hq, hd]; returns [T, Hq * hd] (values of another size than
+    the keys', the tcgen05 kernel only: [T, Hq * value size]).
     impl: "auto" (the fastest that fits), "tc" (tcgen05), "mma" (mma.sync), or "plain".  ``chunk`` > 0: a query sees only
     the keys of its own block of ``chunk`` positions, counted from position 0; ``slopes`` / ``sinks`` (float32 [Hq]): a
     bias slopes[h] * distance off the scaled score, and exp(sinks[h]) in the softmax's denominator (all three: the
@@ -401,7 +412,8 @@ def attn_prefill(q, k_pool, v_pool, page_table, cu_seqlens, pos0, max_new: int, 
     B = pos0.numel()
     if cu_seqlens.numel() != B + 1 or page_table.shape[0] < B:
         raise KernelError("attn_prefill: cu_seqlens / page_table do not fit the batch")
-    out = torch.empty((T, Hq * hd), dtype=q.dtype, device=q.device)
+    vd = v_pool.shape[3]
+    out = torch.empty((T, Hq * vd), dtype=q.dtype, device=q.device)
     group = Hq // max(1, k_pool.shape[1])
     # the tcgen05 kernel works on tiles of 128 rows: it pays from a few dozen new tokens per sequence on
     use_tc = impl == "tc" or (impl == "auto" and max_new * group >= 64 and
@@ -414,13 +426,14 @@ def attn_prefill(q, k_pool, v_pool, page_table, cu_seqlens, pos0, max_new: int, 
                 _need(t, name, torch.float32, 1)
                 if t.numel() != Hq:
                     raise KernelError(f"attn_prefill: {name} of {t.numel()} for {Hq} heads")
-        _call("attention_tc", "qwb_attn_tc_prefill_shaped", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table),
+        _call("attention_tc", "qwb_attn_tc_prefill", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table),
               _ptr(cu_seqlens), _ptr(pos0), _ptr(out), _i(B), _i(T), _i(max_new), _i(k_pool.shape[0]), _i(Hq),
-              _i(k_pool.shape[1]), _i(hd), _i(k_pool.shape[2]), _i(page_table.shape[1]), _f(scale), _i(window), _i(chunk),
+              _i(k_pool.shape[1]), _i(hd), _i(vd), _i(k_pool.shape[2]), _i(page_table.shape[1]), _f(scale), _i(window), _i(chunk),
               _ptr(slopes), _ptr(sinks), _ptr(gemm_tc_error_word(q.device)), _stream())
         return out
-    if chunk or slopes is not None or sinks is not None:
-        raise KernelError("attn_prefill: only the tcgen05 kernel masks by chunks, biases by distance or has a sink")
+    if chunk or slopes is not None or sinks is not None or vd != hd:
+        raise KernelError("attn_prefill: only the tcgen05 kernel masks by chunks, biases by distance, has a sink or takes values of "
+                          "another size than the keys'")
     use_mma = impl == "mma" or (impl == "auto" and mma_attention_fits(q.dtype, hd, k_pool.shape[2]))
     if use_mma:
         if q.dtype != torch.bfloat16:
@@ -457,29 +470,34 @@ def attn_decode(q, k_pool, v_pool, page_table, seq_len, scale: float, max_len: i
     The keys are cut into runs whose partial results are merged.  The plain kernel cuts into runs of
     ``split_tokens`` keys.  The tensor-core kernel cuts a sequence of p pages into runs of
     clamp(ceil(p / runs_target), 1, run_pages_max) pages (``runs_target`` 1: runs of exactly ``run_pages_max``
-    pages): by the sequence's own length, never by what else is in the batch."""
+    pages): by the sequence's own length, never by what else is in the batch.  It also takes (``impl`` "mma") keys and
+    values of other sizes (``part_attention_fits``); the result is then [B, Hq * value size]."""
     _need(q, "q", k_pool.dtype, 3)
     _need(k_pool, "k_pool", ndim=4)
     _need(v_pool, "v_pool", k_pool.dtype, 4)
     _need(page_table, "page_table", torch.int32, 2)
     _need(seq_len, "seq_len", torch.int32, 1)
     B, Hq, hd = q.shape
-    use_mma = impl == "mma" or (impl == "auto" and mma_attention_fits(q.dtype, hd, k_pool.shape[2]))
+    vd = v_pool.shape[3]
+    use_mma = impl == "mma" or (impl == "auto" and mma_attention_fits(q.dtype, hd, k_pool.shape[2]) and vd == hd)
     if use_mma and q.dtype != torch.bfloat16:
         raise KernelError("attn_decode: the tensor-core kernel takes bfloat16 only")
+    if not use_mma and vd != hd:
+        raise KernelError(f"attn_decode: values of {vd} beside keys of {hd}: the tensor-core kernel only")
     if use_mma:
         max_runs = max(1, mma_decode_runs(max_len, runs_target, run_pages_max))
     else:
         max_runs = max(1, math.ceil(max_len / split_tokens))
-    need = attn_decode_scratch_floats(B, Hq, hd, max_runs) if max_runs > 1 else 0
+    held = (64 if vd <= 64 else 128) if use_mma else hd         # values of a partial result
+    need = attn_decode_scratch_floats(B, Hq, held, max_runs) if max_runs > 1 else 0
     if need and (scratch is None or scratch.numel() < need):
         scratch = torch.empty(need, dtype=torch.float32, device=q.device)
     if scratch is not None:
         _need(scratch, "scratch", torch.float32)
-    out = torch.empty((B, Hq * hd), dtype=q.dtype, device=q.device)
+    out = torch.empty((B, Hq * vd), dtype=q.dtype, device=q.device)
     if use_mma:
         _call("attention_mma", "qwb_attn_mma_decode", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table),
-              _ptr(seq_len), _ptr(scratch), _ptr(out), _i(B), _i(Hq), _i(k_pool.shape[1]), _i(hd), _i(k_pool.shape[2]),
+              _ptr(seq_len), _ptr(scratch), _ptr(out), _i(B), _i(Hq), _i(k_pool.shape[1]), _i(hd), _i(vd), _i(k_pool.shape[2]),
               _i(page_table.shape[1]), _f(scale), _i(window), _i(runs_target), _i(run_pages_max), _i(max_len), _stream(),
               kernels=2 if max_runs > 1 else 1)
         return out
@@ -1146,8 +1164,7 @@ def pool_attention(q: torch.Tensor, k_pool, v_pool, pk_pool, pv_pool, page_table
                    scale: float, window: int, pool: int, interleaved: bool, impl: str = "auto") -> torch.Tensor:
     """Attention of a step's tokens over their window and the block rows before it.  ``q`` [T, H, dim] in the cache's
     dtype; returns [T, H * vdim] in that dtype, each head turned back by the query's position if ``cos_v`` is given.
-    Steps of one token per sequence take the kernels that cut the keys into runs (one uncapped map over all keys with keys
-    and values of 64 or 128: plain grouped-query attention's; other sizes that are multiples of 8: the one for maps); other
+    Steps of one token per sequence take the kernel that cuts the keys into runs (sizes that are multiples of 8); other
     steps the tensor-core kernel where it fits (``impl`` "auto" or "mma"), else the plain one ("plain")."""
     _need(q, "q", k_pool.dtype, 3)
     T, H, dim = q.shape
@@ -1247,9 +1264,11 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
     the cache's dtype; returns [T, H * vdim] in that dtype: map 0's output, minus ``lam`` times map 1's if there are two,
     then (``norm_out``) divided by its root mean square over vdim and multiplied by ``out_scale``.  Scores are scaled,
     soft-capped (``softcap`` > 0) and masked causally, and to the query's chunk of ``chunk`` positions if that is > 0.
-    Steps of one token per sequence take the kernel that cuts the keys into runs (sizes that are multiples of 8); other
-    steps the tensor-core kernels where they fit (``impl`` "auto"; "tc": tcgen05, for one uncapped map with keys and values
-    of 64 or 128; "mma": mma.sync), else the plain one ("plain")."""
+    One uncapped map in bfloat16 with keys and values of up to 128 (multiples of 8) is plain grouped-query attention and
+    takes its kernels (``impl`` "auto" or "tc"): in steps of one token per sequence the tensor-core decode kernel (all keys
+    visible), in others the tcgen05 one.  Else steps of one token per sequence take the kernel for maps that cuts the keys
+    into runs (sizes that are multiples of 8), and other steps the tensor-core kernel for maps where it fits ("mma":
+    mma.sync), else the plain one ("plain")."""
     _need(q, "q", k_pool.dtype, 3)
     T, H, kdim = q.shape
     G, vdim = k_pool.shape[1], v_pool.shape[3]
@@ -1258,9 +1277,10 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
     dim = kdim // maps
     out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
     width = page_table.shape[1]
-    plain = maps == 1 and softcap <= 0.0 and not norm_out and out_scale == 1.0 and dim == vdim
-    if ctx.single_token and impl == "auto" and plain and chunk == 0 and mma_attention_fits(q.dtype, dim, k_pool.shape[2]):
-        return attn_decode(q, k_pool, v_pool, page_table, ctx.seq_len, scale, ctx.max_len)
+    one_map = (maps == 1 and softcap <= 0.0 and not norm_out and out_scale == 1.0 and impl in ("auto", "tc")
+               and part_attention_fits(q.dtype, dim, vdim, k_pool.shape[2], H // G))
+    if ctx.single_token and one_map and chunk == 0:
+        return attn_decode(q, k_pool, v_pool, page_table, ctx.seq_len, scale, ctx.max_len, impl="mma")
     if ctx.single_token and dim % MAPS_FAST_STEP == 0 and vdim % MAPS_FAST_STEP == 0:
         lib = _lookup("attention_maps", "qwb_maps_decode_runs")[0]
         n_runs = lib.qwb_maps_decode_runs(_i(ctx.max_len), _i(chunk))
@@ -1271,9 +1291,8 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
               _ptr(scratch), _ptr(out), _i(_dt(q.dtype)), _i(T), _i(H), _i(G), _i(maps), _i(dim), _i(vdim), _i(width), _f(scale),
               _f(softcap), _i(chunk), _i(n_runs), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), _stream(), kernels=2)
         return out
-    # one map, no cap, keys and values of one size: the prompt kernel of plain grouped-query attention, with the chunk mask
-    if (impl in ("auto", "tc") and plain and q.dtype == torch.bfloat16
-            and ctx.max_new * (H // G) >= 64 and tc_attention_fits(q.dtype, dim, k_pool.shape[2], H // G)):
+    # one map, no cap: the prompt kernel of plain grouped-query attention, with the chunk mask
+    if one_map and ctx.max_new * (H // G) >= 64:
         return attn_prefill(q, k_pool, v_pool, page_table, ctx.cu_seqlens, ctx.pos0, ctx.max_new, scale, impl="tc", chunk=chunk)
     if impl == "mma" or (impl == "auto" and maps_prefill_mma_fits(q.dtype, maps, dim, vdim)):
         _call("attention_maps", "qwb_maps_prefill_mma", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), _ptr(ctx.cu_seqlens),

@@ -324,9 +324,9 @@ class ScoreMapsAttention(Mixer):
 
     def kernel_modules(self):
         mods = ["attention_maps", "rope_kv", "elementwise", *(("recurrent",) if self.taps else ()), *linear_modules(self.runtime.dtype)]
-        if (self.maps == 1 and self.softcap <= 0.0 and self.head_dim == self.value_dim
-                and ops.tc_attention_fits(self.runtime.dtype, self.head_dim, ops.PAGE_SIZE, self.n_heads // self.n_kv_heads)):
-            mods.append("attention_tc")         # prompts of one uncapped map with keys and values of 64 or 128 ...
+        if (self.maps == 1 and self.softcap <= 0.0
+                and ops.part_attention_fits(self.runtime.dtype, self.head_dim, self.value_dim, ops.PAGE_SIZE, self.n_heads // self.n_kv_heads)):
+            mods.append("attention_tc")         # prompts of one uncapped map ...
             if self.chunk == 0:
                 mods.append("attention_mma")    # ... and its single tokens over all keys
         return tuple(mods)

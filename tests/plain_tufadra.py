@@ -106,6 +106,23 @@ def route(z, correction, router):
     return chosen, weights
 
 
+def route_margin(z, correction, router):
+    """How far each token's choice is from another one: the least gap, in choice scores, between what is taken and the next
+    best that is not (groups, and experts inside the groups that are taken)."""
+    n, E = z.shape
+    groups = router.get("groups") or {"count": 1, "keep": 1}
+    count, keep, top = groups["count"], groups["keep"], router["top"]
+    c = (sigmoid(z) + correction).reshape(n, count, E // count)
+    g = np.sort(c, axis=-1)[..., -2:].sum(axis=-1)
+    order = np.argsort(-g, axis=-1, kind="stable")
+    ranked = np.take_along_axis(g, order, axis=-1)
+    margin = ranked[:, keep - 1] - ranked[:, keep] if keep < count else np.full(n, np.inf)
+    inside = -np.sort(-np.take_along_axis(c, order[:, :keep, None], axis=1).reshape(n, -1), axis=-1)
+    if top < inside.shape[1]:
+        margin = np.minimum(margin, inside[:, top - 1] - inside[:, top])
+    return margin
+
+
 def expert(h, w, px, round16=False):
     return product(gelu_exact(product(h, w[px + "up"], round16)), w[px + "down"], round16)
 
@@ -115,8 +132,11 @@ def shared_expert(h, w, px, round16=False):
     return expert(h, w, px, round16) * sigmoid(product(h, w[px + "sg"], round16))
 
 
-def experts(h, mlp, w, px, round16=False):
-    chosen, weights = route(product(h, w[px + "router"], round16), w[px + "correction"], mlp["router"])
+def experts(h, mlp, w, px, round16=False, margins=None):
+    z = product(h, w[px + "router"], round16)
+    chosen, weights = route(z, w[px + "correction"], mlp["router"])
+    if margins is not None:
+        margins.append(route_margin(z, w[px + "correction"], mlp["router"]))
     out = np.zeros_like(h)
     for e in range(mlp["router"]["experts"]):
         t, k = np.nonzero(chosen == e)
@@ -135,8 +155,9 @@ def weights_layer(cfg, i):
     return i
 
 
-def forward(cfg, w, tokens, round16=False, taps=None):
-    """Logits [n, vocab] of one sequence; ``taps``, a list, receives the stream after every layer."""
+def forward(cfg, w, tokens, round16=False, taps=None, margins=None):
+    """Logits [n, vocab] of one sequence; ``taps``, a list, receives the stream after every layer, ``margins`` every
+    router's margin for every token."""
     eps = cfg["norm"]["eps"]
     x = embed(tokens, w)
     for i, layer in enumerate(cfg["layers"]):
@@ -144,7 +165,7 @@ def forward(cfg, w, tokens, round16=False, taps=None):
         h = norm_about_one(x, w[px + "norm1"], eps)
         y = MIXERS[layer["type"]](h, layer["mixer"], w, px + "mix.", eps, round16)
         if layer.get("mlp") is not None:
-            y = y + experts(h, layer["mlp"], w, px + "mlp.", round16)
+            y = y + experts(h, layer["mlp"], w, px + "mlp.", round16, margins)
         x = x + y
         if taps is not None:
             taps.append(x.copy())

@@ -29,14 +29,11 @@ def close(got, ref, dtype, tol=FP32_TOL):
     return np.sqrt(np.mean((got - ref) ** 2)) <= BF16_RMS_TOL * np.sqrt(np.mean(ref ** 2))
 
 
-def close_rows(got, ref, dtype):
-    """``close`` for a whole model.  In bfloat16 a router's choice between two experts with nearly equal choice scores can
-    fall either way, so a row in twenty (or one) may be off; every other row is held to the tolerance by itself."""
-    if dtype == torch.float32:
-        return close(got, ref, dtype)
-    got, ref = np.asarray(got, dtype=np.float64), np.asarray(ref, dtype=np.float64)
+def most_rows_close(got, ref):
+    """Of a bfloat16 model's tokens, where a router's choice between two experts with nearly equal choice scores can fall
+    either way: a row in ten may be off; every other row is held to the tolerance by itself."""
     err = np.sqrt(np.mean((got - ref) ** 2, axis=-1)) / np.sqrt(np.mean(ref ** 2))
-    return np.sum(err > BF16_RMS_TOL) <= max(1, len(err) // 10)
+    return np.sum(err > BF16_RMS_TOL) <= len(err) // 10
 
 
 def dev(a, dtype=torch.float32):
@@ -149,22 +146,10 @@ def test_norms_over_whole_projections_and_the_query_factor(H, G, maps, dim, vdim
 
 # ----------------------------------------------------------------------------- the router and the experts
 def decided(z, correction, router, margin=1e-5):
-    """Tokens whose choice no rounding can change: the best group (or expert) that is left out is at least ``margin``
-    behind the worst that is taken."""
-    E, count, keep, top = router["experts"], router["groups"]["count"], router["groups"]["keep"], router["top"]
-    c = pt.sigmoid(z) + correction
-    g = np.sort(c.reshape(len(z), count, E // count), axis=-1)[..., -2:].sum(-1)
-    order = np.sort(g, axis=-1)[:, ::-1]
-    ok = np.ones(len(z), dtype=bool) if keep == count else order[:, keep - 1] - order[:, keep] > margin
-    kept = np.argsort(-g, axis=-1, kind="stable")[:, :keep]
-    inside = np.full_like(c, -np.inf)
-    for t in range(len(z)):
-        for grp in kept[t]:
-            s = slice(grp * (E // count), (grp + 1) * (E // count))
-            inside[t, s] = c[t, s]
-    best = np.sort(inside, axis=-1)[:, ::-1][:, :top + 1]
-    gaps = best[:, :-1] - best[:, 1:]                       # also between the chosen ones: their order is compared
-    return ok & (np.nan_to_num(gaps[:, :min(top, E - 1)], nan=1.0, posinf=1.0).min(axis=-1, initial=1.0) > margin)
+    """Tokens whose choice, and whose order of the chosen, no rounding can change."""
+    chosen, _ = pt.route(z, correction, router)
+    c = np.take_along_axis(pt.sigmoid(z) + correction, chosen, axis=-1)
+    return (pt.route_margin(z, correction, router) > margin) & ((c[:, :-1] - c[:, 1:]).min(axis=-1, initial=1.0) > margin)
 
 
 @pytest.mark.parametrize("E, top, count, keep", [(6, 3, 3, 2), (12, 5, 2, 1), (5, 5, 1, 1), (4, 2, 4, 3), (1, 1, 1, 1), (64, 8, 8, 4), (96, 6, 3, 1),
@@ -322,6 +307,61 @@ def test_attention_alone(entry, dtype):
             assert close(g, ref, dtype)
 
 
+@pytest.mark.parametrize("H, G, dim, vdim", [(4, 2, 64, 32), (8, 2, 128, 64), (6, 1, 64, 128), (4, 4, 96, 120), (2, 1, 128, 128), (40, 2, 8, 8), (3, 3, 120, 16),
+                                             (16, 1, 64, 64), (4, 2, 80, 128), (2, 2, 136, 64)])
+def test_keys_and_values_of_their_own_sizes(H, G, dim, vdim):
+    """The tensor-core kernels (and, for the last sizes, those they leave to others) against an oracle over a random cache
+    whose other pages hold large numbers: whole unequal prompts, later portions that start inside a page, and single tokens
+    after up to 2,300 keys; per sequence one query whose key stands out, far away or at a page's edge."""
+    from questwend_b200.parts.base import KVSpec
+    rng = np.random.default_rng(H * 1000 + dim + vdim)
+    for lens, news in (([300, 70, 17, 64], ([300, 70, 17, 64], [121, 70, 3, 1])), ([2300, 65, 1, 1024], ([1, 1, 1, 1], [40, 64, 1, 2]))):
+        cache = CacheManager([(KVSpec(G, dim, 0, value_dim=vdim), None, None)], sum(lens) + 64 * 8, 4, max(lens) + 64, torch.bfloat16, DEV)
+        unit = cache.unit_cache(0)
+        unit.k_pool.fill_(50.0)
+        unit.v_pool.fill_(-1000.0)
+        ks = [pt.round_bf16(rng.standard_normal((n, G, dim))) for n in lens]
+        vs = [pt.round_bf16(rng.standard_normal((n, G, vdim))) for n in lens]
+        for counts in news:
+            slots = cache.open(4)
+            before = [n - c for n, c in zip(lens, counts)]
+            for s, n in zip(slots, before):
+                if n:
+                    build_step_context(cache, [StepEntry(s, [0] * n, [])], 10, DEV)
+                    cache.advance(s, n)
+            ctx = build_step_context(cache, [StepEntry(s, [0] * c, []) for s, c in zip(slots, counts)], 10, DEV)[0]
+            table = ctx.page_tables[unit.group_id]
+            qs = [pt.round_bf16(rng.standard_normal((c, H, dim))) for c in counts]
+            for b in range(4):
+                for i in range(0, counts[b], 7):
+                    p = before[b] + i
+                    far = [0, 1, 63, 64, p // 2, 64 * (p // 64), 64 * (p // 64) - 1][(i // 7) % 7]
+                    if 0 <= far <= p:                               # every head's query along its own key head's vector there
+                        qs[b][i] = pt.round_bf16(np.repeat(ks[b][far], H // G, axis=0) * 3.0)
+            host_table = table.cpu().numpy()
+            for b, (k, v) in enumerate(zip(ks, vs)):                 # the cache as a prep kernel would have left it
+                for page in range(-(-lens[b] // 64)):
+                    rows = slice(64 * page, min(64 * page + 64, lens[b]))
+                    n = rows.stop - rows.start
+                    unit.k_pool[host_table[b, page], :, :n] = dev(k[rows].transpose(1, 0, 2), torch.bfloat16)
+                    unit.v_pool[host_table[b, page], :, :n] = dev(v[rows].transpose(1, 0, 2), torch.bfloat16)
+            want = []
+            for q, k, v, n0 in zip(qs, ks, vs, before):
+                o = np.zeros((len(q), H, vdim))
+                seen = np.arange(len(k))[None, :] <= n0 + np.arange(len(q))[:, None]
+                for h in range(H):
+                    s = np.where(seen, q[:, h] @ k[:, h // (H // G)].T * 0.2, -np.inf)
+                    e = np.exp(s - s.max(-1, keepdims=True))
+                    o[:, h] = e @ v[:, h // (H // G)] / e.sum(-1, keepdims=True)
+                want.append(o.reshape(len(q), -1))
+            want = np.concatenate(want)
+            got = host(ops.maps_attention(dev(np.concatenate(qs), torch.bfloat16), unit.k_pool, unit.v_pool, table, ctx, 1, 0.2))
+            ops.gemm_tc_check(DEV)
+            assert got.shape == want.shape
+            assert np.abs(got - want).max() <= 0.02 * np.abs(want).max(), (counts, np.abs(got - want).max())
+            cache.close(slots)
+
+
 def standing_out(w, entry, T, width, seed, pairs):
     """Weights whose keys point where the queries of a token point, and inputs in which, for each (query, keys) of
     ``pairs``, the keys' tokens repeat the query's direction at another length: with sharp q and k that query's weight goes
@@ -364,7 +404,7 @@ def test_far_keys_the_first_tokens_and_page_borders(dim, vdim, dtype):
 @pytest.fixture(scope="module")
 def models(tmp_path_factory):
     out = {}
-    for name, cfgd, seed in (("mixed", th.MIXED, 23), ("ones", th.ONES, 22)):
+    for name, cfgd, seed in (("mixed", th.MIXED, 21), ("ones", th.ONES, 22)):
         w = th.draw_weights(cfgd, seed)
         out[name] = (th.write_folder(str(tmp_path_factory.mktemp(name)), cfgd, w), cfgd, w)
     return out
@@ -380,22 +420,20 @@ def test_model_whole_in_batches_in_portions_and_decoded(models, which, dtype):
     folder, cfgd, w = models[which]
     td = torch.float32 if dtype == "float32" else torch.bfloat16
     eng = Engine.from_folder(folder, dtype=dtype, max_tokens=2048, max_batch=4)
-    rng = np.random.default_rng(31)
-    seqs = [rng.integers(0, cfgd["vocab"], n).tolist() for n in (150, 1, 7, 66)]
-    refs = [pt.forward(cfgd, w, t, round16=td == torch.bfloat16) for t in seqs]
+    seqs, refs = zip(*(th.clear_choices(cfgd, w, n, 31 + n, round16=td == torch.bfloat16) for n in (150, 1, 7, 66)))
     alone = []
     for t, ref in zip(seqs, refs):                          # each alone, whole
         (s,) = eng.open_sequences(1)
         alone.append(all_rows(eng, s, t))
         eng.close_sequences([s])
-        assert close_rows(alone[-1], ref, td)
+        assert close(alone[-1], ref, td)
     # all in one batch of unequal lengths, in slots and pages that were used before: the same as alone
     slots = eng.open_sequences(4)
     out = host(eng.step([StepEntry(s, t, list(range(len(t)))) for s, t in zip(slots, seqs)]))
     eng.close_sequences(slots)
     off = 0
     for t, ref, one in zip(seqs, refs, alone):
-        assert close_rows(out[off:off + len(t)], ref, td)
+        assert close(out[off:off + len(t)], ref, td)
         if td == torch.float32:
             assert np.abs(out[off:off + len(t)] - one).max() <= FP32_TOL * np.abs(ref).max()
         off += len(t)
@@ -405,7 +443,7 @@ def test_model_whole_in_batches_in_portions_and_decoded(models, which, dtype):
     for n in (2, 3, 60, 2, 17, 64, 2):
         rows.append(all_rows(eng, s, seqs[0][at:at + n]))
         at += n
-    assert at == 150 and close_rows(np.concatenate(rows), refs[0], td)
+    assert at == 150 and close(np.concatenate(rows), refs[0], td)
     eng.close_sequences([s])
     # prompts cut at unequal places, then token by token together; the shorter ones end earlier and give their slots back
     cuts = [60, 1, 3, 8]
@@ -427,7 +465,7 @@ def test_model_whole_in_batches_in_portions_and_decoded(models, which, dtype):
         eng.close_sequences([slots[i] for i in done])
         live = [i for i in live if i not in done]
     for i, ref in enumerate(refs):
-        assert close_rows(np.stack(rows[i]), ref, td), i
+        assert close(np.stack(rows[i]), ref, td), i
     assert eng.cache.slots.n_free == eng.max_batch and eng.cache.free_pages() == [g.pool.n for g in eng.cache._groups]
 
 
@@ -475,13 +513,13 @@ def test_a_wide_model_with_many_rows(tmp_path):
     for t in tokens[600:]:
         rows.append(host(eng.step([StepEntry(s, [t], [0])]))[0])
     eng.close_sequences([s])
-    assert close_rows(np.stack(rows), ref, torch.bfloat16)
+    assert most_rows_close(np.stack(rows), ref)
     slots = eng.open_sequences(20)
     out = host(eng.step([StepEntry(s, tokens[i:i + 3], [2]) for i, s in enumerate(slots)]))
     out2 = host(eng.step([StepEntry(s, [tokens[i + 3]], [0]) for i, s in enumerate(slots)]))
     want = [pt.forward(cfgd, w, tokens[i:i + 4], round16=True) for i in range(20)]
-    assert close_rows(out, np.stack([r[2] for r in want]), torch.bfloat16)
-    assert close_rows(out2, np.stack([r[3] for r in want]), torch.bfloat16)
+    assert most_rows_close(out, np.stack([r[2] for r in want]))
+    assert most_rows_close(out2, np.stack([r[3] for r in want]))
 
 
 def test_the_position_table_bounds_every_sequence(models):

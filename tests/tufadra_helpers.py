@@ -82,6 +82,22 @@ def draw_weights(cfgd, seed=0, sharp=1.0):
     return {k: pt.round_bf16(v) for k, v in w.items()}
 
 
+def clear_choices(cfgd, w, n, seed, round16=False, margin=0.02):
+    """A random sequence of n tokens in which no router's choice is a close call (a token with one is drawn again), and the
+    plain implementation's logits: rounding then changes no choice, and every row can be held to a tolerance."""
+    rng = np.random.default_rng(seed)
+    tokens = rng.integers(0, cfgd["vocab"], n).tolist()
+    for _ in range(20 * n):
+        margins = []
+        logits = pt.forward(cfgd, w, tokens, round16, margins=margins)
+        close = np.nonzero(np.min(margins, axis=0) < margin)[0]
+        if not close.size:
+            return tokens, logits
+        for i in close:
+            tokens[i] = int(rng.integers(0, cfgd["vocab"]))
+    raise AssertionError("no sequence without close calls was found")
+
+
 def write_folder(path, cfgd, w):
     from questwend_b200.weights import write_safetensors
     os.makedirs(path, exist_ok=True)
