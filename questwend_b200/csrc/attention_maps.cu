@@ -20,6 +20,8 @@
 //                     takes the difference and the norm
 #include "common.cuh"
 
+#include <type_traits>
+
 #define QWB_MAPS_MAX_DIM 256
 #define QWB_MAPS_PAGE 64
 #define QWB_MAPS_MAX 2
@@ -97,8 +99,9 @@ __global__ void maps_prep_kernel(const float* __restrict__ qkv, const float* __r
 // prep with norms over whole projections: all H * maps * dim values of q (and all G * maps * dim of k) are divided by ONE
 // root mean square and multiplied by weights of that size, then turned as above; q is then multiplied by
 // 1 + t_coef * ln(floor((p + 1) / t_every) + 1), a factor that grows with the position p (t_coef 0: 1).
-// grid (T, 3): a block for a token's q, one for its k, one for its v.  FOURS: 4 values at a time (no rotation, all sizes
-// multiples of 4); a row of up to 16 values a thread then stays in registers between the sum and the result.
+// maps_row_prep_fours: a block per token, 4 values at a time, all of the token's values in registers between the sums and
+// the results (no rotation, all sizes multiples of 4, rows that fit); maps_row_prep: grid (T, 3), a block for a token's q,
+// one for its k, one for its v, value by value.
 // ---------------------------------------------------------------------------------
 template <typename T> __device__ __forceinline__ void maps_store4(T* dst, float4 v);
 template <> __device__ __forceinline__ void maps_store4<float>(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
@@ -107,7 +110,82 @@ template <> __device__ __forceinline__ void maps_store4<bf16>(bf16* dst, float4 
     *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 
-template <typename T, bool FOURS>
+// the factor on q at position p
+__device__ __forceinline__ float maps_q_factor(int p, float coef, float every) {
+    return coef == 0.f ? 1.f : 1.f + coef * logf((float)floor((double)(p + 1) / (double)every) + 1.f);
+}
+
+#define QWB_ROW_PREP_THREADS 256
+#define QWB_ROW_PREP_Q 4          // pieces of 4 values a thread holds of q ...
+#define QWB_ROW_PREP_KV 4         // ... and of k and v together
+// The qkv product runs right before this kernel, which may have been launched early: qkv is read past the read-only cache.
+template <typename T>
+__global__ void __launch_bounds__(QWB_ROW_PREP_THREADS)
+maps_row_prep_fours_kernel(const float* qkv, const float* __restrict__ bias, const float* __restrict__ qw, const float* __restrict__ kw,
+                           const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ page_table,
+                           int table_width, T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool, int H, int G, int kdim,
+                           int vdim, float eps, float t_coef, float t_every, int store_kv) {
+    pdl_launch_dependents();            // the trigger first: see qwb_launch_link
+    pdl_wait();
+    __shared__ float sums[2][QWB_ROW_PREP_THREADS / 32];
+    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+    const int nq4 = H * kdim / 4, nk4 = G * kdim / 4, nkv4 = nk4 + G * vdim / 4;
+    const float4* src = reinterpret_cast<const float4*>(qkv) + (size_t)t * (nq4 + nkv4);
+    const float4* bs = reinterpret_cast<const float4*>(bias);
+    auto load = [&](int i) {
+        float4 v = __ldcg(src + i);
+        if (bs) { const float4 b = bs[i]; v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+        return v;
+    };
+    // what the results need beside the values, on its way with them
+    const int p = tok_pos[t];
+    const size_t page = store_kv ? page_table[(size_t)tok_seq[t] * table_width + p / QWB_MAPS_PAGE] : 0;
+    auto square = [](float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+    float4 hq[QWB_ROW_PREP_Q], hkv[QWB_ROW_PREP_KV];
+    float ssq = 0.f, ssk = 0.f;
+#pragma unroll
+    for (int j = 0; j < QWB_ROW_PREP_Q; ++j) {
+        const int i = tid + j * nt;
+        if (i < nq4) { hq[j] = load(i); ssq += square(hq[j]); }
+    }
+#pragma unroll
+    for (int j = 0; j < QWB_ROW_PREP_KV; ++j) {
+        const int i = tid + j * nt;
+        if (store_kv && i < nkv4) { hkv[j] = load(nq4 + i); if (i < nk4) ssk += square(hkv[j]); }
+    }
+    const float factor = maps_q_factor(p, t_coef, t_every);
+    ssq = warp_sum(ssq);
+    ssk = warp_sum(ssk);
+    if ((tid & 31) == 0) { sums[0][tid >> 5] = ssq; sums[1][tid >> 5] = ssk; }
+    __syncthreads();
+    ssq = ssk = 0.f;
+    for (int w = 0; w < (nt >> 5); ++w) { ssq += sums[0][w]; ssk += sums[1][w]; }
+    const float mq = factor * (qw ? rsqrtf(ssq / (float)(4 * nq4) + eps) : 1.f);
+    const float mk = kw ? rsqrtf(ssk / (float)(4 * nk4) + eps) : 1.f;
+    auto times = [](float4 v, float m, const float* w, int i) {
+        float4 f = make_float4(m, m, m, m);
+        if (w) { const float4 a = reinterpret_cast<const float4*>(w)[i]; f.x *= a.x; f.y *= a.y; f.z *= a.z; f.w *= a.w; }
+        return make_float4(v.x * f.x, v.y * f.y, v.z * f.z, v.w * f.w);
+    };
+#pragma unroll
+    for (int j = 0; j < QWB_ROW_PREP_Q; ++j) {
+        const int i = tid + j * nt;
+        if (i < nq4) maps_store4<T>(q_out + ((size_t)t * nq4 + i) * 4, times(hq[j], mq, qw, i));
+    }
+    if (!store_kv) return;
+    const int row = p % QWB_MAPS_PAGE;
+#pragma unroll
+    for (int j = 0; j < QWB_ROW_PREP_KV; ++j) {
+        const int i = tid + j * nt;
+        if (i >= nkv4) continue;
+        const bool is_k = i < nk4;
+        const int c = 4 * (is_k ? i : i - nk4), per = is_k ? kdim : vdim, head = c / per;
+        T* dst = (is_k ? k_pool : v_pool) + ((page * G + head) * QWB_MAPS_PAGE + row) * (size_t)per + (c - head * per);
+        maps_store4<T>(dst, is_k ? times(hkv[j], mk, kw, i) : hkv[j]);
+    }
+}
+
+template <typename T>
 __global__ void __launch_bounds__(256)
 maps_row_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ qw,
                      const float* __restrict__ kw, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
@@ -133,56 +211,25 @@ maps_row_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
         dst = (part == 1 ? k_pool : v_pool) + (page * G * QWB_MAPS_PAGE + p % QWB_MAPS_PAGE) * (size_t)per;
         head_step = (size_t)QWB_MAPS_PAGE * per;
     }
-    float factor = 1.f;
-    if (part == 0 && t_coef != 0.f) factor = 1.f + t_coef * logf((float)floor((double)(p + 1) / (double)t_every) + 1.f);
-
-    if constexpr (FOURS) {
-        constexpr int KEEP = 4;
-        float4 held[KEEP];
-        auto load = [&](int i) {
-            float4 v = *reinterpret_cast<const float4*>(src + 4 * i);
-            if (bs) { const float4 b = *reinterpret_cast<const float4*>(bs + 4 * i); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
-            return v;
-        };
-        float ss = 0.f;
-#pragma unroll
-        for (int j = 0; j < KEEP; ++j) {
-            const int i = tid + j * nt;
-            held[j] = i < n / 4 ? load(i) : make_float4(0.f, 0.f, 0.f, 0.f);
-            ss += held[j].x * held[j].x + held[j].y * held[j].y + held[j].z * held[j].z + held[j].w * held[j].w;
+    const float factor = part == 0 ? maps_q_factor(p, t_coef, t_every) : 1.f;
+    float ss = 0.f;
+    for (int i = tid; i < n; i += nt) { const float v = src[i] + (bs ? bs[i] : 0.f); ss += v * v; }
+    float mul = 1.f;
+    if (w) mul = rsqrtf(block_sum(ss, scratch) / (float)n + eps);
+    auto normed = [&](int i) { return (src[i] + (bs ? bs[i] : 0.f)) * mul * (w ? w[i] : 1.f); };
+    const int rd = part < 2 ? rdims : 0;
+    const float* cs = cos_t + (size_t)t * (rd >> 1);
+    const float* sn = sin_t + (size_t)t * (rd >> 1);
+    for (int i = tid; i < n; i += nt) {
+        const int head = i / per, in_map = part == 2 ? i - head * per : (i - head * per) % dim;
+        float v = normed(i);
+        if (in_map < rd) {
+            const int m = interleaved ? in_map >> 1 : (in_map < rd / 2 ? in_map : in_map - rd / 2);
+            const bool first = interleaved ? !(in_map & 1) : in_map < rd / 2;
+            const int other = interleaved ? (first ? i + 1 : i - 1) : (first ? i + rd / 2 : i - rd / 2);
+            v = first ? v * cs[m] - normed(other) * sn[m] : v * cs[m] + normed(other) * sn[m];
         }
-        for (int i = tid + KEEP * nt; i < n / 4; i += nt) { const float4 v = load(i); ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
-        float mul = factor;
-        if (w) mul *= rsqrtf(block_sum(ss, scratch) / (float)n + eps);
-        auto store = [&](int i, float4 v) {
-            float4 f = make_float4(mul, mul, mul, mul);
-            if (w) { const float4 a = *reinterpret_cast<const float4*>(w + 4 * i); f.x *= a.x; f.y *= a.y; f.z *= a.z; f.w *= a.w; }
-            const int head = 4 * i / per;
-            maps_store4<T>(dst + head * head_step + (4 * i - head * per), make_float4(v.x * f.x, v.y * f.y, v.z * f.z, v.w * f.w));
-        };
-#pragma unroll
-        for (int j = 0; j < KEEP; ++j) { const int i = tid + j * nt; if (i < n / 4) store(i, held[j]); }
-        for (int i = tid + KEEP * nt; i < n / 4; i += nt) store(i, load(i));
-    } else {
-        float ss = 0.f;
-        for (int i = tid; i < n; i += nt) { const float v = src[i] + (bs ? bs[i] : 0.f); ss += v * v; }
-        float mul = 1.f;
-        if (w) mul = rsqrtf(block_sum(ss, scratch) / (float)n + eps);
-        auto normed = [&](int i) { return (src[i] + (bs ? bs[i] : 0.f)) * mul * (w ? w[i] : 1.f); };
-        const int rd = part < 2 ? rdims : 0;
-        const float* cs = cos_t + (size_t)t * (rd >> 1);
-        const float* sn = sin_t + (size_t)t * (rd >> 1);
-        for (int i = tid; i < n; i += nt) {
-            const int head = i / per, in_map = part == 2 ? i - head * per : (i - head * per) % dim;
-            float v = normed(i);
-            if (in_map < rd) {
-                const int m = interleaved ? in_map >> 1 : (in_map < rd / 2 ? in_map : in_map - rd / 2);
-                const bool first = interleaved ? !(in_map & 1) : in_map < rd / 2;
-                const int other = interleaved ? (first ? i + 1 : i - 1) : (first ? i + rd / 2 : i - rd / 2);
-                v = first ? v * cs[m] - normed(other) * sn[m] : v * cs[m] + normed(other) * sn[m];
-            }
-            dst[head * head_step + (i - head * per)] = from_f32<T>(v * factor);
-        }
+        dst[head * head_step + (i - head * per)] = from_f32<T>(v * factor);
     }
 }
 
@@ -225,21 +272,23 @@ extern "C" int qwb_maps_row_prep(const float* qkv, const float* bias, const floa
     if (rdims < 0 || rdims > dim || rdims % 2) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a rotation of %d of %d values", rdims, dim);
     if (rdims > 0 && (!cos_t || !sin_t)) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a rotation without its table");
     if (t_coef != 0.f && !(t_every > 0.f)) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a query factor in steps of %g positions", t_every);
-    const bool fours = rdims == 0 && dim % 4 == 0 && vdim % 4 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 &&
+    const int nq = H * maps * dim, nkv = G * (maps * dim + vdim);
+    const bool fours = rdims == 0 && (maps * dim) % 4 == 0 && vdim % 4 == 0 && nq <= 4 * QWB_ROW_PREP_THREADS * QWB_ROW_PREP_Q &&
+                       nkv <= 4 * QWB_ROW_PREP_THREADS * QWB_ROW_PREP_KV && (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 &&
                        (uintptr_t)qw % 16 == 0 && (uintptr_t)kw % 16 == 0;
-    const int widest = H * maps * dim;
-    const dim3 grid(T, 3), block(widest >= 1024 ? 256 : 128);
-    auto go = [&](auto kernel, auto* q, auto* k, auto* v) {
-        qwb_launch(kernel, grid, block, 0, stream, qkv, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos, page_table, table_width, q, k, v, H, G, maps,
-                   dim, vdim, rdims, interleaved, eps, t_coef, t_every, store_kv);
+    auto go = [&](auto* q, auto* k, auto* v) {
+        using E = std::remove_pointer_t<decltype(q)>;
+        if (fours)      // as many threads as two pieces each of q and of k and v want, if that is fewer
+            qwb_launch_link(T, QWB_LINK_ROWS_NORM, maps_row_prep_fours_kernel<E>, dim3(T),
+                            dim3(nq <= 4 * 128 * QWB_ROW_PREP_Q / 2 && nkv <= 4 * 128 * QWB_ROW_PREP_KV / 2 ? 128 : QWB_ROW_PREP_THREADS), 0, stream,
+                            qkv, bias, qw, kw, tok_seq, tok_pos, page_table, table_width, q, k, v, H, G, maps * dim, vdim, eps, t_coef, t_every, store_kv);
+        else
+            qwb_launch(maps_row_prep_kernel<E>, dim3(T, 3), dim3(nq >= 1024 ? 256 : 128), 0, stream, qkv, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos,
+                       page_table, table_width, q, k, v, H, G, maps, dim, vdim, rdims, interleaved, eps, t_coef, t_every, store_kv);
     };
-    if (dtype == QWB_DT_F32) {
-        if (fours) go(maps_row_prep_kernel<float, true>, (float*)q_out, (float*)k_pool, (float*)v_pool);
-        else go(maps_row_prep_kernel<float, false>, (float*)q_out, (float*)k_pool, (float*)v_pool);
-    } else if (dtype == QWB_DT_BF16) {
-        if (fours) go(maps_row_prep_kernel<bf16, true>, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool);
-        else go(maps_row_prep_kernel<bf16, false>, (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool);
-    } else return qwb_fail(QWB_ERR_ARG, "maps_row_prep: unknown dtype %d", dtype);
+    if (dtype == QWB_DT_F32) go((float*)q_out, (float*)k_pool, (float*)v_pool);
+    else if (dtype == QWB_DT_BF16) go((bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool);
+    else return qwb_fail(QWB_ERR_ARG, "maps_row_prep: unknown dtype %d", dtype);
     return qwb_check_launch("maps_row_prep");
 }
 

@@ -695,6 +695,22 @@ __global__ void bias_act_kernel(const float* x, int ld, const float* __restrict_
     }
 }
 
+// The same for whole rows (ld = F) with F a multiple of 4: four values a thread and step.
+template <typename TOut>
+__global__ void bias_act_fours_kernel(const float4* x, const float4* __restrict__ bias, TOut* out, unsigned n4, unsigned f4, int act,
+                                      const float* __restrict__ params) {
+    pdl_wait();
+    pdl_launch_dependents();
+    float up = 0.f, down = 0.f;
+    if (act == 4) { up = softplus32(params[0]); down = 0.5f + softplus32(params[1]); }
+    auto f = [&](float v) { return act == 4 ? (v > 0.f ? up * v * v + 0.5f * v : down * (expm1f(v) - v) + 0.5f * v) : qwb_activate(v, act); };
+    for (unsigned i = blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += gridDim.x * blockDim.x) {
+        float4 v = x[i];
+        if (bias) { const float4 b = bias[i % f4]; v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+        Pack4<TOut>::store(out + (size_t)i * 4, f(v.x), f(v.y), f(v.z), f(v.w));
+    }
+}
+
 extern "C" int qwb_bias_act(const float* x, int ld, const float* bias, void* out, int out_dtype, int T, int F, int act,
                             const float* params, cudaStream_t stream) {
     if (T <= 0 || F <= 0) return 0;
@@ -703,6 +719,16 @@ extern "C" int qwb_bias_act(const float* x, int ld, const float* bias, void* out
     if (act == 4 && !params) return qwb_fail(QWB_ERR_ARG, "bias_act: this activation needs its two numbers");
     const size_t n = (size_t)T * F;
     const int block = 256;
+    if (ld == F && F % 4 == 0 && n / 4 < (1u << 30) && (uintptr_t)x % 16 == 0 && (uintptr_t)bias % 16 == 0 && (uintptr_t)out % 16 == 0) {
+        const unsigned n4 = (unsigned)(n / 4);
+        const int g4 = (int)((n4 + block - 1) / block < 148 * 32 ? (n4 + block - 1) / block : 148 * 32);
+        if (out_dtype == QWB_DT_F32)
+            qwb_launch(bias_act_fours_kernel<float>, g4, block, 0, stream, (const float4*)x, (const float4*)bias, (float*)out, n4, (unsigned)(F / 4), act, params);
+        else if (out_dtype == QWB_DT_BF16)
+            qwb_launch(bias_act_fours_kernel<bf16>, g4, block, 0, stream, (const float4*)x, (const float4*)bias, (bf16*)out, n4, (unsigned)(F / 4), act, params);
+        else return qwb_fail(QWB_ERR_ARG, "bias_act: unknown dtype %d", out_dtype);
+        return qwb_check_launch("bias_act");
+    }
     const int grid = (int)((n + block - 1) / block < 148 * 16 ? (n + block - 1) / block : 148 * 16);
     if (out_dtype == QWB_DT_F32) qwb_launch(bias_act_kernel<float>, grid, block, 0, stream, x, ld, bias, (float*)out, n, F, act, params);
     else if (out_dtype == QWB_DT_BF16) qwb_launch(bias_act_kernel<bf16>, grid, block, 0, stream, x, ld, bias, (bf16*)out, n, F, act, params);

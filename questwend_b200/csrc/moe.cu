@@ -26,86 +26,86 @@
 //   weight    score of a chosen expert, / (their sum + sum_eps) if `renorm`, * weight_scale
 //   gate_out  1 / (1 + exp(-z[E]))
 // ---------------------------------------------------------------------------------
-__global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int* __restrict__ chosen,
+// The choice works on keys, the scores' bits in an order that unsigned integers keep; 0 (below every number's key) is out.
+__device__ __forceinline__ unsigned order_key(float v) {
+    const unsigned b = __float_as_uint(v);
+    return b ^ ((b >> 31) ? 0xffffffffu : 0x80000000u);
+}
+// The place of the largest of n keys in shared memory (the lowest of equal ones), which is then out; the whole warp calls.
+__device__ __forceinline__ int take_best(unsigned* key, int n, int lane) {
+    unsigned best = 0;
+    int at = n;
+    for (int e = lane; e < n; e += 32) {
+        const unsigned v = key[e];
+        if (v > best || at == n) { best = v; at = e; }
+    }
+    const unsigned top = __reduce_max_sync(0xffffffffu, best);
+    const int first = (int)__reduce_min_sync(0xffffffffu, best == top && at < n ? (unsigned)at : 0x7fffffffu);
+    if (lane == 0) key[first] = 0;
+    __syncwarp();
+    return first;
+}
+
+__global__ void moe_route_kernel(const float* logits, int ld, const float* __restrict__ correction, int* __restrict__ chosen,
                                  float* __restrict__ weight, float* __restrict__ gate_out, int T, int E, int top, int sigmoid,
                                  int groups, int keep, int renorm, float sum_eps, float weight_scale) {
+    pdl_launch_dependents();            // the trigger first: see qwb_launch_link
     pdl_wait();
-    pdl_launch_dependents();
-    extern __shared__ float route_smem[];
+    extern __shared__ unsigned route_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= T) return;
-    float* choice = route_smem + warp * (E + groups);       // [E], then the groups' scores [groups]
-    float* gscore = choice + E;
+    unsigned* key = route_smem + warp * (2 * E + groups);   // [E] keys of the choice scores
+    float* score = reinterpret_cast<float*>(key + E);       // [E]
+    unsigned* gkey = key + 2 * E;                           // [groups]
     const float* z = logits + (size_t)t * ld;
-    const unsigned full = 0xffffffffu;
     float mx = 0.f, sum = 1.f;
     if (!sigmoid) {
         mx = -INFINITY;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, __ldcg(z + e));
         mx = warp_max(mx);
         sum = 0.f;
-        for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+        for (int e = lane; e < E; e += 32) sum += expf(__ldcg(z + e) - mx);
         sum = warp_sum(sum);
     }
-    auto score_of = [&](float v) { return sigmoid ? 1.f / (1.f + expf(-v)) : expf(v - mx) / sum; };
     const bool by_logit = !sigmoid && !correction && groups == 1;       // a softmax keeps the logits' order
-    for (int e = lane; e < E; e += 32) choice[e] = by_logit ? z[e] : score_of(z[e]) + (correction ? correction[e] : 0.f);
+    for (int e = lane; e < E; e += 32) {
+        const float v = __ldcg(z + e);
+        const float s = sigmoid ? 1.f / (1.f + expf(-v)) : expf(v - mx) / sum;
+        score[e] = s;
+        key[e] = order_key(by_logit ? v : s + (correction ? correction[e] : 0.f));
+    }
     __syncwarp();
-    // the largest of n values in shared memory (ties to the lower index), marked as taken
-    auto take_best = [&](float* v, int n) {
-        float best = -INFINITY;
-        int at = n;
-        for (int e = lane; e < n; e += 32)
-            if (v[e] > best) { best = v[e]; at = e; }
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(full, best, o);
-            const int oa = __shfl_xor_sync(full, at, o);
-            if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-        }
-        __syncwarp();
-        if (lane == 0 && at < n) v[at] = -INFINITY;
-        __syncwarp();
-        return at;
-    };
     if (keep < groups) {
         const int size = E / groups;
+        auto value = [&](int e) { const unsigned k = key[e]; return __uint_as_float((k >> 31) ? k ^ 0x80000000u : ~k); };
         for (int g = lane; g < groups; g += 32) {
-            float a = -INFINITY, b = -INFINITY;             // the two largest
-            for (int e = g * size; e < (g + 1) * size; ++e) {
-                const float c = choice[e];
-                if (c > a) { b = a; a = c; }
-                else if (c > b) b = c;
+            float a = value(g * size), b = -INFINITY;       // the two largest
+            for (int e = g * size + 1; e < (g + 1) * size; ++e) {
+                const float c = value(e);
+                b = fmaxf(b, fminf(a, c));
+                a = fmaxf(a, c);
             }
-            gscore[g] = size > 1 ? a + b : a;
+            gkey[g] = order_key(size > 1 ? a + b : a);
         }
         __syncwarp();
-        for (int k = 0; k < keep; ++k) take_best(gscore, groups);
+        for (int k = 0; k < keep; ++k) take_best(gkey, groups, lane);
         for (int e = lane; e < E; e += 32)
-            if (gscore[e / size] != -INFINITY) choice[e] = -INFINITY;       // a group that was not taken
+            if (gkey[e / size]) key[e] = 0;                 // of a group that was not taken
         __syncwarp();
     }
-    int picked[QWB_MOE_MAX_TOP];
-    float score[QWB_MOE_MAX_TOP];
-    float total = 0.f;
-#pragma unroll
-    for (int k = 0; k < QWB_MOE_MAX_TOP; ++k) {
-        if (k >= top) break;
-        const int at = take_best(choice, E);
-        picked[k] = at < E ? at : k;                        // nothing comparable left (not-a-number logits): a valid index
-        score[k] = score_of(z[picked[k]]);
-        total += score[k];
+    int mine = 0;                                           // lane k's choice
+    for (int k = 0; k < top; ++k) {
+        const int at = take_best(key, E, lane);
+        if (lane == k) mine = at;
     }
-    if (lane == 0) {
-        const float mul = weight_scale;
-#pragma unroll
-        for (int k = 0; k < QWB_MOE_MAX_TOP; ++k) {
-            if (k >= top) break;
-            chosen[(size_t)t * top + k] = picked[k];
-            weight[(size_t)t * top + k] = (renorm ? score[k] / (total + sum_eps) : score[k]) * mul;
-        }
-        if (gate_out) gate_out[t] = 1.f / (1.f + expf(-z[E]));
+    const float s = lane < top ? score[mine] : 0.f;
+    const float total = warp_sum(s);
+    if (lane < top) {
+        chosen[(size_t)t * top + lane] = mine;
+        weight[(size_t)t * top + lane] = (renorm ? s / (total + sum_eps) : s) * weight_scale;
     }
+    if (gate_out && lane == 31) gate_out[t] = 1.f / (1.f + expf(-__ldcg(z + E)));
 }
 
 extern "C" int qwb_moe_route(const float* logits, int ld, const float* correction, int* chosen, float* weight, float* gate_out, int T,
@@ -118,8 +118,8 @@ extern "C" int qwb_moe_route(const float* logits, int ld, const float* correctio
         return qwb_fail(QWB_ERR_ARG, "moe_route: %d of %d experts from %d of %d groups", top, E, keep, groups);
     if (ld < E + (gate_out ? 1 : 0)) return qwb_fail(QWB_ERR_ARG, "moe_route: rows of %d logits for %d experts", ld, E);
     const int warps = T >= 592 ? 4 : 1;                     // few tokens: a block each, side by side on the SMs
-    const size_t smem = (size_t)warps * (E + groups) * sizeof(float);       // at most 32 KB
-    qwb_launch(moe_route_kernel, (T + warps - 1) / warps, 32 * warps, smem, stream, logits, ld, correction, chosen, weight, gate_out, T, E, top,
+    const size_t smem = (size_t)warps * (2 * E + groups) * sizeof(float);   // at most 48 KB
+    qwb_launch_link(T, QWB_LINK_ROWS_NORM, moe_route_kernel, (T + warps - 1) / warps, 32 * warps, smem, stream, logits, ld, correction, chosen, weight, gate_out, T, E, top,
                sigmoid, groups, keep, renorm, sum_eps, weight_scale);
     return qwb_check_launch("moe_route");
 }
@@ -281,69 +281,57 @@ extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, co
 //   moe_act       act[s, f] = f(u[s, f]), u [S, F], or silu(u[s, f]) * u[s, F + f], u [S, 2F]
 //   moe_combine   out[t, :] (+)= sum_k weight[t, k] * y[place[t, k], :] + gate[t] * shared[t, :]
 // ---------------------------------------------------------------------------------
-// One block; each warp counts and then places a run of neighbouring copies, 32 at a time (lanes with the same expert find
-// their ranks by __match_any_sync), so that nothing depends on the order in which warps run.
-#define MOE_SORT_WARPS 32
+// A block per expert: it counts the copies of lower experts (where its own run starts) and ranks its own ones.  Each warp
+// walks over a run of neighbouring copies twice, 32 at a time (a ballot finds the ranks): once for its counts, then, knowing
+// what the warps before it counted, to write the places.  Nothing depends on the order in which warps or blocks run.
+#define MOE_SORT_WARPS 16
+#define MOE_SORT_AHEAD 8          // groups of 32 whose loads are on their way together
 __global__ void __launch_bounds__(MOE_SORT_WARPS * 32)
 moe_sort_kernel(const int* __restrict__ chosen, int* __restrict__ place, int* __restrict__ ends, int S, int E) {
     pdl_wait();
     pdl_launch_dependents();
-    extern __shared__ int sort_smem[];
-    int* hist = sort_smem;                              // [warps][E]: counts, then the next row of each (warp, expert)
-    int* base = hist + MOE_SORT_WARPS * E;              // [E]
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const unsigned full = 0xffffffffu;
-    for (int i = threadIdx.x; i < MOE_SORT_WARPS * E; i += blockDim.x) hist[i] = 0;
-    __syncthreads();
+    __shared__ int own[MOE_SORT_WARPS], lower[MOE_SORT_WARPS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, expert = blockIdx.x;
+    const unsigned full = 0xffffffffu, before = (1u << lane) - 1u;
     const int per = ((S + MOE_SORT_WARPS - 1) / MOE_SORT_WARPS + 31) & ~31;
     const int lo = min(S, warp * per), hi = min(S, lo + per);
-    int* mine = hist + warp * E;
-    for (int i0 = lo; i0 < hi; i0 += 32) {
-        const int i = i0 + lane;
-        const int e = i < hi ? min(max(chosen[i], 0), E - 1) : -1;
-        const unsigned same = __match_any_sync(full, e);
-        if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
-        __syncwarp();
-    }
-    __syncthreads();
-    for (int e = threadIdx.x; e < E; e += blockDim.x) {
-        int run = 0;
-#pragma unroll 8
-        for (int w = 0; w < MOE_SORT_WARPS; ++w) { const int c = hist[w * E + e]; hist[w * E + e] = run; run += c; }
-        base[e] = run;
-    }
-    __syncthreads();
-    if (warp == 0) {
-        int run = 0;
-        for (int e0 = 0; e0 < E; e0 += 32) {
-            const int c = e0 + lane < E ? base[e0 + lane] : 0;
-            int s = c;
-            for (int o = 1; o < 32; o <<= 1) { const int up = __shfl_up_sync(full, s, o); if (lane >= o) s += up; }
-            if (e0 + lane < E) { base[e0 + lane] = run + s - c; ends[e0 + lane] = run + s; }
-            run += __shfl_sync(full, s, 31);
+    auto expert_of = [&](int i) { return i < hi ? min(max(chosen[i], 0), E - 1) : E; };        // E: not a copy
+    int n_own = 0, n_lower = 0;
+    for (int i0 = lo; i0 < hi; i0 += 32 * MOE_SORT_AHEAD) {
+        int es[MOE_SORT_AHEAD];
+#pragma unroll
+        for (int a = 0; a < MOE_SORT_AHEAD; ++a) es[a] = expert_of(i0 + 32 * a + lane);
+#pragma unroll
+        for (int a = 0; a < MOE_SORT_AHEAD; ++a) {
+            n_own += __popc(__ballot_sync(full, es[a] == expert));
+            n_lower += __popc(__ballot_sync(full, es[a] < expert));
         }
     }
+    if (lane == 0) { own[warp] = n_own; lower[warp] = n_lower; }
     __syncthreads();
-    for (int i0 = lo; i0 < hi; i0 += 32) {
-        const int i = i0 + lane;
-        const int e = i < hi ? min(max(chosen[i], 0), E - 1) : -1;
-        const unsigned same = __match_any_sync(full, e);
-        if (e >= 0) place[i] = base[e] + mine[e] + __popc(same & ((1u << lane) - 1u));
-        __syncwarp();
-        if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
-        __syncwarp();
+    int at = 0, total = 0;                              // the next row of this warp's copies; where the run ends
+    for (int w = 0; w < MOE_SORT_WARPS; ++w) {
+        at += lower[w] + (w < warp ? own[w] : 0);
+        total += lower[w] + own[w];
+    }
+    if (threadIdx.x == 0) ends[expert] = total;
+    for (int i0 = lo; i0 < hi && n_own > 0; i0 += 32 * MOE_SORT_AHEAD) {
+        int es[MOE_SORT_AHEAD];
+#pragma unroll
+        for (int a = 0; a < MOE_SORT_AHEAD; ++a) es[a] = expert_of(i0 + 32 * a + lane);
+#pragma unroll
+        for (int a = 0; a < MOE_SORT_AHEAD; ++a) {
+            const unsigned mine = __ballot_sync(full, es[a] == expert);
+            if (es[a] == expert) place[i0 + 32 * a + lane] = at + __popc(mine & before);
+            at += __popc(mine);
+        }
     }
 }
 
 extern "C" int qwb_moe_sort(const int* chosen, int* place, int* ends, int S, int E, cudaStream_t stream) {
     if (S <= 0) return 0;
     if (E <= 0 || E > QWB_MOE_MAX_EXPERTS) return qwb_fail(QWB_ERR_ARG, "moe_sort: %d experts (at most %d)", E, QWB_MOE_MAX_EXPERTS);
-    const size_t smem = (size_t)(MOE_SORT_WARPS + 1) * E * sizeof(int);
-    if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(moe_sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "moe_sort: %s", cudaGetErrorString(e));
-    }
-    qwb_launch(moe_sort_kernel, 1, MOE_SORT_WARPS * 32, smem, stream, chosen, place, ends, S, E);
+    qwb_launch(moe_sort_kernel, E, MOE_SORT_WARPS * 32, 0, stream, chosen, place, ends, S, E);
     return qwb_check_launch("moe_sort");
 }
 
@@ -375,33 +363,41 @@ __device__ __forceinline__ uint4 pack_bf16x8(const float* v) {
     return o;
 }
 
-// grid (S, ...): a block per row; 8 values a thread
-__global__ void moe_act_kernel(const Vec16<bf16>* __restrict__ u, uint4* __restrict__ act, int pieces, int kind) {
+// 8 values a thread and step, whatever row they are in; KIND: the activation code
+template <int KIND>
+__global__ void moe_act_kernel(const Vec16<bf16>* __restrict__ u, uint4* __restrict__ act, unsigned n, unsigned pieces) {
     pdl_wait();
     pdl_launch_dependents();
-    const size_t s = blockIdx.x;
-    const bool gated = kind == QWB_MOE_GATED;
-    const Vec16<bf16>* row = u + s * (gated ? 2 * pieces : pieces);
-    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+    for (unsigned i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
         float a[8], b[8];
-        row[i].get(a);
-        if (gated) {
-            row[pieces + i].get(b);
+        if (KIND == QWB_MOE_GATED) {
+            const size_t gate = i + (size_t)(i / pieces) * pieces;          // row s: its gate pieces, then its up pieces
+            u[gate].get(a);
+            u[gate + pieces].get(b);
 #pragma unroll
             for (int e = 0; e < 8; ++e) a[e] = a[e] / (1.f + expf(-a[e])) * b[e];
         } else {
+            u[i].get(a);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) a[e] = qwb_activate(a[e], kind);
+            for (int e = 0; e < 8; ++e) a[e] = qwb_activate(a[e], KIND);
         }
-        act[s * pieces + i] = pack_bf16x8(a);
+        act[i] = pack_bf16x8(a);
     }
 }
 
 extern "C" int qwb_moe_act(const void* u, void* act, int S, int F, int kind, cudaStream_t stream) {
     if (S <= 0 || F <= 0) return 0;
     if (F % 8) return qwb_fail(QWB_ERR_ARG, "moe_act: rows of %d values", F);
-    if (kind != QWB_MOE_GATED && !qwb_activation_known(kind)) return qwb_fail(QWB_ERR_ARG, "moe_act: unknown activation %d", kind);
-    qwb_launch(moe_act_kernel, S, F >= 2048 ? 256 : 128, 0, stream, (const Vec16<bf16>*)u, (uint4*)act, F / 8, kind);
+    const long long n = (long long)S * (F / 8);
+    if (n >= 1LL << 31) return qwb_fail(QWB_ERR_ARG, "moe_act: %d rows of %d values are too many for one launch", S, F);
+    const int grid = (int)((n + 255) / 256 < 148 * 32 ? (n + 255) / 256 : 148 * 32);
+#define QWB_MOE_ACT(KIND) \
+    case KIND: qwb_launch(moe_act_kernel<KIND>, grid, 256, 0, stream, (const Vec16<bf16>*)u, (uint4*)act, (unsigned)n, (unsigned)(F / 8)); break
+    switch (kind) {
+        QWB_MOE_ACT(0); QWB_MOE_ACT(1); QWB_MOE_ACT(2); QWB_MOE_ACT(3); QWB_MOE_ACT(5); QWB_MOE_ACT(QWB_MOE_GATED);
+        default: return qwb_fail(QWB_ERR_ARG, "moe_act: unknown activation %d", kind);
+    }
+#undef QWB_MOE_ACT
     return qwb_check_launch("moe_act");
 }
 
