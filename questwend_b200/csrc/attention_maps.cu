@@ -112,7 +112,10 @@ template <> __device__ __forceinline__ void maps_store4<bf16>(bf16* dst, float4 
 
 // the factor on q at position p
 __device__ __forceinline__ float maps_q_factor(int p, float coef, float every) {
-    return coef == 0.f ? 1.f : 1.f + coef * logf((float)floor((double)(p + 1) / (double)every) + 1.f);
+    if (coef == 0.f) return 1.f;
+    const int whole = (int)fminf(every, 1e9f);              // steps of a whole number of positions need no 64-bit division
+    const float n = whole > 0 && (float)whole == every ? (float)((p + 1) / whole) : (float)floor((double)(p + 1) / (double)every);
+    return 1.f + coef * logf(n + 1.f);
 }
 
 #define QWB_ROW_PREP_THREADS 256

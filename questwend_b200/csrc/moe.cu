@@ -16,6 +16,7 @@
 
 #define QWB_MOE_MAX_TOP 16
 #define QWB_MOE_MAX_EXPERTS 1024
+#define MOE_UP_BLOCKS 5         // blocks of moe_up an SM by registers: more loads on their way beat a few spills in the shared expert's part
 #define QWB_MOE_GATED 16        // activation code of the gated form, silu(gate) * up; others: qwb_activate's codes
 
 // ---------------------------------------------------------------------------------
@@ -167,19 +168,20 @@ __device__ __forceinline__ void lane_dots(const T* __restrict__ w, size_t ldw, i
     }
 }
 
-// grid (ceil(rows / 8), T * top + ceil(T / NT)): the copies of the tokens, then the shared expert with NT tokens a warp.
+// Blocks: per copy of a token (T * top) as many as its expert's features take, 8 warps each, then the shared expert's, with
+// NT tokens a warp.
 // A warp makes two features of a plain expert, one of a gated one (its gate and its up row), two of the shared expert.
 template <typename T, int NT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, MOE_UP_BLOCKS)
 moe_up_kernel(const T* __restrict__ x, const T* __restrict__ wu, const int* __restrict__ chosen, T* __restrict__ act,
               const T* __restrict__ wsu, T* __restrict__ act_s, int n_tok, int D, int F, int Fs, int top, int kind) {
     pdl_wait();
     pdl_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int slot = blockIdx.y, n_slots = n_tok * top;
-    const int item = blockIdx.x * 8 + warp;
-    if (slot < n_slots) {
-        const bool gated = kind == QWB_MOE_GATED;
+    const bool gated = kind == QWB_MOE_GATED;
+    const int per_slot = ((gated ? F : (F + 1) / 2) + 7) / 8, n_routed = n_tok * top * per_slot;
+    if ((int)blockIdx.x < n_routed) {
+        const int slot = blockIdx.x / per_slot, item = (blockIdx.x - slot * per_slot) * 8 + warp;
         const int f = gated ? item : 2 * item;
         if (f >= F) return;
         const size_t first = (size_t)chosen[slot] * (gated ? 2 * F : F) + f;
@@ -191,7 +193,8 @@ moe_up_kernel(const T* __restrict__ x, const T* __restrict__ wu, const int* __re
         if (gated) { if (lane == 0) o[0] = from_f32<T>(a / (1.f + expf(-a)) * b); }
         else if (lane < min(2, F - f)) o[lane] = from_f32<T>(qwb_activate(lane ? b : a, kind));
     } else {
-        const int t0 = (slot - n_slots) * NT, f = 2 * item;
+        const int per_group = ((Fs + 1) / 2 + 7) / 8, group = (blockIdx.x - n_routed) / per_group;
+        const int t0 = group * NT, f = 2 * ((blockIdx.x - n_routed - group * per_group) * 8 + warp);
         if (f >= Fs) return;
         const int nt = min(NT, n_tok - t0), nf = min(2, Fs - f);
         float acc[2 * NT];
@@ -244,14 +247,13 @@ template <typename T>
 static void launch_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight, const void* wsu,
                                const void* wsd, const float* gate, void* act, void* act_s, float* out, int n_tok, int D, int F, int Fs,
                                int top, int kind, int onto, cudaStream_t stream) {
-    const int items = kind == QWB_MOE_GATED ? F : (F + 1) / 2, items_s = Fs > 0 ? (Fs + 1) / 2 : 0;
-    const int rows = items > items_s ? items : items_s;
-    const int nt = n_tok > 1 ? 4 : 1;
-    const dim3 g1((rows + 7) / 8, n_tok * top + (Fs > 0 ? (n_tok + nt - 1) / nt : 0)), g2((D + 3) / 4, n_tok);
+    const int per_slot = ((kind == QWB_MOE_GATED ? F : (F + 1) / 2) + 7) / 8, per_group = Fs > 0 ? ((Fs + 1) / 2 + 7) / 8 : 0;
+    const int nt = n_tok > 1 ? 2 : 1;
+    const dim3 g1(n_tok * top * per_slot + (n_tok + nt - 1) / nt * per_group), g2((D + 3) / 4, n_tok);
     if (nt == 1)
         qwb_launch(moe_up_kernel<T, 1>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
     else
-        qwb_launch(moe_up_kernel<T, 4>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
+        qwb_launch(moe_up_kernel<T, 2>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
     qwb_launch(moe_down_kernel<T, 4>, g2, 32 * (top + (Fs > 0 ? 1 : 0)), 0, stream, (const T*)act, (const T*)wd, chosen, weight, (const T*)act_s,
                (const T*)wsd, gate, out, D, F, Fs, top, onto);
 }
@@ -265,7 +267,8 @@ extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, co
         return qwb_fail(QWB_ERR_ARG, "moe_experts: width %d, expert width %d, shared %d, %d choices", D, F, Fs, top);
     if (Fs > 0 && (!wsu || !wsd || !act_s)) return qwb_fail(QWB_ERR_ARG, "moe_experts: a shared expert without its matrices");
     if (kind != QWB_MOE_GATED && !qwb_activation_known(kind)) return qwb_fail(QWB_ERR_ARG, "moe_experts: unknown activation %d", kind);
-    if ((long long)T * top + T > 65535) return qwb_fail(QWB_ERR_ARG, "moe_experts: %d tokens x %d choices are too many for one launch", T, top);
+    if ((long long)T * top + T > 65535 || ((long long)T * top + T) * ((F > Fs ? F : Fs) / 8 + 1) > 0x7fffffffLL)
+        return qwb_fail(QWB_ERR_ARG, "moe_experts: %d tokens x %d choices are too many for one launch", T, top);
     if (dtype == QWB_DT_F32)
         launch_moe_experts<float>(x, wu, wd, chosen, weight, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
     else if (dtype == QWB_DT_BF16)

@@ -5,6 +5,7 @@
     python -m questwend_b200.kernels.microbench attn_prefill --tokens 2048
     python -m questwend_b200.kernels.microbench rmsnorm --m 8 --k 4096
     python -m questwend_b200.kernels.microbench sample --batch 8 --vocab 151936 --temp 0.8 --top-k 40 --top-p 0.95
+    python -m questwend_b200.kernels.microbench moe --m 8 --k 2048 --n 1408 --experts 64 --top-k 6 --shared 2816
     python -m questwend_b200.kernels.microbench decode_shapes --m 8        (every product of a Qwen3-8B decode step)
 
 Inputs rotate through enough copies to exceed the 126 MB L2, so every timed launch reads from HBM.
@@ -292,9 +293,35 @@ def bench_shaped_attention(B, tokens, ctx, Hq, Hkv, dim, softcap, window, extras
             "gb_s_of_visible_rows": (B * Hkv * (seen / tokens) * 2 * dim * q.element_size() / us / 1e3) if tokens == 1 else None}
 
 
+def bench_moe(T, D, F, E, top, shared, activation, iters, dtype=torch.bfloat16) -> dict:
+    """Routed experts of width ``F`` for ``T`` tokens of ``D`` values, each with ``top`` random experts out of ``E``, and a
+    shared expert of width ``shared`` (0: none): the expert-streaming kernels, or the sorted form where that fits."""
+    gated = activation == "gated_silu"
+    up = (0.02 * torch.randn(E, (2 if gated else 1) * F, D, device=DEV)).to(dtype)
+    down = (0.02 * torch.randn(E, D, F, device=DEV)).to(dtype)
+    s_up, s_down = ((0.02 * torch.randn(shared, D, device=DEV)).to(dtype), (0.02 * torch.randn(D, shared, device=DEV)).to(dtype)) if shared else (None, None)
+    x = torch.randn(T, D, device=DEV).to(dtype)
+    gate = torch.rand(T, device=DEV) if shared else None
+    # one choice for every copy of the inputs, so that the chosen experts do not stay in L2
+    routes = [ops.moe_route(torch.randn(T, E, device=DEV), top, True, scores="sigmoid") for _ in range(8)]
+    grouped = ops.moe_grouped_fits(x, up, down)
+    if grouped:
+        out = torch.zeros(T, D, device=DEV)
+        fn = lambda i: ops.moe_experts_grouped(x, up, down, *routes[i % 8], activation, shared=out if shared else None, gate=gate)
+    else:
+        fn = lambda i: ops.moe_experts(x, up, down, *routes[i % 8], activation, s_up, s_down, gate)
+    us = _time(fn, 8, iters)
+    used = statistics.mean(len(torch.unique(c)) for c, _ in routes)
+    per = (3 if gated else 2) * D * F
+    n_bytes = (used * per + 2 * D * shared) * x.element_size()
+    return {"what": "moe", "tokens": T, "width": D, "expert": F, "experts": E, "top": top, "shared": shared, "activation": activation,
+            "form": "grouped" if grouped else "streamed", "us": us, "experts_used": used, "bytes": n_bytes, "gb_s": n_bytes / us / 1e3,
+            "tflops": 2 * T * top * per / us / 1e6}
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "attn_decode", "attn_prefill", "rmsnorm", "rope", "decode_shapes", "sample", "pool_attn", "maps_attn", "shaped_attn"])
+    ap.add_argument("what", choices=["gemm", "attn_decode", "attn_prefill", "rmsnorm", "rope", "decode_shapes", "sample", "pool_attn", "maps_attn", "shaped_attn", "moe"])
     ap.add_argument("--m", type=int, default=8)
     ap.add_argument("--n", type=int, default=24576)
     ap.add_argument("--k", type=int, default=4096)
@@ -324,6 +351,9 @@ def main() -> int:
     ap.add_argument("--chunk", type=int, default=0, help="maps_attn: positions per chunk (0: plain causal)")
     ap.add_argument("--attn-impl", default="auto", choices=["auto", "tc", "mma", "plain"], help="maps_attn: the prompt kernel")
     ap.add_argument("--pool", type=int, default=16, help="pool_attn: tokens per pooled block")
+    ap.add_argument("--experts", type=int, default=64, help="moe: experts (--m tokens, --k their width, --n an expert's width, --top-k choices)")
+    ap.add_argument("--shared", type=int, default=0, help="moe: width of the shared expert (0: none)")
+    ap.add_argument("--activation", default="gelu", help="moe: the experts' activation ('gated_silu': gated experts)")
     ap.add_argument("--extras", default="", help="shaped_attn: words out of 'slopes sink temp mix gate'")
     args = ap.parse_args()
     dtype = torch.bfloat16 if args.dtype == "bfloat16" else torch.float32
@@ -349,6 +379,8 @@ def main() -> int:
         print(json.dumps(bench_shaped_attention(args.batch, args.tokens, args.ctx if args.tokens == 1 else 0, args.heads, args.kv_heads,
                                                 args.head_dim, args.softcap, args.window if "--window" in sys.argv else 0, args.extras,
                                                 args.iters, dtype, args.attn_impl)))
+    elif args.what == "moe":
+        print(json.dumps(bench_moe(args.m, args.k, args.n, args.experts, args.top_k, args.shared, args.activation, args.iters, dtype)))
     elif args.what == "sample":
         print(json.dumps(bench_sample(args.batch, args.vocab, args.temp, args.top_k, args.top_p, args.iters)))
     elif args.what == "attn_prefill":

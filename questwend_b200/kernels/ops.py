@@ -1277,7 +1277,7 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
     dim = kdim // maps
     out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
     width = page_table.shape[1]
-    one_map = (maps == 1 and softcap <= 0.0 and not norm_out and out_scale == 1.0 and impl in ("auto", "tc")
+    one_map = (maps == 1 and softcap <= 0.0 and not norm_out and impl in ("auto", "tc")
                and part_attention_fits(q.dtype, dim, vdim, k_pool.shape[2], H // G))
     if ctx.single_token and one_map and chunk == 0:
         return attn_decode(q, k_pool, v_pool, page_table, ctx.seq_len, scale, ctx.max_len, impl="mma")
