@@ -16,10 +16,11 @@
 //   q_rot[t, h, :] = the same rotation of q[t, h, K:]; q_plain[h, t, :] = q[t, h, :K] in the products' dtype
 //   or, for the tensor-core prompt kernel (q_full given): q_full[t, h, :] = [q[t, h, :K] | rotated part] and
 //   row_new[t, :] = the cache row again, token by token, both in the products' dtype
-// cos, sin [T, half] already hold any factor on them.
+// q and dkv are rows of ld_q and ld_dkv floats; a layer that reads another layer's rows has no dkv (null): only its queries
+// are prepared.  cos, sin [T, half] already hold any factor on them.
 // ---------------------------------------------------------------------------------
 template <typename T>
-__global__ void latent_prep_kernel(const float* __restrict__ q, const float* __restrict__ dkv, const float* __restrict__ c_weight,
+__global__ void latent_prep_kernel(const float* __restrict__ q, int ld_q, const float* __restrict__ dkv, int ld_dkv, const float* __restrict__ c_weight,
                                    const float* __restrict__ cosv, const float* __restrict__ sinv, const int* __restrict__ tok_seq,
                                    const int* __restrict__ tok_pos, const int* __restrict__ page_table, T* __restrict__ pool,
                                    T* __restrict__ q_plain, float* __restrict__ q_rot, T* __restrict__ q_full, T* __restrict__ row_new,
@@ -29,10 +30,10 @@ __global__ void latent_prep_kernel(const float* __restrict__ q, const float* __r
     pdl_launch_dependents();
     __shared__ float red[32];
     const int t = blockIdx.x;
-    const float* drow = dkv + (size_t)t * (L + R);
+    const float* drow = dkv + (size_t)t * ld_dkv;
     const float* cs = cosv + (size_t)t * half;
     const float* sn = sinv + (size_t)t * half;
-    if (store || row_new) {
+    if (dkv && (store || row_new)) {
         float ss = 0.f;
         for (int i = threadIdx.x; i < L; i += blockDim.x) ss += drow[i] * drow[i];
         const float scale = rsqrtf(block_sum(ss, red) / (float)L + eps);
@@ -54,7 +55,7 @@ __global__ void latent_prep_kernel(const float* __restrict__ q, const float* __r
             if (again) again[L + i] = from_f32<T>(v);
         }
     }
-    const float* qrow = q + (size_t)t * H * (K + R);
+    const float* qrow = q + (size_t)t * ld_q;
     if (q_full) {
         for (int idx = threadIdx.x; idx < H * (K + R); idx += blockDim.x) {
             const int h = idx / (K + R), i = idx - h * (K + R) - K;       // i >= 0: the rotated part
@@ -83,24 +84,52 @@ __global__ void latent_prep_kernel(const float* __restrict__ q, const float* __r
     }
 }
 
-extern "C" int qwb_latent_prep(const float* q, const float* dkv, const float* c_weight, const float* cosv, const float* sinv,
+extern "C" int qwb_latent_prep(const float* q, int ld_q, const float* dkv, int ld_dkv, const float* c_weight, const float* cosv, const float* sinv,
                                const int* tok_seq, const int* tok_pos, const int* page_table, void* pool, int dtype,
                                void* q_plain, float* q_rot, void* q_full, void* row_new, int T, int H, int K, int R, int L,
                                int half, float eps, int page_size, int table_width, int store, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || K <= 0 || R < 0 || L <= 0 || half < 0 || 2 * half > R)
         return qwb_fail(QWB_ERR_ARG, "latent_prep: %d heads of %d + %d, latent %d, %d rotated pairs", H, K, R, L, half);
+    if (ld_q < H * (K + R) || (dkv && ld_dkv < L + R)) return qwb_fail(QWB_ERR_ARG, "latent_prep: rows of %d and %d values", ld_q, ld_dkv);
     if (dtype == QWB_DT_F32)
-        qwb_launch(latent_prep_kernel<float>, T, 128, 0, stream, q, dkv, c_weight, cosv, sinv, tok_seq, tok_pos, page_table,
+        qwb_launch(latent_prep_kernel<float>, T, 128, 0, stream, q, ld_q, dkv, ld_dkv, c_weight, cosv, sinv, tok_seq, tok_pos, page_table,
                    (float*)pool, (float*)q_plain, q_rot, (float*)q_full, (float*)row_new, T, H, K, R, L, half, eps, page_size,
                    table_width, store);
     else if (dtype == QWB_DT_BF16)
-        qwb_launch(latent_prep_kernel<bf16>, T, 128, 0, stream, q, dkv, c_weight, cosv, sinv, tok_seq, tok_pos, page_table,
+        qwb_launch(latent_prep_kernel<bf16>, T, 128, 0, stream, q, ld_q, dkv, ld_dkv, c_weight, cosv, sinv, tok_seq, tok_pos, page_table,
                    (bf16*)pool, (bf16*)q_plain, q_rot, (bf16*)q_full, (bf16*)row_new, T, H, K, R, L, half, eps, page_size,
                    table_width, store);
     else
         return qwb_fail(QWB_ERR_ARG, "latent_prep: unknown dtype %d", dtype);
     return qwb_check_launch("latent_prep");
+}
+
+// The heads' outputs side by side for the output projection: out[t, h * P + p] = v[h, t, p], times the sigmoid of the gate's
+// column h of row t if there is one (gate: rows of ld_gate floats, or null).
+template <typename T>
+__global__ void latent_heads_out_kernel(const float* __restrict__ v, const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int n_tok,
+                                        int H, int P) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * P; i += gridDim.y * blockDim.x) {
+        const int h = i / P, p = i - h * P;
+        float x = v[((size_t)h * n_tok + t) * P + p];
+        if (gate) x *= 1.f / (1.f + expf(-gate[(size_t)t * ld_gate + h]));
+        out[(size_t)t * H * P + i] = from_f32<T>(x);
+    }
+}
+
+extern "C" int qwb_latent_heads_out(const float* v, const float* gate, int ld_gate, void* out, int dtype, int T, int H, int P, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || P <= 0 || (gate && ld_gate < H)) return qwb_fail(QWB_ERR_ARG, "latent_heads_out: %d heads of %d, gate rows of %d", H, P, ld_gate);
+    const int per_row = (H * P + 255) / 256;
+    const dim3 grid(T, T >= 148 ? 1 : (per_row < 32 ? per_row : 32));       // few tokens: a row over several blocks
+    if (dtype == QWB_DT_F32) qwb_launch(latent_heads_out_kernel<float>, grid, 256, 0, stream, v, gate, ld_gate, (float*)out, T, H, P);
+    else if (dtype == QWB_DT_BF16) qwb_launch(latent_heads_out_kernel<bf16>, grid, 256, 0, stream, v, gate, ld_gate, (bf16*)out, T, H, P);
+    else return qwb_fail(QWB_ERR_ARG, "latent_heads_out: unknown dtype %d", dtype);
+    return qwb_check_launch("latent_heads_out");
 }
 
 // ---------------------------------------------------------------------------------

@@ -5,7 +5,7 @@
 // over DQ = dim + rot_dim query/key values and DV value values: cheaper for many tokens than scoring against the
 // latents themselves (csrc/attention_latent.cu does that, for single tokens, continued prompts and the 32-bit engine).
 // Causal, optional window (key j visible from position p when p - window < j <= p), optional sink per head (one more
-// term exp(sink) in the denominator).  Scores, maxima, sums and the output accumulator are 32-bit; probabilities are
+// term exp(sink) in the denominator), optional gate per token and head (its sigmoid multiplies the head's output).  Scores, maxima, sums and the output accumulator are 32-bit; probabilities are
 // rounded to bfloat16 for the second product, as in every tensor-core attention.
 //
 // Block = 64 queries of one (sequence, head), 4 warps of 16 rows; keys in tiles of 64.  Q, K and V tiles sit in shared
@@ -48,7 +48,8 @@ template <int NV>       // n-tiles of 8 value columns the accumulator has room f
 __global__ void __launch_bounds__(128)
 latent_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_plain, const bf16* __restrict__ kr, int ld_kr,
                           const bf16* __restrict__ v, const int* __restrict__ cu_seqlens, const float* __restrict__ sink,
-                          bf16* __restrict__ out, int H, int K, int R, int DV, float scale, int window) {
+                          bf16* __restrict__ out, int H, int K, int R, int DV, float scale, int window, const float* __restrict__ gate,
+                          int ld_gate) {
     pdl_wait();
     pdl_launch_dependents();
     const int DQ = K + R;
@@ -186,7 +187,11 @@ latent_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
 #pragma unroll
         for (int j = 0; j < NV; ++j) { o[j][0] *= r0; o[j][1] *= r0; o[j][2] *= r1; o[j][3] *= r1; }
     }
-    const float inv0 = 1.f / l0, inv1 = 1.f / l1;
+    float inv0 = 1.f / l0, inv1 = 1.f / l1;
+    if (gate) {
+        if (row0 < n) inv0 /= 1.f + expf(-gate[(size_t)(t0 + row0) * ld_gate + h]);
+        if (row1 < n) inv1 /= 1.f + expf(-gate[(size_t)(t0 + row1) * ld_gate + h]);
+    }
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
         if (j < nv_used) {
@@ -199,7 +204,7 @@ latent_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
 
 extern "C" int qwb_latent_prefill_mma(const void* q, const void* k_plain, const void* kr, int ld_kr, const void* v,
                                       const int* cu_seqlens, const float* sink, void* out, int B, int max_new, int H, int K,
-                                      int R, int DV, float scale, int window, cudaStream_t stream) {
+                                      int R, int DV, float scale, int window, const float* gate, int ld_gate, cudaStream_t stream) {
     if (B <= 0 || max_new <= 0) return 0;
     if (H <= 0 || K <= 0 || R < 0 || DV <= 0 || K % 8 || R % 8 || DV % 8 || (K + R) % 16 || DV > 256 || ld_kr % 8)
         return qwb_fail(QWB_ERR_ARG, "latent_prefill_mma: heads %d of %d + %d and %d values: parts in multiples of 8, %d + %d a multiple "
@@ -217,7 +222,7 @@ extern "C" int qwb_latent_prefill_mma(const void* q, const void* k_plain, const 
             if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "latent_prefill_mma: %s", cudaGetErrorString(e));               \
         }                                                                                                                       \
         qwb_launch(latent_prefill_mma_kernel<NV>, grid, 128, smem, stream, (const bf16*)q, (const bf16*)k_plain, (const bf16*)kr, ld_kr, \
-                   (const bf16*)v, cu_seqlens, sink, (bf16*)out, H, K, R, DV, scale, window);                                   \
+                   (const bf16*)v, cu_seqlens, sink, (bf16*)out, H, K, R, DV, scale, window, gate, ld_gate);                    \
     } while (0)
     if (DV <= 32) QWB_LM(4); else if (DV <= 64) QWB_LM(8); else if (DV <= 128) QWB_LM(16); else QWB_LM(32);
 #undef QWB_LM

@@ -1,12 +1,15 @@
-// Attention over the paged cache with one or two score maps per head, soft-capped scores and a causal or chunked mask.
+// Attention over the paged cache with one or two score maps per head, soft-capped scores and a causal, chunked or windowed
+// mask.
 //
 // A query head has `maps` (1 or 2) query vectors of `dim` values, laid out one after the other, and so has a key head;
 // map m of query head h is scored against map m of key head h / (H / G).  Each map is a softmax attention of its own
 // over the SAME values (size vdim).  With two maps the head's output is their difference, a1 - lambda * a2 (differential
 // attention; lambda is one number for the layer); with `norm_out` the output is then divided by its root mean square
-// over vdim (eps inside the root) and multiplied by out_scale.
+// over vdim (eps inside the root) and multiplied by out_scale.  With a gate (a number per token and head) head h's output is
+// multiplied by its sigmoid.
 //   score = q . k * scale;  softcap > 0:  score <- softcap * tanh(score / softcap)
-//   mask:  key j is seen from position p when j <= p and (chunk > 0) floor(j / chunk) = floor(p / chunk); chunks are
+//   mask:  key j is seen from position p when j <= p, (chunk > 0) floor(j / chunk) = floor(p / chunk), and (window > 0)
+//          p - j < window; chunks are
 //          counted from position 0 of the sequence.
 // Scores, maxima, sums, accumulators, the difference and the norm are 32-bit; q and the cache are float or bfloat16.
 // The cache: K pool [pages, G, 64, maps * dim], V pool [pages, G, 64, vdim].
@@ -41,16 +44,27 @@ __device__ __forceinline__ float maps_turned(const float* v, int i, int n, const
     return first ? a * c - b * s : b * c + a * s;
 }
 
-__device__ __forceinline__ int maps_first_key(int p, int chunk) { return chunk > 0 ? (p / chunk) * chunk : 0; }
+struct MapsMask { int chunk, window; };             // 0: none
+struct MapsGate { const float* rows; int ld; };     // a number per token and head, its sigmoid multiplies the head's output; null: none
+
+__host__ __device__ __forceinline__ int maps_first_key(int p, MapsMask mask) {
+    const int c = mask.chunk > 0 ? (p / mask.chunk) * mask.chunk : 0;
+    const int w = mask.window > 0 && p >= mask.window ? p - mask.window + 1 : 0;
+    return c > w ? c : w;
+}
+
+__device__ __forceinline__ float maps_gate(MapsGate gate, size_t t, int h) {
+    return gate.rows ? 1.f / (1.f + expf(-gate.rows[t * gate.ld + h])) : 1.f;
+}
 
 __device__ __forceinline__ float maps_cap(float s, float cap, float inv_cap) { return cap > 0.f ? cap * tanhf(s * inv_cap) : s; }
 
 // ---------------------------------------------------------------------------------
 // prep: grid (T, ceil(items / 4)), 4 warps, a warp per (token, item); items = H * maps query maps, G * maps key maps,
-// G values.  qkv [T, (H + G) * maps * dim + G * vdim] float: the projections (after a convolution, if the mixer has one).
+// G values.  qkv: rows of ld floats that begin with the (H + G) * maps * dim + G * vdim projections (after a convolution, if the mixer has one).
 // ---------------------------------------------------------------------------------
 template <typename T>
-__global__ void maps_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ qw,
+__global__ void maps_prep_kernel(const float* __restrict__ qkv, int ld, const float* __restrict__ bias, const float* __restrict__ qw,
                                  const float* __restrict__ kw, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                                  const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ page_table,
                                  int table_width, T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool, int H, int G,
@@ -63,7 +77,6 @@ __global__ void maps_prep_kernel(const float* __restrict__ qkv, const float* __r
     const int nq = H * maps, nk = G * maps;
     if (item >= nq + nk + G) return;
     float* buf = bufs[warp];
-    const int ld = (nq + nk) * dim + G * vdim;
     const bool is_q = item < nq, is_k = !is_q && item < nq + nk;
     const int n = (is_q || is_k) ? dim : vdim;
     const int col = is_q ? item * dim : (is_k ? nq * dim + (item - nq) * dim : (nq + nk) * dim + (item - nq - nk) * vdim);
@@ -124,7 +137,7 @@ __device__ __forceinline__ float maps_q_factor(int p, float coef, float every) {
 // The qkv product runs right before this kernel, which may have been launched early: qkv is read past the read-only cache.
 template <typename T>
 __global__ void __launch_bounds__(QWB_ROW_PREP_THREADS)
-maps_row_prep_fours_kernel(const float* qkv, const float* __restrict__ bias, const float* __restrict__ qw, const float* __restrict__ kw,
+maps_row_prep_fours_kernel(const float* qkv, int ld, const float* __restrict__ bias, const float* __restrict__ qw, const float* __restrict__ kw,
                            const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ page_table,
                            int table_width, T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool, int H, int G, int kdim,
                            int vdim, float eps, float t_coef, float t_every, int store_kv) {
@@ -133,7 +146,7 @@ maps_row_prep_fours_kernel(const float* qkv, const float* __restrict__ bias, con
     __shared__ float sums[2][QWB_ROW_PREP_THREADS / 32];
     const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
     const int nq4 = H * kdim / 4, nk4 = G * kdim / 4, nkv4 = nk4 + G * vdim / 4;
-    const float4* src = reinterpret_cast<const float4*>(qkv) + (size_t)t * (nq4 + nkv4);
+    const float4* src = reinterpret_cast<const float4*>(qkv) + (size_t)t * (ld / 4);
     const float4* bs = reinterpret_cast<const float4*>(bias);
     auto load = [&](int i) {
         float4 v = __ldcg(src + i);
@@ -190,7 +203,7 @@ maps_row_prep_fours_kernel(const float* qkv, const float* __restrict__ bias, con
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-maps_row_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ qw,
+maps_row_prep_kernel(const float* __restrict__ qkv, int ld, const float* __restrict__ bias, const float* __restrict__ qw,
                      const float* __restrict__ kw, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                      const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ page_table,
                      int table_width, T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool, int H, int G, int maps,
@@ -202,7 +215,7 @@ maps_row_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
     if (part > 0 && !store_kv) return;
     const int kdim = maps * dim, nq = H * kdim, nk = G * kdim, nv = G * vdim;
     const int n = part == 0 ? nq : (part == 1 ? nk : nv), col = part == 0 ? 0 : (part == 1 ? nq : nq + nk);
-    const int ld = nq + nk + nv, per = part == 2 ? vdim : kdim;
+    const int per = part == 2 ? vdim : kdim;
     const float* src = qkv + (size_t)t * ld + col;
     const float* bs = bias ? bias + col : nullptr;
     const float* w = part == 0 ? qw : (part == 1 ? kw : nullptr);
@@ -237,46 +250,49 @@ maps_row_prep_kernel(const float* __restrict__ qkv, const float* __restrict__ bi
 }
 
 // `step`: 1 for the kernels that read value by value, 8 for those that copy 16 bytes at a time
-static int check_maps_sizes(const char* what, int H, int G, int maps, int dim, int vdim, int table_width, int chunk, int step) {
+static int check_maps_sizes(const char* what, int H, int G, int maps, int dim, int vdim, int table_width, MapsMask mask, int step) {
     if (H <= 0 || G <= 0 || H % G) return qwb_fail(QWB_ERR_ARG, "%s: %d query heads are not a multiple of %d key/value heads", what, H, G);
     if (maps < 1 || maps > QWB_MAPS_MAX) return qwb_fail(QWB_ERR_ARG, "%s: %d score maps per head (1 or 2)", what, maps);
     if (dim <= 0 || dim % step || dim > QWB_MAPS_MAX_DIM || vdim <= 0 || vdim % step || vdim > QWB_MAPS_MAX_DIM)
         return qwb_fail(QWB_ERR_ARG, "%s: key size %d or value size %d is not a multiple of %d in [%d, %d]", what, dim, vdim, step, step, QWB_MAPS_MAX_DIM);
-    if (table_width <= 0 || chunk < 0) return qwb_fail(QWB_ERR_ARG, "%s: bad table width %d or chunk %d", what, table_width, chunk);
+    if (table_width <= 0 || mask.chunk < 0 || mask.window < 0)
+        return qwb_fail(QWB_ERR_ARG, "%s: bad table width %d, chunk %d or window %d", what, table_width, mask.chunk, mask.window);
     return 0;
 }
 
-extern "C" int qwb_maps_prep(const float* qkv, const float* bias, const float* qw, const float* kw, const float* cos_t, const float* sin_t,
+extern "C" int qwb_maps_prep(const float* qkv, int ld, const float* bias, const float* qw, const float* kw, const float* cos_t, const float* sin_t,
                              const int* tok_seq, const int* tok_pos, const int* page_table, int table_width, void* q_out, void* k_pool,
                              void* v_pool, int dtype, int T, int H, int G, int maps, int dim, int vdim, int rdims, int interleaved,
                              float eps, int store_kv, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (int rc = check_maps_sizes("maps_prep", H, G, maps, dim, vdim, table_width, 0, 1)) return rc;
+    if (int rc = check_maps_sizes("maps_prep", H, G, maps, dim, vdim, table_width, MapsMask{0, 0}, 1)) return rc;
+    if (ld < (H + G) * maps * dim + G * vdim) return qwb_fail(QWB_ERR_ARG, "maps_prep: rows of %d values", ld);
     if (rdims < 0 || rdims > dim || rdims % 2) return qwb_fail(QWB_ERR_ARG, "maps_prep: a rotation of %d of %d values", rdims, dim);
     if (rdims > 0 && (!cos_t || !sin_t)) return qwb_fail(QWB_ERR_ARG, "maps_prep: a rotation without its table");
     dim3 grid(T, ((H + G) * maps + G + 3) / 4);
     if (dtype == QWB_DT_F32)
-        qwb_launch(maps_prep_kernel<float>, grid, 128, 0, stream, qkv, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos, page_table, table_width,
+        qwb_launch(maps_prep_kernel<float>, grid, 128, 0, stream, qkv, ld, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos, page_table, table_width,
                    (float*)q_out, (float*)k_pool, (float*)v_pool, H, G, maps, dim, vdim, rdims, interleaved, eps, store_kv);
     else if (dtype == QWB_DT_BF16)
-        qwb_launch(maps_prep_kernel<bf16>, grid, 128, 0, stream, qkv, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos, page_table, table_width,
+        qwb_launch(maps_prep_kernel<bf16>, grid, 128, 0, stream, qkv, ld, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos, page_table, table_width,
                    (bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool, H, G, maps, dim, vdim, rdims, interleaved, eps, store_kv);
     else return qwb_fail(QWB_ERR_ARG, "maps_prep: unknown dtype %d", dtype);
     return qwb_check_launch("maps_prep");
 }
 
 // qw [H * maps * dim], kw [G * maps * dim] (either may be null); the rest as qwb_maps_prep.
-extern "C" int qwb_maps_row_prep(const float* qkv, const float* bias, const float* qw, const float* kw, const float* cos_t, const float* sin_t,
+extern "C" int qwb_maps_row_prep(const float* qkv, int ld, const float* bias, const float* qw, const float* kw, const float* cos_t, const float* sin_t,
                                  const int* tok_seq, const int* tok_pos, const int* page_table, int table_width, void* q_out, void* k_pool,
                                  void* v_pool, int dtype, int T, int H, int G, int maps, int dim, int vdim, int rdims, int interleaved,
                                  float eps, float t_coef, float t_every, int store_kv, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (int rc = check_maps_sizes("maps_row_prep", H, G, maps, dim, vdim, table_width, 0, 1)) return rc;
+    if (int rc = check_maps_sizes("maps_row_prep", H, G, maps, dim, vdim, table_width, MapsMask{0, 0}, 1)) return rc;
+    if (ld < (H + G) * maps * dim + G * vdim) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: rows of %d values", ld);
     if (rdims < 0 || rdims > dim || rdims % 2) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a rotation of %d of %d values", rdims, dim);
     if (rdims > 0 && (!cos_t || !sin_t)) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a rotation without its table");
     if (t_coef != 0.f && !(t_every > 0.f)) return qwb_fail(QWB_ERR_ARG, "maps_row_prep: a query factor in steps of %g positions", t_every);
     const int nq = H * maps * dim, nkv = G * (maps * dim + vdim);
-    const bool fours = rdims == 0 && (maps * dim) % 4 == 0 && vdim % 4 == 0 && nq <= 4 * QWB_ROW_PREP_THREADS * QWB_ROW_PREP_Q &&
+    const bool fours = rdims == 0 && ld % 4 == 0 && (maps * dim) % 4 == 0 && vdim % 4 == 0 && nq <= 4 * QWB_ROW_PREP_THREADS * QWB_ROW_PREP_Q &&
                        nkv <= 4 * QWB_ROW_PREP_THREADS * QWB_ROW_PREP_KV && (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 &&
                        (uintptr_t)qw % 16 == 0 && (uintptr_t)kw % 16 == 0;
     auto go = [&](auto* q, auto* k, auto* v) {
@@ -284,9 +300,9 @@ extern "C" int qwb_maps_row_prep(const float* qkv, const float* bias, const floa
         if (fours)      // as many threads as two pieces each of q and of k and v want, if that is fewer
             qwb_launch_link(T, QWB_LINK_ROWS_NORM, maps_row_prep_fours_kernel<E>, dim3(T),
                             dim3(nq <= 4 * 128 * QWB_ROW_PREP_Q / 2 && nkv <= 4 * 128 * QWB_ROW_PREP_KV / 2 ? 128 : QWB_ROW_PREP_THREADS), 0, stream,
-                            qkv, bias, qw, kw, tok_seq, tok_pos, page_table, table_width, q, k, v, H, G, maps * dim, vdim, eps, t_coef, t_every, store_kv);
+                            qkv, ld, bias, qw, kw, tok_seq, tok_pos, page_table, table_width, q, k, v, H, G, maps * dim, vdim, eps, t_coef, t_every, store_kv);
         else
-            qwb_launch(maps_row_prep_kernel<E>, dim3(T, 3), dim3(nq >= 1024 ? 256 : 128), 0, stream, qkv, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos,
+            qwb_launch(maps_row_prep_kernel<E>, dim3(T, 3), dim3(nq >= 1024 ? 256 : 128), 0, stream, qkv, ld, bias, qw, kw, cos_t, sin_t, tok_seq, tok_pos,
                        page_table, table_width, q, k, v, H, G, maps, dim, vdim, rdims, interleaved, eps, t_coef, t_every, store_kv);
     };
     if (dtype == QWB_DT_F32) go((float*)q_out, (float*)k_pool, (float*)v_pool);
@@ -304,7 +320,7 @@ template <typename T, int NC>   // NC = ceil(vdim / 32) rounded up to 2, 4 or 8
 __global__ void maps_prefill_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const T* __restrict__ v_pool,
                                     const int* __restrict__ page_table, const int* __restrict__ cu_seqlens, const int* __restrict__ pos0,
                                     T* __restrict__ out, int H, int G, int maps, int dim, int vdim, int table_width, float scale,
-                                    float softcap, int chunk, float lambda, int norm_out, float eps, float out_scale) {
+                                    float softcap, MapsMask mask, float lambda, int norm_out, float eps, float out_scale, MapsGate gate) {
     pdl_wait();
     pdl_launch_dependents();
     constexpr int BQ = 16, BK = 32, QPW = 4, PG = QWB_MAPS_PAGE;
@@ -325,7 +341,7 @@ __global__ void maps_prefill_kernel(const T* __restrict__ q, const T* __restrict
 
     float res[QPW][NC];                       // map 0's normed sums, then the difference
     const int k_last = p0 + q0 + nq - 1;
-    const int k_first = maps_first_key(p0 + q0, chunk);
+    const int k_first = maps_first_key(p0 + q0, mask);
     const int* pages = page_table + (size_t)b * table_width;
 
     for (int mp = 0; mp < maps; ++mp) {
@@ -368,7 +384,7 @@ __global__ void maps_prefill_kernel(const T* __restrict__ q, const T* __restrict
             for (int i = 0; i < QPW; ++i) {
                 const int qi = warp * QPW + i;
                 const int qp = p0 + q0 + qi;
-                const bool ok = qi < nq && key <= qp && key >= maps_first_key(qp, chunk);
+                const bool ok = qi < nq && key <= qp && key >= maps_first_key(qp, mask);
                 const float si = ok ? maps_cap(s[i], softcap, inv_cap) : -INFINITY;
                 const float m_new = fmaxf(m[i], warp_max(si));
                 if (m_new == -INFINITY) { p[i] = 0.f; continue; }       // nothing visible so far (whole warp agrees)
@@ -416,6 +432,7 @@ __global__ void maps_prefill_kernel(const T* __restrict__ q, const T* __restrict
             mul = rsqrtf(warp_sum(ss) / (float)vdim + eps) * out_scale;
         }
         if (qi >= nq) continue;
+        mul *= maps_gate(gate, t0 + q0 + qi, h);
         T* o = out + ((size_t)(t0 + q0 + qi) * H + h) * vdim;
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
@@ -428,8 +445,8 @@ __global__ void maps_prefill_kernel(const T* __restrict__ q, const T* __restrict
 template <typename T>
 static int launch_maps_prefill(const void* q, const void* k_pool, const void* v_pool, const int* page_table, const int* cu_seqlens,
                                const int* pos0, void* out, int B, int max_new, int H, int G, int maps, int dim, int vdim, int table_width,
-                               float scale, float softcap, int chunk, float lambda, int norm_out, float eps, float out_scale,
-                               cudaStream_t stream) {
+                               float scale, float softcap, MapsMask mask, float lambda, int norm_out, float eps, float out_scale,
+                               MapsGate gate, cudaStream_t stream) {
     const size_t smem = ((size_t)16 * dim + 32 * (dim + 1) + 32 * vdim) * sizeof(float);
     dim3 grid((max_new + 15) / 16, H, B);
     const int nc = (vdim + 31) / 32;
@@ -441,8 +458,8 @@ static int launch_maps_prefill(const void* q, const void* k_pool, const void* v_
             if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "maps_prefill: %s", cudaGetErrorString(e));      \
         }                                                                                                        \
         qwb_launch(maps_prefill_kernel<T, NC>, grid, 128, smem, stream, (const T*)q, (const T*)k_pool, (const T*)v_pool, \
-            page_table, cu_seqlens, pos0, (T*)out, H, G, maps, dim, vdim, table_width, scale, softcap, chunk, lambda, norm_out, \
-            eps, out_scale);                                                                                     \
+            page_table, cu_seqlens, pos0, (T*)out, H, G, maps, dim, vdim, table_width, scale, softcap, mask, lambda, norm_out, \
+            eps, out_scale, gate);                                                                                     \
     } while (0)
     if (nc <= 2) QWB_LAUNCH_MAPS_PREFILL(2);
     else if (nc <= 4) QWB_LAUNCH_MAPS_PREFILL(4);
@@ -454,17 +471,19 @@ static int launch_maps_prefill(const void* q, const void* k_pool, const void* v_
 // q [T, H, maps * dim]; out [T, H * vdim].
 extern "C" int qwb_maps_prefill(const void* q, const void* k_pool, const void* v_pool, const int* page_table, const int* cu_seqlens,
                                 const int* pos0, void* out, int dtype, int B, int max_new, int H, int G, int maps, int dim, int vdim,
-                                int table_width, float scale, float softcap, int chunk, float lambda, int norm_out, float eps,
-                                float out_scale, cudaStream_t stream) {
+                                int table_width, float scale, float softcap, int chunk, int window, float lambda, int norm_out, float eps,
+                                float out_scale, const float* gate_rows, int ld_gate, cudaStream_t stream) {
+    const MapsMask mask{chunk, window};
+    const MapsGate gate{gate_rows, ld_gate};
     if (B <= 0 || max_new <= 0) return 0;
-    if (int rc = check_maps_sizes("maps_prefill", H, G, maps, dim, vdim, table_width, chunk, 1)) return rc;
+    if (int rc = check_maps_sizes("maps_prefill", H, G, maps, dim, vdim, table_width, mask, 1)) return rc;
     if (B > 65535 || H > 65535) return qwb_fail(QWB_ERR_ARG, "maps_prefill: batch %d or heads %d above 65535", B, H);
     if (dtype == QWB_DT_F32)
         return launch_maps_prefill<float>(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, max_new, H, G, maps, dim, vdim, table_width,
-                                          scale, softcap, chunk, lambda, norm_out, eps, out_scale, stream);
+                                          scale, softcap, mask, lambda, norm_out, eps, out_scale, gate, stream);
     if (dtype == QWB_DT_BF16)
         return launch_maps_prefill<bf16>(q, k_pool, v_pool, page_table, cu_seqlens, pos0, out, B, max_new, H, G, maps, dim, vdim, table_width,
-                                         scale, softcap, chunk, lambda, norm_out, eps, out_scale, stream);
+                                         scale, softcap, mask, lambda, norm_out, eps, out_scale, gate, stream);
     return qwb_fail(QWB_ERR_ARG, "maps_prefill: unknown dtype %d", dtype);
 }
 
@@ -529,7 +548,7 @@ __global__ void __launch_bounds__(128)
 maps_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                         const int* __restrict__ page_table, const int* __restrict__ cu_seqlens, const int* __restrict__ pos0,
                         bf16* __restrict__ out, int H, int G, int dim, int vdim, int table_width, float scale, float softcap,
-                        int chunk, float lambda, int norm_out, float eps, float out_scale) {
+                        MapsMask mask, float lambda, int norm_out, float eps, float out_scale, MapsGate gate) {
     pdl_wait();
     pdl_launch_dependents();
     const int ldq = dim + MM_PAD, ldv = vdim + MM_PAD, kdim = MAPS * dim;
@@ -548,15 +567,15 @@ maps_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
     const int nq = min(MM_BQ, n - q0);
     const int gr = lane >> 2, tq = lane & 3;
     const int pos_a = p0 + q0 + warp * 16 + gr, pos_b = pos_a + 8;  // positions of the thread's two rows
-    const int lo_a = maps_first_key(pos_a, chunk), lo_b = maps_first_key(pos_b, chunk);
+    const int lo_a = maps_first_key(pos_a, mask), lo_b = maps_first_key(pos_b, mask);
 
     const int k_hi = p0 + q0 + nq - 1;                              // last key any query of the tile sees
-    const int k_lo = maps_first_key(p0 + q0, chunk);                // first key any of them sees
+    const int k_lo = maps_first_key(p0 + q0, mask);                // first key any of them sees
     const int nv_used = vdim / 8;
     const int first_page = k_lo / MM_BK, n_tiles = k_hi / MM_BK - first_page + 1;
     const int* pages = page_table + (size_t)b * table_width;
     const int warp_lo = p0 + q0 + warp * 16, warp_hi = warp_lo + 15;
-    const int warp_first = maps_first_key(warp_hi, chunk);          // the first key that every row of the warp may see
+    const int warp_first = maps_first_key(warp_hi, mask);          // the first key that every row of the warp may see
     const float log2e = 1.4426950408889634f;
     // Scores in units of ln 2 (ex2 below).  With a cap c: c tanh(x / c) = c - 2 c / (e^(2 x / c) + 1), exact at both ends
     // (e^.. = inf or 0) and a few units of the last place in between: one ex2, one rcp and one fma a score.
@@ -611,8 +630,8 @@ maps_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
             }
             __syncthreads();
             const int key0 = (first_page + it) * MM_BK;
-            // a tile that no row of the warp sees (behind its last row, or before its chunk) is skipped by the warp
-            const bool none = key0 > warp_hi || key0 + MM_BK <= maps_first_key(warp_lo, chunk);
+            // a tile that no row of the warp sees (behind its last row, or before its chunk or window) is skipped by the warp
+            const bool none = key0 > warp_hi || key0 + MM_BK <= maps_first_key(warp_lo, mask);
             float s[8][4];
             if (!none) {
 #pragma unroll
@@ -716,6 +735,8 @@ maps_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
                 mul1 = rsqrtf(ss1 / (float)vdim + eps) * out_scale;
             }
             const int row_a = warp * 16 + gr, row_b = row_a + 8;
+            if (row_a < nq) mul0 *= maps_gate(gate, t0 + q0 + row_a, h);
+            if (row_b < nq) mul1 *= maps_gate(gate, t0 + q0 + row_b, h);
 #pragma unroll
             for (int j = 0; j < NV; ++j) {
                 if (j < nv_used) {
@@ -737,7 +758,7 @@ __global__ void __launch_bounds__(128)
 maps_prefill_mma_pair_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                              const int* __restrict__ page_table, const int* __restrict__ cu_seqlens, const int* __restrict__ pos0,
                              bf16* __restrict__ out, int H, int G, int dim, int vdim, int table_width, float scale, float softcap,
-                             int chunk, float lambda, int norm_out, float eps, float out_scale) {
+                             MapsMask mask, float lambda, int norm_out, float eps, float out_scale, MapsGate gate) {
     pdl_wait();
     pdl_launch_dependents();
     const int kdim = 2 * dim, ldq = kdim + MM_PAD, ldv = vdim + MM_PAD;
@@ -755,13 +776,13 @@ maps_prefill_mma_pair_kernel(const bf16* __restrict__ q, const bf16* __restrict_
     const int nq = min(MM_BQ, n - q0);
     const int gr = lane >> 2, tq = lane & 3;
     const int pos_a = p0 + q0 + warp * 16 + gr, pos_b = pos_a + 8;
-    const int lo_a = maps_first_key(pos_a, chunk), lo_b = maps_first_key(pos_b, chunk);
-    const int k_hi = p0 + q0 + nq - 1, k_lo = maps_first_key(p0 + q0, chunk);
+    const int lo_a = maps_first_key(pos_a, mask), lo_b = maps_first_key(pos_b, mask);
+    const int k_hi = p0 + q0 + nq - 1, k_lo = maps_first_key(p0 + q0, mask);
     const int nv_used = vdim / 8;
     const int first_page = k_lo / MM_BK, n_tiles = k_hi / MM_BK - first_page + 1;
     const int* pages = page_table + (size_t)b * table_width;
     const int warp_lo = p0 + q0 + warp * 16, warp_hi = warp_lo + 15;
-    const int warp_first = maps_first_key(warp_hi, chunk);
+    const int warp_first = maps_first_key(warp_hi, mask);
     const float log2e = 1.4426950408889634f;
     const float mul_s = softcap > 0.f ? scale / softcap * 2.f * log2e : scale * log2e;
     const float cap2 = softcap * log2e;
@@ -805,7 +826,7 @@ maps_prefill_mma_pair_kernel(const bf16* __restrict__ q, const bf16* __restrict_
         if (more) { copy_keys(it + 1, (it + 1) & 1); mm_wait<2>(); } else { mm_wait<1>(); }
         __syncthreads();
         const int key0 = (first_page + it) * MM_BK;
-        const bool none = key0 > warp_hi || key0 + MM_BK <= maps_first_key(warp_lo, chunk);
+        const bool none = key0 > warp_hi || key0 + MM_BK <= maps_first_key(warp_lo, mask);
         const bool whole = key0 + MM_BK - 1 <= warp_lo && key0 >= warp_first;
         uint32_t pk[2][4][4];                                       // both maps' probabilities as the second product's A operands
         if (!none) {
@@ -908,6 +929,8 @@ maps_prefill_mma_pair_kernel(const bf16* __restrict__ q, const bf16* __restrict_
         mul1 = rsqrtf(ss1 / (float)vdim + eps) * out_scale;
     }
     const int row_a = warp * 16 + gr, row_b = row_a + 8;
+    if (row_a < nq) mul0 *= maps_gate(gate, t0 + q0 + row_a, h);
+    if (row_b < nq) mul1 *= maps_gate(gate, t0 + q0 + row_b, h);
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
         if (j < nv_used) {
@@ -931,10 +954,12 @@ extern "C" int qwb_maps_prefill_mma_fits(int dtype, int maps, int dim, int vdim)
 // q [T, H, maps * dim] bfloat16; out [T, H * vdim] bfloat16.
 extern "C" int qwb_maps_prefill_mma(const void* q, const void* k_pool, const void* v_pool, const int* page_table, const int* cu_seqlens,
                                     const int* pos0, void* out, int B, int max_new, int H, int G, int maps, int dim, int vdim,
-                                    int table_width, float scale, float softcap, int chunk, float lambda, int norm_out, float eps,
-                                    float out_scale, cudaStream_t stream) {
+                                    int table_width, float scale, float softcap, int chunk, int window, float lambda, int norm_out, float eps,
+                                    float out_scale, const float* gate_rows, int ld_gate, cudaStream_t stream) {
+    const MapsMask mask{chunk, window};
+    const MapsGate gate{gate_rows, ld_gate};
     if (B <= 0 || max_new <= 0) return 0;
-    if (int rc = check_maps_sizes("maps_prefill_mma", H, G, maps, dim, vdim, table_width, chunk, 8)) return rc;
+    if (int rc = check_maps_sizes("maps_prefill_mma", H, G, maps, dim, vdim, table_width, mask, 8)) return rc;
     if (!qwb_maps_prefill_mma_fits(QWB_DT_BF16, maps, dim, vdim))
         return qwb_fail(QWB_ERR_ARG, "maps_prefill_mma: keys of %d (a multiple of 16) and values of %d (of 8) that fit in shared memory", dim, vdim);
     if (B > 65535 || H > 65535) return qwb_fail(QWB_ERR_ARG, "maps_prefill_mma: batch %d or heads %d above 65535", B, H);
@@ -950,7 +975,7 @@ extern "C" int qwb_maps_prefill_mma(const void* q, const void* k_pool, const voi
         }                                                                                                                       \
         qwb_launch(maps_prefill_mma_kernel<NV, MAPS>, grid, 128, smem, stream, (const bf16*)q, (const bf16*)k_pool,             \
                    (const bf16*)v_pool, page_table, cu_seqlens, pos0, (bf16*)out, H, G, dim, vdim, table_width, scale, softcap, \
-                   chunk, lambda, norm_out, eps, out_scale);                                                                    \
+                   mask, lambda, norm_out, eps, out_scale, gate);                                                                    \
     } while (0)
 #define QWB_MM_SIZES(MAPS)                                                                                                      \
     do {                                                                                                                        \
@@ -967,7 +992,7 @@ extern "C" int qwb_maps_prefill_mma(const void* q, const void* k_pool, const voi
         }                                                                                                                       \
         qwb_launch(maps_prefill_mma_pair_kernel<NV>, grid, 128, smem_pair, stream, (const bf16*)q, (const bf16*)k_pool,         \
                    (const bf16*)v_pool, page_table, cu_seqlens, pos0, (bf16*)out, H, G, dim, vdim, table_width, scale, softcap, \
-                   chunk, lambda, norm_out, eps, out_scale);                                                                    \
+                   mask, lambda, norm_out, eps, out_scale, gate);                                                                    \
     } while (0)
         if (vdim <= 32) QWB_MM_PAIR(4); else if (vdim <= 64) QWB_MM_PAIR(8); else QWB_MM_PAIR(16);
 #undef QWB_MM_PAIR
@@ -979,7 +1004,7 @@ extern "C" int qwb_maps_prefill_mma(const void* q, const void* k_pool, const voi
 
 // ---------------------------------------------------------------------------------
 // decode: one new token per sequence (its position is len - 1).  The keys it sees, first .. len - 1 with first the start
-// of its chunk (or 0), are cut into runs of whole pages counted from the page of the first key: 2 pages a run, doubled
+// of its chunk or window (or 0), are cut into runs of whole pages counted from the page of the first key: 2 pages a run, doubled
 // while that would give more than 64 runs.  Which keys a run holds follows from the sequence's own length alone.
 // Block = (run, key/value head and slice of its rows, sequence), 128 threads; a row is a (query head, map) pair, up to 8 a
 // block: a page's K and V tiles go to shared memory; thread (key, half of the rows) forms the scores; a warp per row
@@ -1001,13 +1026,13 @@ template <typename T>
 __global__ void maps_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const T* __restrict__ v_pool,
                                    const int* __restrict__ page_table, const int* __restrict__ seq_len, float* __restrict__ part_acc,
                                    float* __restrict__ part_m, float* __restrict__ part_l, int H, int G, int maps, int dim, int vdim,
-                                   int table_width, float scale, float softcap, int chunk, int n_runs) {
+                                   int table_width, float scale, float softcap, MapsMask mask, int n_runs) {
     pdl_wait();
     pdl_launch_dependents();
     constexpr int RT = QWB_MAPS_ROWS, VEC = Vec16<T>::N, PG = QWB_MAPS_PAGE;
     const int b = blockIdx.z, run = blockIdx.x;
     const int len = seq_len[b];
-    const int first = maps_first_key(len - 1, chunk);
+    const int first = maps_first_key(len - 1, mask);
     const int rp = maps_run_pages(first, len);
     const int page_lo = first / PG;
     const int row_first = max(first, (page_lo + run * rp) * PG);
@@ -1166,15 +1191,15 @@ __global__ void maps_decode_kernel(const T* __restrict__ q, const T* __restrict_
 // warp m first makes map m's weights e^(m_r - M) / L once for all columns, then thread d sums its column.
 template <typename T>
 __global__ void maps_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_m, const float* __restrict__ part_l,
-                                  const int* __restrict__ seq_len, T* __restrict__ out, int H, int maps, int vdim, int chunk, int n_runs,
-                                  float lambda, int norm_out, float eps, float out_scale) {
+                                  const int* __restrict__ seq_len, T* __restrict__ out, int H, int maps, int vdim, MapsMask mask, int n_runs,
+                                  float lambda, int norm_out, float eps, float out_scale, MapsGate gate) {
     pdl_wait();
     pdl_launch_dependents();
     __shared__ float red[32];
     __shared__ float wts[QWB_MAPS_MAX][QWB_MAPS_MAX_RUNS];
     const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int len = seq_len[b];
-    const int first = maps_first_key(len - 1, chunk);
+    const int first = maps_first_key(len - 1, mask);
     const int rp = maps_run_pages(first, len);
     const int runs = min(n_runs, ((len - 1) / QWB_MAPS_PAGE - first / QWB_MAPS_PAGE) / rp + 1);
     if (warp < maps) {
@@ -1214,6 +1239,7 @@ __global__ void maps_merge_kernel(const float* __restrict__ part_acc, const floa
         for (int c = 0; c < 2; ++c) if (tid + c * 128 < vdim) ss += res[c] * res[c];
         mul = rsqrtf(block_sum(ss, red) / (float)vdim + eps) * out_scale;
     }
+    mul *= maps_gate(gate, b, h);
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
         const int d = tid + c * 128;
@@ -1222,11 +1248,12 @@ __global__ void maps_merge_kernel(const float* __restrict__ part_acc, const floa
 }
 
 // runs of the grid for sequences of up to max_len tokens
-extern "C" int qwb_maps_decode_runs(int max_len, int chunk) {
+extern "C" int qwb_maps_decode_runs(int max_len, int chunk, int window) {
     if (max_len <= 0) return 1;
-    // the most pages a sequence's visible keys touch: a chunk may begin anywhere in its first page
+    // the most pages a sequence's visible keys touch: a chunk or a window may begin anywhere in its first page
     const int pages_all = (max_len + QWB_MAPS_PAGE - 1) / QWB_MAPS_PAGE;
-    const int pages = chunk > 0 ? min(pages_all, (chunk + QWB_MAPS_PAGE - 2) / QWB_MAPS_PAGE + 1) : pages_all;
+    const int most = chunk > 0 && window > 0 ? min(chunk, window) : max(chunk, window);
+    const int pages = most > 0 ? min(pages_all, (most + QWB_MAPS_PAGE - 2) / QWB_MAPS_PAGE + 1) : pages_all;
     const int runs = (pages + QWB_MAPS_RUN_PAGES - 1) / QWB_MAPS_RUN_PAGES;
     return runs < QWB_MAPS_MAX_RUNS ? runs : QWB_MAPS_MAX_RUNS;
 }
@@ -1238,8 +1265,8 @@ extern "C" long long qwb_maps_decode_scratch_floats(int B, int H, int maps, int 
 template <typename T>
 static int launch_maps_decode(const void* q, const void* k_pool, const void* v_pool, const int* page_table, const int* seq_len,
                               float* scratch, void* out, int B, int H, int G, int maps, int dim, int vdim, int table_width, float scale,
-                              float softcap, int chunk, int n_runs, float lambda, int norm_out, float eps, float out_scale,
-                              cudaStream_t stream) {
+                              float softcap, MapsMask mask, int n_runs, float lambda, int norm_out, float eps, float out_scale,
+                              MapsGate gate, cudaStream_t stream) {
     constexpr int VEC = Vec16<T>::N;
     const int kdim = maps * dim;
     const size_t rows = (size_t)B * H * maps;
@@ -1254,26 +1281,28 @@ static int launch_maps_decode(const void* q, const void* k_pool, const void* v_p
     }
     const int rows_g = (H / G) * maps, slices = (rows_g + QWB_MAPS_ROWS - 1) / QWB_MAPS_ROWS;
     qwb_launch(maps_decode_kernel<T>, dim3(n_runs, G * slices, B), 128, smem, stream, (const T*)q, (const T*)k_pool, (const T*)v_pool,
-               page_table, seq_len, part_acc, part_m, part_l, H, G, maps, dim, vdim, table_width, scale, softcap, chunk, n_runs);
+               page_table, seq_len, part_acc, part_m, part_l, H, G, maps, dim, vdim, table_width, scale, softcap, mask, n_runs);
     if (int rc = qwb_check_launch("maps_decode")) return rc;
     qwb_launch(maps_merge_kernel<T>, dim3(H, B), 128, 0, stream, (const float*)part_acc, (const float*)part_m, (const float*)part_l,
-               seq_len, (T*)out, H, maps, vdim, chunk, n_runs, lambda, norm_out, eps, out_scale);
+               seq_len, (T*)out, H, maps, vdim, mask, n_runs, lambda, norm_out, eps, out_scale, gate);
     return qwb_check_launch("maps_merge");
 }
 
 // q [B, H, maps * dim]; out [B, H * vdim]; scratch: qwb_maps_decode_scratch_floats floats.
 extern "C" int qwb_maps_decode(const void* q, const void* k_pool, const void* v_pool, const int* page_table, const int* seq_len,
                                float* scratch, void* out, int dtype, int B, int H, int G, int maps, int dim, int vdim, int table_width,
-                               float scale, float softcap, int chunk, int n_runs, float lambda, int norm_out, float eps, float out_scale,
-                               cudaStream_t stream) {
+                               float scale, float softcap, int chunk, int window, int n_runs, float lambda, int norm_out, float eps, float out_scale,
+                               const float* gate_rows, int ld_gate, cudaStream_t stream) {
+    const MapsMask mask{chunk, window};
+    const MapsGate gate{gate_rows, ld_gate};
     if (B <= 0) return 0;
-    if (int rc = check_maps_sizes("maps_decode", H, G, maps, dim, vdim, table_width, chunk, 8)) return rc;
+    if (int rc = check_maps_sizes("maps_decode", H, G, maps, dim, vdim, table_width, mask, 8)) return rc;
     if (n_runs <= 0 || n_runs > 65535 || B > 65535) return qwb_fail(QWB_ERR_ARG, "maps_decode: %d runs, %d sequences", n_runs, B);
     if (dtype == QWB_DT_F32)
         return launch_maps_decode<float>(q, k_pool, v_pool, page_table, seq_len, scratch, out, B, H, G, maps, dim, vdim, table_width, scale,
-                                         softcap, chunk, n_runs, lambda, norm_out, eps, out_scale, stream);
+                                         softcap, mask, n_runs, lambda, norm_out, eps, out_scale, gate, stream);
     if (dtype == QWB_DT_BF16)
         return launch_maps_decode<bf16>(q, k_pool, v_pool, page_table, seq_len, scratch, out, B, H, G, maps, dim, vdim, table_width, scale,
-                                        softcap, chunk, n_runs, lambda, norm_out, eps, out_scale, stream);
+                                        softcap, mask, n_runs, lambda, norm_out, eps, out_scale, gate, stream);
     return qwb_fail(QWB_ERR_ARG, "maps_decode: unknown dtype %d", dtype);
 }

@@ -5,6 +5,8 @@
 //                 ties to the lower index; weights from the scores alone
 //   moe_up        act[t, k, :] = silu(Wg[e] x_t) * (Wu[e] x_t) (gated) or f(Wu[e] x_t), e = the k-th choice of token t
 //   moe_down      out[t, :] = sum_k weight[t, k] * Wd[e_k] act[t, k, :]
+// The weights may stand on the experts' inputs instead: act = f(Wu[e] (w x_t)), formed as f(w (Wu[e] x_t)) in 32-bit (both
+// factors of the gated form), and the sum over the choices is then plain.
 // A shared expert (ungated, a width of its own) that every token uses rides in the same two kernels; its output is
 // multiplied by a number per token.
 //
@@ -173,7 +175,7 @@ __device__ __forceinline__ void lane_dots(const T* __restrict__ w, size_t ldw, i
 // A warp makes two features of a plain expert, one of a gated one (its gate and its up row), two of the shared expert.
 template <typename T, int NT>
 __global__ void __launch_bounds__(256, MOE_UP_BLOCKS)
-moe_up_kernel(const T* __restrict__ x, const T* __restrict__ wu, const int* __restrict__ chosen, T* __restrict__ act,
+moe_up_kernel(const T* __restrict__ x, const T* __restrict__ wu, const int* __restrict__ chosen, const float* __restrict__ weight_in, T* __restrict__ act,
               const T* __restrict__ wsu, T* __restrict__ act_s, int n_tok, int D, int F, int Fs, int top, int kind) {
     pdl_wait();
     pdl_launch_dependents();
@@ -188,7 +190,8 @@ moe_up_kernel(const T* __restrict__ x, const T* __restrict__ wu, const int* __re
         float acc[2];
         lane_dots<T, 2, 1>(wu + first * D, gated ? (size_t)F * D : (size_t)D, gated ? 2 : min(2, F - f), x + (size_t)(slot / top) * D, 0, 1, D,
                            lane, acc);
-        const float a = warp_sum(acc[0]), b = warp_sum(acc[1]);
+        const float w = weight_in ? weight_in[slot] : 1.f;
+        const float a = warp_sum(acc[0]) * w, b = warp_sum(acc[1]) * w;
         T* o = act + (size_t)slot * F + f;
         if (gated) { if (lane == 0) o[0] = from_f32<T>(a / (1.f + expf(-a)) * b); }
         else if (lane < min(2, F - f)) o[lane] = from_f32<T>(qwb_activate(lane ? b : a, kind));
@@ -224,7 +227,7 @@ __global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__
     if (k < top) {
         const size_t slot = (size_t)t * top + k;
         lane_dots<T, NR, 1>(wd + ((size_t)chosen[slot] * D + d) * F, F, nr, act + slot * F, 0, 1, F, lane, acc);
-        mul = weight[slot];
+        mul = weight ? weight[slot] : 1.f;
     } else {
         lane_dots<T, NR, 1>(wsd + (size_t)d * Fs, Fs, nr, act_s + (size_t)t * Fs, 0, 1, Fs, lane, acc);
         mul = gate ? gate[t] : 1.f;
@@ -244,22 +247,23 @@ __global__ void moe_down_kernel(const T* __restrict__ act, const T* __restrict__
 }
 
 template <typename T>
-static void launch_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight, const void* wsu,
+static void launch_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight_in, const float* weight, const void* wsu,
                                const void* wsd, const float* gate, void* act, void* act_s, float* out, int n_tok, int D, int F, int Fs,
                                int top, int kind, int onto, cudaStream_t stream) {
     const int per_slot = ((kind == QWB_MOE_GATED ? F : (F + 1) / 2) + 7) / 8, per_group = Fs > 0 ? ((Fs + 1) / 2 + 7) / 8 : 0;
     const int nt = n_tok > 1 ? 2 : 1;
     const dim3 g1(n_tok * top * per_slot + (n_tok + nt - 1) / nt * per_group), g2((D + 3) / 4, n_tok);
     if (nt == 1)
-        qwb_launch(moe_up_kernel<T, 1>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
+        qwb_launch(moe_up_kernel<T, 1>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, weight_in, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
     else
-        qwb_launch(moe_up_kernel<T, 2>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
+        qwb_launch(moe_up_kernel<T, 2>, g1, 256, 0, stream, (const T*)x, (const T*)wu, chosen, weight_in, (T*)act, (const T*)wsu, (T*)act_s, n_tok, D, F, Fs, top, kind);
     qwb_launch(moe_down_kernel<T, 4>, g2, 32 * (top + (Fs > 0 ? 1 : 0)), 0, stream, (const T*)act, (const T*)wd, chosen, weight, (const T*)act_s,
                (const T*)wsd, gate, out, D, F, Fs, top, onto);
 }
 
+// weight [T, top]: on the experts' inputs (on_input) or outputs.
 // wsu [Fs, D], wsd [D, Fs], gate [T] (or null: 1), act_s [T, Fs]: the shared expert, Fs = 0 for none.
-extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight, const void* wsu,
+extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, const int* chosen, const float* weight, int on_input, const void* wsu,
                                const void* wsd, const float* gate, void* act, void* act_s, float* out, int dtype, int T, int D, int F,
                                int Fs, int top, int kind, int onto, cudaStream_t stream) {
     if (T <= 0) return 0;
@@ -269,10 +273,11 @@ extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, co
     if (kind != QWB_MOE_GATED && !qwb_activation_known(kind)) return qwb_fail(QWB_ERR_ARG, "moe_experts: unknown activation %d", kind);
     if ((long long)T * top + T > 65535 || ((long long)T * top + T) * ((F > Fs ? F : Fs) / 8 + 1) > 0x7fffffffLL)
         return qwb_fail(QWB_ERR_ARG, "moe_experts: %d tokens x %d choices are too many for one launch", T, top);
+    const float *weight_in = on_input ? weight : nullptr, *weight_out = on_input ? nullptr : weight;
     if (dtype == QWB_DT_F32)
-        launch_moe_experts<float>(x, wu, wd, chosen, weight, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
+        launch_moe_experts<float>(x, wu, wd, chosen, weight_in, weight_out, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
     else if (dtype == QWB_DT_BF16)
-        launch_moe_experts<bf16>(x, wu, wd, chosen, weight, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
+        launch_moe_experts<bf16>(x, wu, wd, chosen, weight_in, weight_out, wsu, wsd, gate, act, act_s, out, T, D, F, Fs, top, kind, onto, stream);
     else return qwb_fail(QWB_ERR_ARG, "moe_experts: unknown dtype %d", dtype);
     return qwb_check_launch("moe_experts");
 }
@@ -280,8 +285,8 @@ extern "C" int qwb_moe_experts(const void* x, const void* wu, const void* wd, co
 // ---------------------------------------------------------------------------------
 // Around a grouped product over token copies sorted by expert (bfloat16; D and F multiples of 8):
 //   moe_sort      place[c] = the row of copy c = t * top + k in the order (expert, copy); ends[e] = where expert e's run ends
-//   moe_spread    xs[place[t, k], :] = x[t, :]
-//   moe_act       act[s, f] = f(u[s, f]), u [S, F], or silu(u[s, f]) * u[s, F + f], u [S, 2F]
+//   moe_spread    xs[place[t, k], :] = x[t, :], and row_weight[place[t, k]] = weight[t, k] where the weights are on the inputs
+//   moe_act       act[s, f] = f(u[s, f]), u [S, F], or silu(u[s, f]) * u[s, F + f], u [S, 2F]; u times row_weight[s] if given
 //   moe_combine   out[t, :] (+)= sum_k weight[t, k] * y[place[t, k], :] + gate[t] * shared[t, :]
 // ---------------------------------------------------------------------------------
 // A block per expert: it counts the copies of lower experts (where its own run starts) and ranks its own ones.  Each warp
@@ -338,20 +343,24 @@ extern "C" int qwb_moe_sort(const int* chosen, int* place, int* ends, int S, int
     return qwb_check_launch("moe_sort");
 }
 
-__global__ void moe_spread_kernel(const uint4* __restrict__ x, const int* __restrict__ place, uint4* __restrict__ xs, int pieces, int top) {
+__global__ void moe_spread_kernel(const uint4* __restrict__ x, const int* __restrict__ place, uint4* __restrict__ xs, const float* __restrict__ weight,
+                                  float* __restrict__ row_weight, int pieces, int top) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
+    if (row_weight && (int)threadIdx.x < top) row_weight[place[(size_t)t * top + threadIdx.x]] = weight[(size_t)t * top + threadIdx.x];
     for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
         const uint4 v = x[(size_t)t * pieces + i];
         for (int k = 0; k < top; ++k) xs[(size_t)place[(size_t)t * top + k] * pieces + i] = v;
     }
 }
 
-extern "C" int qwb_moe_spread(const void* x, const int* place, void* xs, int T, int D, int top, cudaStream_t stream) {
+// weight [T, top] and row_weight [T * top], or both null
+extern "C" int qwb_moe_spread(const void* x, const int* place, void* xs, const float* weight, float* row_weight, int T, int D, int top,
+                              cudaStream_t stream) {
     if (T <= 0 || D <= 0) return 0;
     if (D % 8) return qwb_fail(QWB_ERR_ARG, "moe_spread: rows of %d values", D);
-    qwb_launch(moe_spread_kernel, T, D >= 2048 ? 256 : 128, 0, stream, (const uint4*)x, place, (uint4*)xs, D / 8, top);
+    qwb_launch(moe_spread_kernel, T, D >= 2048 ? 256 : 128, 0, stream, (const uint4*)x, place, (uint4*)xs, weight, row_weight, D / 8, top);
     return qwb_check_launch("moe_spread");
 }
 
@@ -368,34 +377,36 @@ __device__ __forceinline__ uint4 pack_bf16x8(const float* v) {
 
 // 8 values a thread and step, whatever row they are in; KIND: the activation code
 template <int KIND>
-__global__ void moe_act_kernel(const Vec16<bf16>* __restrict__ u, uint4* __restrict__ act, unsigned n, unsigned pieces) {
+__global__ void moe_act_kernel(const Vec16<bf16>* __restrict__ u, const float* __restrict__ row_weight, uint4* __restrict__ act, unsigned n, unsigned pieces) {
     pdl_wait();
     pdl_launch_dependents();
     for (unsigned i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
         float a[8], b[8];
+        const float w = row_weight ? row_weight[i / pieces] : 1.f;
         if (KIND == QWB_MOE_GATED) {
             const size_t gate = i + (size_t)(i / pieces) * pieces;          // row s: its gate pieces, then its up pieces
             u[gate].get(a);
             u[gate + pieces].get(b);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) a[e] = a[e] / (1.f + expf(-a[e])) * b[e];
+            for (int e = 0; e < 8; ++e) { const float g = a[e] * w; a[e] = g / (1.f + expf(-g)) * (b[e] * w); }
         } else {
             u[i].get(a);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) a[e] = qwb_activate(a[e], KIND);
+            for (int e = 0; e < 8; ++e) a[e] = qwb_activate(a[e] * w, KIND);
         }
         act[i] = pack_bf16x8(a);
     }
 }
 
-extern "C" int qwb_moe_act(const void* u, void* act, int S, int F, int kind, cudaStream_t stream) {
+// row_weight [S] or null
+extern "C" int qwb_moe_act(const void* u, const float* row_weight, void* act, int S, int F, int kind, cudaStream_t stream) {
     if (S <= 0 || F <= 0) return 0;
     if (F % 8) return qwb_fail(QWB_ERR_ARG, "moe_act: rows of %d values", F);
     const long long n = (long long)S * (F / 8);
     if (n >= 1LL << 31) return qwb_fail(QWB_ERR_ARG, "moe_act: %d rows of %d values are too many for one launch", S, F);
     const int grid = (int)((n + 255) / 256 < 148 * 32 ? (n + 255) / 256 : 148 * 32);
 #define QWB_MOE_ACT(KIND) \
-    case KIND: qwb_launch(moe_act_kernel<KIND>, grid, 256, 0, stream, (const Vec16<bf16>*)u, (uint4*)act, (unsigned)n, (unsigned)(F / 8)); break
+    case KIND: qwb_launch(moe_act_kernel<KIND>, grid, 256, 0, stream, (const Vec16<bf16>*)u, row_weight, (uint4*)act, (unsigned)n, (unsigned)(F / 8)); break
     switch (kind) {
         QWB_MOE_ACT(0); QWB_MOE_ACT(1); QWB_MOE_ACT(2); QWB_MOE_ACT(3); QWB_MOE_ACT(5); QWB_MOE_ACT(QWB_MOE_GATED);
         default: return qwb_fail(QWB_ERR_ARG, "moe_act: unknown activation %d", kind);
@@ -419,7 +430,7 @@ __global__ void moe_combine_kernel(const Vec16<bf16>* __restrict__ y, const int*
         for (int k = 0; k < top; ++k) {
             float v[8];
             y[(size_t)place[(size_t)t * top + k] * pieces + i].get(v);
-            const float w = weight[(size_t)t * top + k];
+            const float w = weight ? weight[(size_t)t * top + k] : 1.f;
 #pragma unroll
             for (int e = 0; e < 8; ++e) total[e] += w * v[e];
         }
@@ -435,7 +446,7 @@ __global__ void moe_combine_kernel(const Vec16<bf16>* __restrict__ y, const int*
     }
 }
 
-// y [S, D] bfloat16; shared [T, D] float (or null) and gate [T] (or null: 1)
+// y [S, D] bfloat16; weight [T, top] (or null: 1); shared [T, D] float (or null) and gate [T] (or null: 1)
 extern "C" int qwb_moe_combine(const void* y, const int* place, const float* weight, const float* shared, const float* gate, float* out,
                                int T, int D, int top, int onto, cudaStream_t stream) {
     if (T <= 0 || D <= 0) return 0;

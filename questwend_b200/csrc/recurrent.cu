@@ -813,12 +813,13 @@ extern "C" int qwb_retention_chunked(const float* qkv, int ld, const float* deca
 //   mode 1: out = y / rms(y over the part) * w * sigmoid(gate)          (the gate after the norm)
 //   mode 2: out = y / rms(y over the part) * w * silu(gate)
 // w has w_len entries and is indexed by column % w_len (the whole row, or one part shared by all parts).
+// divisor [T, n_parts], if given: every y is first divided by its part's number.
 // One warp per (token, part).
 // ---------------------------------------------------------------------------------
 template <typename TOut>
 __global__ void gated_part_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, int ld_gate,
-                                       const float* __restrict__ w, int w_len, TOut* __restrict__ out, int T, int n_parts,
-                                       int part, float eps, int mode) {
+                                       const float* __restrict__ w, int w_len, const float* __restrict__ divisor, TOut* __restrict__ out, int T,
+                                       int n_parts, int part, float eps, int mode) {
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31;
@@ -828,12 +829,13 @@ __global__ void gated_part_norm_kernel(const float* __restrict__ y, const float*
     const int D = n_parts * part;
     const float* yr = y + (size_t)t * D + g * part;
     const float* gr = gate + (size_t)t * ld_gate + g * part;
+    const float inv = divisor ? 1.f / divisor[unit] : 1.f;
     float ss = 0.f;
     for (int i = lane; i < part; i += 32) {
-        const float v = mode == 0 ? yr[i] * silu_f(gr[i]) : yr[i];
+        const float v = (mode == 0 ? yr[i] * silu_f(gr[i]) : yr[i]) * inv;
         ss += v * v;
     }
-    const float scale = rsqrtf(warp_sum(ss) / (float)part + eps);
+    const float scale = rsqrtf(warp_sum(ss) / (float)part + eps) * inv;
     TOut* orow = out + (size_t)t * D + g * part;
     for (int i = lane; i < part; i += 32) {
         const float wi = w[(g * part + i) % w_len];
@@ -842,7 +844,7 @@ __global__ void gated_part_norm_kernel(const float* __restrict__ y, const float*
     }
 }
 
-extern "C" int qwb_gated_part_norm(const float* y, const float* gate, int ld_gate, const float* w, int w_len, void* out,
+extern "C" int qwb_gated_part_norm(const float* y, const float* gate, int ld_gate, const float* w, int w_len, const float* divisor, void* out,
                                    int out_dtype, int T, int n_parts, int part, float eps, int mode, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (n_parts <= 0 || part <= 0 || w_len <= 0 || mode < 0 || mode > 2)
@@ -850,9 +852,9 @@ extern "C" int qwb_gated_part_norm(const float* y, const float* gate, int ld_gat
     const long long units = (long long)T * n_parts;
     const unsigned blocks = (unsigned)((units + 3) / 4);
     if (out_dtype == QWB_DT_F32)
-        qwb_launch(gated_part_norm_kernel<float>, blocks, 128, 0, stream, y, gate, ld_gate, w, w_len, (float*)out, T, n_parts, part, eps, mode);
+        qwb_launch(gated_part_norm_kernel<float>, blocks, 128, 0, stream, y, gate, ld_gate, w, w_len, divisor, (float*)out, T, n_parts, part, eps, mode);
     else if (out_dtype == QWB_DT_BF16)
-        qwb_launch(gated_part_norm_kernel<bf16>, blocks, 128, 0, stream, y, gate, ld_gate, w, w_len, (bf16*)out, T, n_parts, part, eps, mode);
+        qwb_launch(gated_part_norm_kernel<bf16>, blocks, 128, 0, stream, y, gate, ld_gate, w, w_len, divisor, (bf16*)out, T, n_parts, part, eps, mode);
     else
         return qwb_fail(QWB_ERR_ARG, "gated_part_norm: unknown dtype %d", out_dtype);
     return qwb_check_launch("gated_part_norm");

@@ -55,6 +55,16 @@ def _need(t: torch.Tensor, name: str, dtype=None, ndim=None):
         raise KernelError(f"{name}: must have {ndim} dimensions, got {t.dim()}")
 
 
+def _column_gate(what: str, gate: torch.Tensor | None, col0: int, T: int, H: int):
+    """The arguments (pointer, row stride) of a gate: columns ``col0 ..`` of the float32 matrix ``gate`` [T, ld], one a head."""
+    if gate is None:
+        return _ptr(None), _i(0)
+    _need(gate, "gate", torch.float32, 2)
+    if gate.shape[0] != T or col0 < 0 or col0 + H > gate.shape[1]:
+        raise KernelError(f"{what}: gate {tuple(gate.shape)} from column {col0} for {T} tokens of {H} heads")
+    return ctypes.c_void_p(gate.data_ptr() + 4 * col0), _i(gate.shape[1])
+
+
 LAUNCHES = [0]          # kernels of this library launched so far (through these entry points)
 
 
@@ -1029,11 +1039,12 @@ def gla_scan(qkv: torch.Tensor, a_raw: torch.Tensor, a_bias: torch.Tensor | None
 
 
 def gated_part_norm(y: torch.Tensor, gate: torch.Tensor, gate_col0: int, weight: torch.Tensor, n_parts: int, eps: float,
-                    gate_first: bool, out_dtype: torch.dtype, gate_activation: str = "sigmoid") -> torch.Tensor:
+                    gate_first: bool, out_dtype: torch.dtype, gate_activation: str = "sigmoid",
+                    divisor: torch.Tensor | None = None) -> torch.Tensor:
     """RMS norm over ``n_parts`` equal parts of every row of float32 ``y`` [T, D], with a gate from columns
     ``gate_col0 ..`` of float32 ``gate`` [T, ld].  ``gate_first``: y * silu(gate) is normed, times the weight; else y is
     normed, times the weight, times sigmoid(gate) (or silu(gate): ``gate_activation`` "silu").  ``weight`` has D entries,
-    or D / n_parts shared by all parts."""
+    or D / n_parts shared by all parts.  ``divisor`` float32 [T, n_parts]: every y is first divided by its part's number."""
     if gate_activation not in ("sigmoid", "silu"):
         raise KernelError(f"gated_part_norm: unknown gate activation '{gate_activation}'")
     _need(y, "y", torch.float32, 2)
@@ -1043,11 +1054,63 @@ def gated_part_norm(y: torch.Tensor, gate: torch.Tensor, gate_col0: int, weight:
     if D % n_parts or weight.numel() not in (D, D // n_parts) or gate_col0 + D > gate.shape[1] or gate.shape[0] != T:
         raise KernelError(f"gated_part_norm: y {tuple(y.shape)} in {n_parts} parts, weight of {weight.numel()}, gate "
                           f"{tuple(gate.shape)} from column {gate_col0}")
+    if divisor is not None:
+        _need(divisor, "divisor", torch.float32, 2)
+        if tuple(divisor.shape) != (T, n_parts):
+            raise KernelError(f"gated_part_norm: divisor {tuple(divisor.shape)} for {T} rows of {n_parts} parts")
     out = torch.empty((T, D), dtype=out_dtype, device=y.device)
     _call("recurrent", "qwb_gated_part_norm", _ptr(y), ctypes.c_void_p(gate.data_ptr() + 4 * gate_col0), _i(gate.shape[1]),
-          _ptr(weight), _i(weight.numel()), _ptr(out), _i(_dt(out_dtype)), _i(T), _i(n_parts), _i(D // n_parts), _f(eps),
+          _ptr(weight), _i(weight.numel()), _ptr(divisor), _ptr(out), _i(_dt(out_dtype)), _i(T), _i(n_parts), _i(D // n_parts), _f(eps),
           _i(0 if gate_first else (2 if gate_activation == "silu" else 1)), _stream())
     return out
+
+
+# ----------------------------------------------------------------------------- matrix memory with exponential gates
+MLSTM_CHUNKED_FROM = 64         # steps whose longest sequence brings at least this many tokens take the chunked form
+
+
+def mlstm_scan(proj: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tensor, f_bias: torch.Tensor, gate_cap: float,
+               state: torch.Tensor, m_state: torch.Tensor, ctx, heads: int, key_dim: int, vdim: int, q_scale: float, tiny: float,
+               write_state: bool = True, chunked: bool | None = None):
+    """The mLSTM's matrix memory over a step's tokens (csrc/mlstm.cu).  ``proj`` float32 [T, ld]: columns q [heads * key_dim] |
+    k [heads * key_dim] | v [heads * vdim] from 0 on, the raw input gates from ``i_col``, the raw forget gates from ``f_col``;
+    ``i_bias``, ``f_bias`` float32 [heads].  ``state`` float32 [slots, heads, vdim + 1, key_dim] (column by column, the last one
+    the normaliser) and ``m_state`` float32 [slots, heads, vdim + 1] (the running maximum, once per column) are read and written
+    back.  Returns (raw float32 [T, heads * vdim], the memory read out by q * ``q_scale``; divisor float32 [T, heads],
+    max(|n . q|, e^-m) + ``tiny``): the output is raw / divisor."""
+    _need(proj, "proj", torch.float32, 2)
+    _need(state, "state", torch.float32, 4)
+    _need(m_state, "m_state", torch.float32, 3)
+    T, ld = proj.shape
+    n_qkv = heads * (2 * key_dim + vdim)
+    if (min(i_col, f_col) < n_qkv or max(i_col, f_col) + heads > ld or tuple(state.shape[1:]) != (heads, vdim + 1, key_dim)
+            or tuple(m_state.shape) != tuple(state.shape[:3])):
+        raise KernelError(f"mlstm_scan: rows of {ld} with gates at {i_col} and {f_col}, state {tuple(state.shape)}, maxima "
+                          f"{tuple(m_state.shape)} do not fit {heads} heads of {key_dim} x {vdim}")
+    for name, t in (("i_bias", i_bias), ("f_bias", f_bias)):
+        _need(t, name, torch.float32, 1)
+        if t.numel() != heads:
+            raise KernelError(f"mlstm_scan: {name} of {t.numel()} for {heads} heads")
+    dev = proj.device
+    raw = torch.empty((T, heads * vdim), dtype=torch.float32, device=dev)
+    divisor = torch.empty((T, heads), dtype=torch.float32, device=dev)
+    single = ctx.single_token and T == ctx.n_seqs
+    gate_rows = None if single else torch.empty((3, T, heads), dtype=torch.float32, device=dev)
+    if chunked is None:
+        chunked = ctx.max_new >= MLSTM_CHUNKED_FROM
+    inputs = (_ptr(proj), _i(ld), _i(i_col), _i(f_col), _ptr(i_bias), _ptr(f_bias), _f(gate_cap), _ptr(state), _ptr(m_state),
+              _ptr(ctx.cu_seqlens), _ptr(ctx.slots), _ptr(gate_rows))
+    if chunked and not single:
+        lib = _lookup("mlstm", "qwb_mlstm_scratch_floats")[0]
+        lib.qwb_mlstm_scratch_floats.restype = ctypes.c_longlong
+        scratch = torch.empty((lib.qwb_mlstm_scratch_floats(_i(ctx.n_seqs), _i(ctx.max_new), _i(heads), _i(key_dim), _i(vdim)),),
+                              dtype=torch.float32, device=dev)
+        _call("mlstm", "qwb_mlstm_chunked", *inputs, _ptr(scratch), _ptr(raw), _ptr(divisor), _i(T), _i(ctx.n_seqs), _i(ctx.max_new),
+              _i(heads), _i(key_dim), _i(vdim), _f(q_scale), _f(tiny), _i(1 if write_state else 0), _stream(), kernels=4)
+    else:
+        _call("mlstm", "qwb_mlstm_scan", *inputs, _ptr(raw), _ptr(divisor), _i(T), _i(ctx.n_seqs), _i(heads), _i(key_dim), _i(vdim),
+              _f(q_scale), _f(tiny), _i(1 if single else 0), _i(1 if write_state else 0), _stream(), kernels=1 if single else 2)
+    return raw, divisor
 
 
 # ----------------------------------------------------------------------------- real-gated linear recurrent unit
@@ -1209,20 +1272,21 @@ def maps_prep(qkv: torch.Tensor, bias, q_weight, k_weight, cos, sin, ctx, page_t
               n_kv_heads: int, maps: int, dim: int, vdim: int, rotary_dim: int, interleaved: bool, eps: float,
               store_kv: bool = True, whole_norm: bool = False, temp_coef: float = 0.0, temp_every: float = 1.0) -> torch.Tensor:
     """Bias (float32 over all columns, or None), per-map RMS norm of q and k (weights [dim] shared by heads and maps, or
-    None), rotation of the first ``rotary_dim`` values of every map of q and k, cache write.  ``qkv`` float32
-    [T, (H + G) * maps * dim + G * vdim]; the pools [pages, G, 64, maps * dim] / [pages, G, 64, vdim].  Returns q
+    None), rotation of the first ``rotary_dim`` values of every map of q and k, cache write.  ``qkv`` float32 [T, ld] whose
+    first (H + G) * maps * dim + G * vdim columns are q | k | v; the pools [pages, G, 64, maps * dim] / [pages, G, 64, vdim].  Returns q
     [T, H, maps * dim] in the cache's dtype.  ``whole_norm``: one norm over all of q (weights [H * maps * dim]) and one over
     all of k ([G * maps * dim]) instead; with it q is multiplied by 1 + ``temp_coef`` ln(floor((p + 1) / ``temp_every``) + 1)
     at position p."""
     _need(qkv, "qkv", torch.float32, 2)
     T = qkv.shape[0]
-    ld = (n_heads + n_kv_heads) * maps * dim + n_kv_heads * vdim
-    if qkv.shape[1] != ld:
+    n_cols = (n_heads + n_kv_heads) * maps * dim + n_kv_heads * vdim
+    ld = qkv.shape[1]
+    if ld < n_cols:
         raise KernelError(f"maps_prep: qkv {tuple(qkv.shape)} for {n_heads}+{n_kv_heads} heads of {maps} x {dim}, values of {vdim}")
     if tuple(k_pool.shape[1:]) != (n_kv_heads, PAGE_SIZE, maps * dim) or tuple(v_pool.shape[1:]) != (n_kv_heads, PAGE_SIZE, vdim):
         raise KernelError(f"maps_prep: pools {tuple(k_pool.shape)}, {tuple(v_pool.shape)} do not fit")
     norm_sizes = (n_heads * maps * dim, n_kv_heads * maps * dim) if whole_norm else (dim, dim)
-    for name, t, n in (("bias", bias, ld), ("q_weight", q_weight, norm_sizes[0]), ("k_weight", k_weight, norm_sizes[1])):
+    for name, t, n in (("bias", bias, n_cols), ("q_weight", q_weight, norm_sizes[0]), ("k_weight", k_weight, norm_sizes[1])):
         if t is not None:
             _need(t, name, torch.float32, 1)
             if t.numel() != n:
@@ -1238,12 +1302,12 @@ def maps_prep(qkv: torch.Tensor, bias, q_weight, k_weight, cos, sin, ctx, page_t
                 raise KernelError(f"maps_prep: table {name} {tuple(t.shape)} for {T} tokens and {rotary_dim} turned values")
     q = torch.empty((T, n_heads, maps * dim), dtype=k_pool.dtype, device=qkv.device)
     if whole_norm:
-        _call("attention_maps", "qwb_maps_row_prep", _ptr(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos), _ptr(sin),
+        _call("attention_maps", "qwb_maps_row_prep", _ptr(qkv), _i(ld), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos), _ptr(sin),
               _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(page_table), _i(page_table.shape[1]), _ptr(q), _ptr(k_pool), _ptr(v_pool),
               _i(_dt(k_pool.dtype)), _i(T), _i(n_heads), _i(n_kv_heads), _i(maps), _i(dim), _i(vdim), _i(rotary_dim),
               _i(1 if interleaved else 0), _f(eps), _f(temp_coef), _f(temp_every), _i(1 if store_kv else 0), _stream())
         return q
-    _call("attention_maps", "qwb_maps_prep", _ptr(qkv), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos), _ptr(sin),
+    _call("attention_maps", "qwb_maps_prep", _ptr(qkv), _i(ld), _ptr(bias), _ptr(q_weight), _ptr(k_weight), _ptr(cos), _ptr(sin),
           _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(page_table), _i(page_table.shape[1]), _ptr(q), _ptr(k_pool), _ptr(v_pool),
           _i(_dt(k_pool.dtype)), _i(T), _i(n_heads), _i(n_kv_heads), _i(maps), _i(dim), _i(vdim), _i(rotary_dim),
           _i(1 if interleaved else 0), _f(eps), _i(1 if store_kv else 0), _stream())
@@ -1259,11 +1323,13 @@ def maps_prefill_mma_fits(dtype: torch.dtype, maps: int, dim: int, vdim: int) ->
 
 def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, scale: float, softcap: float = 0.0,
                    chunk: int = 0, lam: float = 0.0, norm_out: bool = False, eps: float = 0.0, out_scale: float = 1.0,
-                   impl: str = "auto") -> torch.Tensor:
+                   impl: str = "auto", window: int = 0, gate: torch.Tensor | None = None, gate_col0: int = 0) -> torch.Tensor:
     """Attention of a step's tokens with ``maps`` score maps per head over the same values.  ``q`` [T, H, maps * dim] in
     the cache's dtype; returns [T, H * vdim] in that dtype: map 0's output, minus ``lam`` times map 1's if there are two,
     then (``norm_out``) divided by its root mean square over vdim and multiplied by ``out_scale``.  Scores are scaled,
-    soft-capped (``softcap`` > 0) and masked causally, and to the query's chunk of ``chunk`` positions if that is > 0.
+    soft-capped (``softcap`` > 0) and masked causally, to the query's chunk of ``chunk`` positions if that is > 0, and to
+    the last ``window`` positions if that is > 0.  ``gate``: head h's output times the sigmoid of column ``gate_col0 + h`` of
+    the float32 matrix ``gate`` [T, ld].
     One uncapped map in bfloat16 with keys and values of up to 128 (multiples of 8) is plain grouped-query attention and
     takes its kernels (``impl`` "auto" or "tc"): in steps of one token per sequence the tensor-core decode kernel (all keys
     visible), in others the tcgen05 one.  Else steps of one token per sequence take the kernel for maps that cuts the keys
@@ -1277,31 +1343,34 @@ def maps_attention(q: torch.Tensor, k_pool, v_pool, page_table, ctx, maps: int, 
     dim = kdim // maps
     out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
     width = page_table.shape[1]
-    one_map = (maps == 1 and softcap <= 0.0 and not norm_out and impl in ("auto", "tc")
+    gate_args = _column_gate("maps_attention", gate, gate_col0, T, H)
+    one_map = (maps == 1 and softcap <= 0.0 and not norm_out and gate is None and not (chunk and window) and impl in ("auto", "tc")
                and part_attention_fits(q.dtype, dim, vdim, k_pool.shape[2], H // G))
     if ctx.single_token and one_map and chunk == 0:
-        return attn_decode(q, k_pool, v_pool, page_table, ctx.seq_len, scale, ctx.max_len, impl="mma")
+        return attn_decode(q, k_pool, v_pool, page_table, ctx.seq_len, scale, ctx.max_len, window=window, impl="mma")
     if ctx.single_token and dim % MAPS_FAST_STEP == 0 and vdim % MAPS_FAST_STEP == 0:
         lib = _lookup("attention_maps", "qwb_maps_decode_runs")[0]
-        n_runs = lib.qwb_maps_decode_runs(_i(ctx.max_len), _i(chunk))
+        n_runs = lib.qwb_maps_decode_runs(_i(ctx.max_len), _i(chunk), _i(window))
         lib.qwb_maps_decode_scratch_floats.restype = ctypes.c_longlong
         scratch = torch.empty((lib.qwb_maps_decode_scratch_floats(_i(T), _i(H), _i(maps), _i(vdim), _i(n_runs)),),
                               dtype=torch.float32, device=q.device)
         _call("attention_maps", "qwb_maps_decode", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), _ptr(ctx.seq_len),
               _ptr(scratch), _ptr(out), _i(_dt(q.dtype)), _i(T), _i(H), _i(G), _i(maps), _i(dim), _i(vdim), _i(width), _f(scale),
-              _f(softcap), _i(chunk), _i(n_runs), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), _stream(), kernels=2)
+              _f(softcap), _i(chunk), _i(window), _i(n_runs), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), *gate_args,
+              _stream(), kernels=2)
         return out
     # one map, no cap: the prompt kernel of plain grouped-query attention, with the chunk mask
     if one_map and ctx.max_new * (H // G) >= 64:
-        return attn_prefill(q, k_pool, v_pool, page_table, ctx.cu_seqlens, ctx.pos0, ctx.max_new, scale, impl="tc", chunk=chunk)
+        return attn_prefill(q, k_pool, v_pool, page_table, ctx.cu_seqlens, ctx.pos0, ctx.max_new, scale, window=window, impl="tc",
+                            chunk=chunk)
     if impl == "mma" or (impl == "auto" and maps_prefill_mma_fits(q.dtype, maps, dim, vdim)):
         _call("attention_maps", "qwb_maps_prefill_mma", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), _ptr(ctx.cu_seqlens),
               _ptr(ctx.pos0), _ptr(out), _i(ctx.n_seqs), _i(ctx.max_new), _i(H), _i(G), _i(maps), _i(dim), _i(vdim), _i(width),
-              _f(scale), _f(softcap), _i(chunk), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), _stream())
+              _f(scale), _f(softcap), _i(chunk), _i(window), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), *gate_args, _stream())
         return out
     _call("attention_maps", "qwb_maps_prefill", _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(page_table), _ptr(ctx.cu_seqlens),
           _ptr(ctx.pos0), _ptr(out), _i(_dt(q.dtype)), _i(ctx.n_seqs), _i(ctx.max_new), _i(H), _i(G), _i(maps), _i(dim), _i(vdim),
-          _i(width), _f(scale), _f(softcap), _i(chunk), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), _stream())
+          _i(width), _f(scale), _f(softcap), _i(chunk), _i(window), _f(lam), _i(1 if norm_out else 0), _f(eps), _f(out_scale), *gate_args, _stream())
     return out
 
 
@@ -1462,17 +1531,21 @@ LATENT_MAX_ROW = 1024       # ... QWB_LATENT_MAX_ROW: latent + rotated key part
 LATENT_RUN_KEYS = 64        # ... QWB_LATENT_RUN_KEYS: keys per block in a step of one token per sequence
 
 
-def latent_prep(q: torch.Tensor, dkv: torch.Tensor, c_weight: torch.Tensor, cos, sin, ctx, page_table, pool,
-                heads: int, dim: int, rot_dim: int, rank: int, eps: float, store: bool = True, whole_heads: bool = False):
+def latent_prep(q: torch.Tensor, dkv: torch.Tensor | None, c_weight: torch.Tensor | None, cos, sin, ctx, page_table, pool,
+                heads: int, dim: int, rot_dim: int, rank: int, eps: float, store: bool = True, whole_heads: bool = False,
+                dkv_col0: int = 0):
     """Per token: the latent (``dkv[:, :rank]``, RMS-normed, times ``c_weight``) and the rotated shared key part
     (``dkv[:, rank:]``, pairs (2i, 2i + 1) turned by cos/sin [T, half]) go into the cache row of the token's position;
-    each head's rotated query part is turned the same way.  ``q`` float32 [T, heads * (dim + rot_dim)].
+    each head's rotated query part is turned the same way.  ``q`` float32 [T, >= heads * (dim + rot_dim)] (the first columns);
+    ``dkv`` float32 [T, ld], from column ``dkv_col0`` on, or None: a layer that reads another layer's rows prepares its
+    queries only (no rows with ``whole_heads``).
     Returns (q_plain [heads, T, dim] in the pool's dtype, q_rot float32 [T, heads, rot_dim]); or, with ``whole_heads``
     (for the tensor-core prompt kernel), (q [T, heads, dim + rot_dim] with the rotated parts turned, the tokens' cache
     rows once more as [T, rank + rot_dim]), both in the pool's dtype."""
     _need(q, "q", torch.float32, 2)
-    _need(dkv, "dkv", torch.float32, 2)
-    _need(c_weight, "c_weight", torch.float32, 1)
+    if dkv is not None:
+        _need(dkv, "dkv", torch.float32, 2)
+        _need(c_weight, "c_weight", torch.float32, 1)
     _need(pool, "pool", ndim=4)
     _need(page_table, "page_table", torch.int32, 2)
     T = q.shape[0]
@@ -1483,18 +1556,20 @@ def latent_prep(q: torch.Tensor, dkv: torch.Tensor, c_weight: torch.Tensor, cos,
         half = cos.shape[1]
         if cos.shape[0] != T or sin.shape != cos.shape or 2 * half > rot_dim:
             raise KernelError(f"latent_prep: cos/sin {tuple(cos.shape)} do not fit {T} tokens and {rot_dim} rotated values")
-    if (q.shape[1] != heads * (dim + rot_dim) or tuple(dkv.shape) != (T, rank + rot_dim) or c_weight.numel() != rank
+    if (q.shape[1] < heads * (dim + rot_dim)
+            or (dkv is not None and (dkv.shape[0] != T or dkv_col0 < 0 or dkv_col0 + rank + rot_dim > dkv.shape[1] or c_weight.numel() != rank))
             or pool.shape[1] != 1 or pool.shape[3] != rank + rot_dim):
-        raise KernelError(f"latent_prep: q {tuple(q.shape)}, dkv {tuple(dkv.shape)}, pool {tuple(pool.shape)} do not fit "
+        raise KernelError(f"latent_prep: q {tuple(q.shape)}, dkv {None if dkv is None else tuple(dkv.shape)}, pool {tuple(pool.shape)} do not fit "
                           f"{heads} heads of {dim} + {rot_dim}, latent {rank}")
     q_plain = q_rot = q_full = row_new = None
     if whole_heads:
         q_full = torch.empty((T, heads, dim + rot_dim), dtype=pool.dtype, device=q.device)
-        row_new = torch.empty((T, rank + rot_dim), dtype=pool.dtype, device=q.device)
+        row_new = torch.empty((T, rank + rot_dim), dtype=pool.dtype, device=q.device) if dkv is not None else None
     else:
         q_plain = torch.empty((heads, T, dim), dtype=pool.dtype, device=q.device)
         q_rot = torch.empty((T, heads, rot_dim), dtype=torch.float32, device=q.device)
-    _call("attention_latent", "qwb_latent_prep", _ptr(q), _ptr(dkv), _ptr(c_weight), _ptr(cos), _ptr(sin), _ptr(ctx.tok_seq),
+    _call("attention_latent", "qwb_latent_prep", _ptr(q), _i(q.shape[1]),
+          ctypes.c_void_p(dkv.data_ptr() + 4 * dkv_col0) if dkv is not None else _ptr(None), _i(dkv.shape[1] if dkv is not None else 0), _ptr(c_weight), _ptr(cos), _ptr(sin), _ptr(ctx.tok_seq),
           _ptr(ctx.tok_pos), _ptr(page_table), _ptr(pool), _i(_dt(pool.dtype)), _ptr(q_plain), _ptr(q_rot), _ptr(q_full),
           _ptr(row_new), _i(T), _i(heads), _i(dim), _i(rot_dim), _i(rank), _i(half), _f(eps), _i(pool.shape[2]),
           _i(page_table.shape[1]), _i(1 if store else 0), _stream())
@@ -1509,11 +1584,13 @@ def latent_prefill_fits(dtype: torch.dtype, dim: int, rot_dim: int, vdim: int, r
 
 
 def latent_prefill(q: torch.Tensor, k_plain: torch.Tensor, rows: torch.Tensor, v: torch.Tensor, ctx, sink, scale: float,
-                   window: int, heads: int, dim: int, rot_dim: int, vdim: int) -> torch.Tensor:
+                   window: int, heads: int, dim: int, rot_dim: int, vdim: int, gate: torch.Tensor | None = None,
+                   gate_col0: int = 0) -> torch.Tensor:
     """Attention of prompts that START their sequences (every position 0 is in this step), on the tensor cores.
     bfloat16: ``q`` [T, heads, dim + rot_dim]; ``k_plain`` [T, heads * dim] and ``v`` [T, heads * vdim], the keys' unrotated
     parts and the values made from the latents; ``rows`` [T, rank + rot_dim], whose last ``rot_dim`` values are the
-    rotated key part that the heads share.  Returns [T, heads * vdim]."""
+    rotated key part that the heads share.  ``gate``: head h's output times the sigmoid of column ``gate_col0 + h`` of the
+    float32 matrix ``gate`` [T, ld].  Returns [T, heads * vdim]."""
     for name, t in (("q", q), ("k_plain", k_plain), ("rows", rows), ("v", v)):
         _need(t, name, torch.bfloat16)
     T = q.shape[0]
@@ -1526,7 +1603,19 @@ def latent_prefill(q: torch.Tensor, k_plain: torch.Tensor, rows: torch.Tensor, v
     ld = rows.shape[1]
     _call("attention_latent_mma", "qwb_latent_prefill_mma", _ptr(q), _ptr(k_plain),
           ctypes.c_void_p(rows.data_ptr() + 2 * (ld - rot_dim)), _i(ld), _ptr(v), _ptr(ctx.cu_seqlens), _ptr(sink), _ptr(out),
-          _i(ctx.n_seqs), _i(ctx.max_new), _i(heads), _i(dim), _i(rot_dim), _i(vdim), _f(scale), _i(window), _stream())
+          _i(ctx.n_seqs), _i(ctx.max_new), _i(heads), _i(dim), _i(rot_dim), _i(vdim), _f(scale), _i(window),
+          *_column_gate("latent_prefill", gate, gate_col0, T, heads), _stream())
+    return out
+
+
+def latent_heads_out(values: torch.Tensor, dtype: torch.dtype, gate: torch.Tensor | None = None, gate_col0: int = 0) -> torch.Tensor:
+    """Float32 ``values`` [heads, T, vdim] -> [T, heads * vdim] in ``dtype``, head h's times the sigmoid of column
+    ``gate_col0 + h`` of the float32 matrix ``gate`` [T, ld] if that is given."""
+    _need(values, "values", torch.float32, 3)
+    H, T, P = values.shape
+    out = torch.empty((T, H * P), dtype=dtype, device=values.device)
+    _call("attention_latent", "qwb_latent_heads_out", _ptr(values), *_column_gate("latent_heads_out", gate, gate_col0, T, H), _ptr(out),
+          _i(_dt(dtype)), _i(T), _i(H), _i(P), _stream())
     return out
 
 
@@ -1613,8 +1702,8 @@ def _moe_sizes(what, x, w_up, w_down, chosen, weight, kind):
 
 def moe_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor, weight: torch.Tensor,
                 activation: str = "gated_silu", shared_up: torch.Tensor | None = None, shared_down: torch.Tensor | None = None,
-                gate: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
-    """sum_k weight[t, k] * down_e(act(up_e x_t)), e = chosen[t, k].  ``x`` [T, D] and the stacked weights (``w_up``
+                gate: torch.Tensor | None = None, out: torch.Tensor | None = None, weight_on_input: bool = False) -> torch.Tensor:
+    """sum_k weight[t, k] * down_e(act(up_e x_t)), e = chosen[t, k] (``weight_on_input``: sum_k down_e(act(up_e (weight[t, k] x_t)))).  ``x`` [T, D] and the stacked weights (``w_up``
     [E, F, D]; "gated_silu": [E, 2F, D], gate rows, then up rows, silu(gate x) * up x; ``w_down`` [E, D, F]) in one dtype.
     A shared expert (``shared_up`` [Fs, D], ``shared_down`` [D, Fs], the same activation, plain) is added for every token,
     times ``gate`` [T] if given.  Returns float32 [T, D], or adds onto ``out`` if that is given."""
@@ -1641,7 +1730,7 @@ def moe_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chose
     for t0 in range(0, T, per):
         n = min(per, T - t0)
         cut = (lambda t: None if t is None else t[t0:t0 + n])
-        _call("moe", "qwb_moe_experts", _ptr(cut(x)), _ptr(w_up), _ptr(w_down), _ptr(cut(chosen)), _ptr(cut(weight)), _ptr(shared_up),
+        _call("moe", "qwb_moe_experts", _ptr(cut(x)), _ptr(w_up), _ptr(w_down), _ptr(cut(chosen)), _ptr(cut(weight)), _i(1 if weight_on_input else 0), _ptr(shared_up),
               _ptr(shared_down), _ptr(cut(gate)), _ptr(act[t0 * top:(t0 + n) * top]), _ptr(cut(act_s)), _ptr(cut(out)), _i(_dt(x.dtype)),
               _i(n), _i(D), _i(F), _i(Fs), _i(top), _i(MOE_ACTIVATIONS[activation]), _i(1 if onto else 0), _stream(), kernels=2)
     return out
@@ -1669,7 +1758,7 @@ def moe_sort(chosen: torch.Tensor, experts: int):
 
 def moe_experts_grouped(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor, weight: torch.Tensor,
                         activation: str = "gated_silu", shared: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                        out: torch.Tensor | None = None) -> torch.Tensor:
+                        out: torch.Tensor | None = None, weight_on_input: bool = False) -> torch.Tensor:
     """``moe_experts`` for many bfloat16 tokens: the tokens' copies are sorted by expert (in an order that does not depend
     on which blocks finish first), each expert's run goes through the library's grouped matrix product (32-bit sums,
     bfloat16 results) for up and for down, with the activation between them and the weighted sum of every token's copies
@@ -1685,15 +1774,16 @@ def moe_experts_grouped(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tenso
                 raise KernelError(f"moe_experts_grouped: {name} {tuple(t.shape)}, wanted {shape}")
     place, ends = moe_sort(chosen, E)
     xs = torch.empty((T * top, D), dtype=torch.bfloat16, device=x.device)
-    _call("moe", "qwb_moe_spread", _ptr(x), _ptr(place), _ptr(xs), _i(T), _i(D), _i(top), _stream())
+    row_weight = torch.empty((T * top,), dtype=torch.float32, device=x.device) if weight_on_input else None
+    _call("moe", "qwb_moe_spread", _ptr(x), _ptr(place), _ptr(xs), _ptr(weight if weight_on_input else None), _ptr(row_weight), _i(T), _i(D), _i(top), _stream())
     u = torch._grouped_mm(xs, w_up.transpose(1, 2), offs=ends).contiguous()
     act = torch.empty((T * top, F), dtype=torch.bfloat16, device=x.device)
-    _call("moe", "qwb_moe_act", _ptr(u), _ptr(act), _i(T * top), _i(F), _i(MOE_ACTIVATIONS[activation]), _stream())
+    _call("moe", "qwb_moe_act", _ptr(u), _ptr(row_weight), _ptr(act), _i(T * top), _i(F), _i(MOE_ACTIVATIONS[activation]), _stream())
     y = torch._grouped_mm(act, w_down.transpose(1, 2), offs=ends).contiguous()
     onto = out is not None
     if not onto:
         out = torch.empty((T, D), dtype=torch.float32, device=x.device)
-    _call("moe", "qwb_moe_combine", _ptr(y), _ptr(place), _ptr(weight), _ptr(shared), _ptr(gate), _ptr(out), _i(T), _i(D), _i(top),
+    _call("moe", "qwb_moe_combine", _ptr(y), _ptr(place), _ptr(None if weight_on_input else weight), _ptr(shared), _ptr(gate), _ptr(out), _i(T), _i(D), _i(top),
           _i(1 if onto else 0), _stream())
     return out
 

@@ -13,7 +13,7 @@ from ..kernels.limits import (conv_taps_refusal, head_dim_refusal, maps_attentio
                               shaped_attention_refusal)
 from ..weights.manifest import MATRIX, NORM_WEIGHT, VECTOR, TensorSpec
 from .base import KVSpec, Mixer, StateSpec, take_weight
-from .linear import kernel_modules as linear_modules, linear, linear_onto
+from .linear import filled_rows, kernel_modules as linear_modules, linear, linear_onto
 from .registry import register_mixer
 
 FUSED_DECODE_MAX_BATCH = 16     # up to here a kernel less per layer pays (3-4 % of a small model's step); with more sequences
@@ -221,10 +221,11 @@ class ScoreMapsAttention(Mixer):
     """Grouped-query softmax attention whose heads carry ``maps`` score maps (1 or 2) over the same values.  A query head
     has ``maps`` query vectors of ``head_dim`` values laid out one after the other, a key head as many key vectors; each
     map is an attention of its own (score = q . k * ``scale``, then ``softcap`` * tanh(score / ``softcap``) if that is
-    > 0, a causal mask, and with ``chunk`` > 0 only the keys of the query's own block of ``chunk`` positions, counted
-    from the sequence's start).  With two maps the head's output is differential: a1 - lambda * a2 with
+    > 0, a causal mask, with ``chunk`` > 0 only the keys of the query's own block of ``chunk`` positions, counted
+    from the sequence's start, and with ``window`` > 0 only the last ``window`` keys, the query's own among them).  With two maps the head's output is differential: a1 - lambda * a2 with
     lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + ``diff`` (four learned vectors of the layer), divided by its root mean
-    square over the value size (eps inside the root) and multiplied by 1 - ``diff``.  In front of the scores, in this
+    square over the value size (eps inside the root) and multiplied by 1 - ``diff``.  ``head_gate``: head h's output times
+    sigmoid(W_g h)_h, one number per head, in front of the output projection.  In front of the scores, in this
     order and each optional: biases on q, k and v, a short causal convolution over time on every channel of q, k and v
     (``conv`` taps, no activation; its last inputs are per-sequence state), an RMS norm of every map of q and k with a
     weight shared by heads and maps (``qk_norm_over`` "head") or of the whole projections of q and of k with weights of
@@ -233,13 +234,14 @@ class ScoreMapsAttention(Mixer):
 
     params: hidden_size, n_heads, n_kv_heads, head_dim, value_dim, maps (default 1), biases (q, k, v), out_bias, conv
     (0: none), qk_norm, qk_norm_over (default "head"), norm_eps, q_temp_coef (0: none), q_temp_every, scale (default
-    1/sqrt(head_dim)), softcap (0: none), chunk (0: plain causal), diff, layout ("halves": pairs (i, i + n/2); "interleaved": (2i, 2i + 1)), names (optional overrides).  ``position``: an
-    encoding that gives cos and sin [T, n/2].
+    1/sqrt(head_dim)), softcap (0: none), chunk (0: plain causal), window (0: all keys), diff, head_gate, layout ("halves":
+    pairs (i, i + n/2); "interleaved": (2i, 2i + 1)), names (optional overrides).  ``position``: an encoding that gives cos
+    and sin [T, n/2].
     The cache: keys (all maps of a head in one row) and values per token; with a convolution also its tail."""
 
     NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "o_bias": "o.b",
              "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "q_norm": "q.norm", "k_norm": "k.norm",
-             "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2"}
+             "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2", "gate": "g"}
     LAYOUTS = ("halves", "interleaved")
     NORMS = ("head", "projection")
 
@@ -260,7 +262,9 @@ class ScoreMapsAttention(Mixer):
         self.scale = float(p.get("scale", 1.0 / math.sqrt(self.head_dim)))
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
         self.chunk = int(p.get("chunk", 0) or 0)
+        self.window = int(p.get("window", 0) or 0)
         self.diff = float(p.get("diff", 0.0))
+        self.head_gate = bool(p.get("head_gate", False))
         self.layout = str(p.get("layout", "halves"))
         self.names = {**self.NAMES, **dict(p.get("names", {}))}
         self.position = position[0] if isinstance(position, (tuple, list)) else position
@@ -303,6 +307,8 @@ class ScoreMapsAttention(Mixer):
                     TensorSpec(px + n["k_norm"], (self.n_k if whole else self.head_dim,), VECTOR, NORM_WEIGHT)]
         if self.maps == 2:
             out += [TensorSpec(px + n[x], (self.head_dim,), VECTOR) for x in ("lq1", "lk1", "lq2", "lk2")]
+        if self.head_gate:
+            out.append(TensorSpec(px + n["gate"], (self.n_heads, D), MATRIX))
         return out
 
     def bind(self, weights):
@@ -311,7 +317,9 @@ class ScoreMapsAttention(Mixer):
         def f32(name):
             return weights[px + n[name]].to(torch.float32).contiguous()
 
-        self.w_qkv = torch.cat([take_weight(weights, px + n[x]) for x in "qkv"], dim=0).contiguous()
+        # one projection for everything that reads the mixer's input: q | k | v | (gate)
+        mats = [take_weight(weights, px + n[x]) for x in "qkv"]
+        self.w_in = filled_rows(mats + [take_weight(weights, px + n["gate"])]) if self.head_gate else torch.cat(mats, dim=0).contiguous()
         self.w_o = weights[px + n["o"]]
         self.b_qkv = torch.cat([f32(x + "_bias") for x in "qkv"]).contiguous() if self.biases else None
         self.b_o = f32("o_bias") if self.out_bias else None
@@ -324,25 +332,25 @@ class ScoreMapsAttention(Mixer):
 
     def kernel_modules(self):
         mods = ["attention_maps", "rope_kv", "elementwise", *(("recurrent",) if self.taps else ()), *linear_modules(self.runtime.dtype)]
-        if (self.maps == 1 and self.softcap <= 0.0
+        if (self.maps == 1 and self.softcap <= 0.0 and not self.head_gate and not (self.chunk and self.window)
                 and ops.part_attention_fits(self.runtime.dtype, self.head_dim, self.value_dim, ops.PAGE_SIZE, self.n_heads // self.n_kv_heads)):
             mods.append("attention_tc")         # prompts of one uncapped map ...
             if self.chunk == 0:
-                mods.append("attention_mma")    # ... and its single tokens over all keys
+                mods.append("attention_mma")    # ... and its single tokens over all keys or a window
         return tuple(mods)
 
     def kv_spec(self):
-        return KVSpec(self.n_kv_heads, self.maps * self.head_dim, 0, value_dim=self.value_dim)
+        return KVSpec(self.n_kv_heads, self.maps * self.head_dim, self.window, value_dim=self.value_dim)
 
     def state_spec(self):
         return StateSpec((self.taps - 1, self.channels), torch.float32) if self.taps > 1 else None
 
     def forward(self, x, ctx, cache):
-        qkv = linear(x, self.w_qkv)
+        proj = qkv = linear(x, self.w_in)
         bias = self.b_qkv
         if self.taps:
             tail = cache.state if self.taps > 1 else qkv.new_zeros((1, 0, self.channels))
-            qkv = ops.short_conv(qkv, 0, self.channels, self.conv_w, None, tail, ctx, activation=False,
+            qkv = ops.short_conv(proj, 0, self.channels, self.conv_w, None, tail, ctx, activation=False,
                                  update_tail=cache.writable, in_bias=bias)
             bias = None
         cos = sin = None
@@ -355,8 +363,9 @@ class ScoreMapsAttention(Mixer):
                           whole_norm=self.norm_over == "projection", temp_coef=self.temp_coef, temp_every=self.temp_every)
         two = self.maps == 2
         att = ops.maps_attention(q, cache.k_pool, cache.v_pool, table, ctx, self.maps, self.scale, softcap=self.softcap,
-                                 chunk=self.chunk, lam=self.lam, norm_out=two, eps=self.eps,
-                                 out_scale=(1.0 - self.diff) if two else 1.0)
+                                 chunk=self.chunk, window=self.window, lam=self.lam, norm_out=two, eps=self.eps,
+                                 out_scale=(1.0 - self.diff) if two else 1.0, gate=proj if self.head_gate else None,
+                                 gate_col0=self.channels)
         out = linear(att, self.w_o)
         return ops.bias_act(out, self.b_o, "none", torch.float32) if self.b_o is not None else out
 

@@ -15,23 +15,33 @@ from .registry import build_part, register_block
 
 
 class PreNormBlock(Block):
-    """params: mixer_norm, ffn_norm (tensor-name stems of the two norms), mixer_prefix, ffn_prefix."""
+    """A layer without a feed-forward (``feed_forward`` None) has the first half only (its second norm may lie in the files).
+    params: mixer_norm, ffn_norm (tensor-name stems of the two norms), whole_names (default False; True: the norms' tensors
+    are named by the stems alone, without ".weight"), mixer_prefix, ffn_prefix."""
 
     def __init__(self, spec, runtime, layer=None, position=None):
         super().__init__(spec, runtime)
         p = spec.params
         px = spec.prefix
-        self.norm1 = build_part("norm", replace(layer.norm, prefix=px + p.get("mixer_norm", "input_layernorm") + "."), runtime)
-        self.norm2 = build_part("norm", replace(layer.norm, prefix=px + p.get("ffn_norm", "post_attention_layernorm") + "."), runtime)
+        whole = bool(p.get("whole_names", False))
+
+        def norm(stem):
+            spec = replace(layer.norm, prefix=px, params={**dict(layer.norm.params), "name": stem}) if whole else replace(layer.norm, prefix=px + stem + ".")
+            return build_part("norm", spec, runtime)
+
+        self.norm1, self.norm2 = norm(p.get("mixer_norm", "input_layernorm")), norm(p.get("ffn_norm", "post_attention_layernorm"))
         self.mixer = build_part("mixer", replace(layer.mixer, prefix=px + p.get("mixer_prefix", "self_attn") + "."),
                                 runtime, position=position)
-        self.ffn = build_part("feed_forward", replace(layer.feed_forward, prefix=px + p.get("ffn_prefix", "mlp") + "."), runtime)
+        self.ffn = None
+        if layer.feed_forward is not None:
+            self.ffn = build_part("feed_forward", replace(layer.feed_forward, prefix=px + p.get("ffn_prefix", "mlp") + "."), runtime)
 
     def parts(self):
-        return [self.norm1, self.mixer, self.norm2, self.ffn]
+        return [self.norm1, self.mixer] if self.ffn is None else [self.norm1, self.mixer, self.norm2, self.ffn]
 
     def tensors(self):
-        return [t for part in self.parts() for t in part.tensors()]
+        out = [t for part in self.parts() for t in part.tensors()]
+        return out if self.ffn is not None else out + [replace(t, ignored=True) for t in self.norm2.tensors()]
 
     def bind(self, weights):
         for part in self.parts():
@@ -46,6 +56,8 @@ class PreNormBlock(Block):
             delta = self.mixer.forward(x, ctx, cache, residual=h)
         else:
             delta = self.mixer.forward(x, ctx, cache)
+        if self.ffn is None:
+            return h, delta
         x = self.norm2.forward(h, settle(h, delta, self.norm2), write_sum=True)
         if self.ffn.adds_to_residual:
             delta = self.ffn.forward(x, ctx, residual=h)

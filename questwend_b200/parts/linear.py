@@ -94,6 +94,21 @@ def _check_true_fp32() -> None:
                            "mode was switched on after the engine was made")
 
 
+FILL_ROWS = 8           # matrices joined into one projection are filled up to a multiple of this many rows
+
+
+def filled_rows(mats) -> torch.Tensor:
+    """Matrices [n_i, K] on top of each other, and rows of zeros up to a multiple of ``FILL_ROWS``: a part with a few rows
+    (one a head) then does not leave the projection, and the rows of its result, at an odd size."""
+    rows = sum(m.shape[0] for m in mats)
+    out = mats[0].new_zeros((-(-rows // FILL_ROWS) * FILL_ROWS, mats[0].shape[1]))
+    at = 0
+    for m in mats:
+        out[at:at + m.shape[0]].copy_(m)
+        at += m.shape[0]
+    return out
+
+
 def linear(x: torch.Tensor, weight: torch.Tensor, add_to: torch.Tensor | None = None) -> torch.Tensor:
     """x [M, K] (the weight's dtype) times weight [N, K] transposed -> float32 [M, N].
     With ``add_to`` (float32 [M, N]) the product is added onto it in place and it is returned."""

@@ -22,7 +22,8 @@ class RoutedExperts(FeedForward):
     that joins the scores for the choice only), groups and groups_kept (default 1 and 1: the experts form that many groups
     of neighbours, and only the best groups, by the sum of their two largest choice scores, can be chosen from);
     renormalize (default False: the weights are the chosen experts' scores as they are; True: divided by their sum +
-    ``sum_eps``), weight_scale (default 1);
+    ``sum_eps``), weight_scale (default 1), weight_on ("output", the default: it multiplies the expert's output; "input": the
+    expert sees w * h);
     shared_size (default 0: none; the size of an ungated expert that every token uses), shared_gate (default False; True:
     its output is multiplied by sigmoid(W_sg h), one number a token);
     names (router; correction; expert: a pattern with {e}; gate, up, down; shared, shared_gate).
@@ -43,6 +44,7 @@ class RoutedExperts(FeedForward):
         self.groups, self.keep = int(p.get("groups", 1)), int(p.get("groups_kept", 1))
         self.renormalize = bool(p.get("renormalize", False))
         self.sum_eps, self.weight_scale = float(p.get("sum_eps", 0.0)), float(p.get("weight_scale", 1.0))
+        self.weight_on = str(p.get("weight_on", "output"))
         self.shared = int(p.get("shared_size", 0) or 0)
         self.shared_gate = bool(p.get("shared_gate", False)) and self.shared > 0
         self.names = {**self.NAMES, **dict(p.get("names", {}))}
@@ -51,6 +53,8 @@ class RoutedExperts(FeedForward):
             refusal = f"unknown activation '{self.activation}'; known: {', '.join(ops.MOE_ACTIVATIONS)}"
         if refusal is None and self.scores not in ops.MOE_SCORES:
             refusal = f"unknown scores '{self.scores}'; known: {', '.join(ops.MOE_SCORES)}"
+        if refusal is None and self.weight_on not in ("input", "output"):
+            refusal = f"the weights are on the experts' 'input' or 'output', not '{self.weight_on}'"
         if refusal is None and self.shared and self.gated:
             refusal = "a shared expert beside gated experts is not built"
         if refusal:
@@ -113,16 +117,17 @@ class RoutedExperts(FeedForward):
         routed = ops.moe_route(linear(x, self.w_router), self.top, self.renormalize, experts=self.experts, scores=self.scores,
                                correction=self.w_correction, groups=self.groups, keep=self.keep, sum_eps=self.sum_eps,
                                weight_scale=self.weight_scale, gate=self.shared_gate)
+        on_input = self.weight_on == "input"
         chosen, weight, gate = routed if self.shared_gate else (*routed, None)
         if ops.moe_grouped_fits(x, self.w_up, self.w_down):
             shared = None
             if self.shared:
                 shared = linear(linear_act(x, self.w_shared_up, None, self.activation, self.runtime.dtype), self.w_shared_down)
             out = ops.moe_experts_grouped(x, self.w_up, self.w_down, chosen, weight, self.activation, shared=shared, gate=gate,
-                                          out=residual)
+                                          out=residual, weight_on_input=on_input)
         else:
             out = ops.moe_experts(x, self.w_up, self.w_down, chosen, weight, self.activation, shared_up=self.w_shared_up,
-                                  shared_down=self.w_shared_down, gate=gate, out=residual)
+                                  shared_down=self.w_shared_down, gate=gate, out=residual, weight_on_input=on_input)
         return None if residual is not None else out
 
 

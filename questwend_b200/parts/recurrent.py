@@ -1,7 +1,7 @@
 """Mixers that carry a state of fixed size from token to token instead of keys and values: the state-space
 recurrence of Mamba-2, the gated delta rule with a decay per key channel or per head, gated linear attention (a decay per
 key channel, a plain outer-product write), retention (the same write with a fixed decay per head and rotated queries and
-keys), and the recurrent block around a real-gated linear recurrent unit (one number of state per channel).  All keep, per sequence, a 32-bit
+keys), the matrix memory with exponential gates of the mLSTM, and the recurrent block around a real-gated linear recurrent unit (one number of state per channel).  All keep, per sequence, a 32-bit
 state matrix per head and the last inputs of a short causal convolution, in the cache's per-slot state rows; a
 prompt and a single token run through the same kernels (``csrc/recurrent.cu``).  The projections are matrix
 products in the engine's dtype with 32-bit results; everything between them is 32-bit.
@@ -14,7 +14,7 @@ from ..kernels import ops
 from ..kernels.limits import conv_taps_refusal, state_matrix_refusal
 from ..weights.manifest import MATRIX, NORM_WEIGHT, VECTOR, TensorSpec
 from .base import Mixer, StateSpec, take_weight
-from .linear import kernel_modules as linear_modules, linear
+from .linear import filled_rows, kernel_modules as linear_modules, linear
 from .registry import register_mixer
 
 
@@ -435,7 +435,69 @@ class RetentionMixer(Mixer):
         return linear(g, self.w_out)
 
 
+class MLSTMMixer(Mixer):
+    """The matrix memory of the mLSTM.  q = W_q h * ``q_scale`` and k = W_k h (heads x key_dim), v = W_v h (heads x vdim); per
+    head a log input gate i = cap tanh((W_i h + b_i) / cap) and a log forget gate f = log sigmoid(cap tanh((W_f h + b_f) / cap)),
+    cap = ``gate_cap``.  With a running maximum m from 0, m' = max(f + m, i):  S <- e^(f + m - m') S + e^(i - m') k v^T, n the
+    same with k alone, o = S^T q / (max(|n . q|, e^-m') + ``tiny``).  Each head's o is divided by its root mean square over
+    vdim, times a weight per value, times sigmoid(W_g h); then the output projection.
+
+    params: hidden_size, heads, key_dim, vdim, gate_cap, norm_eps, q_scale (default key_dim^-1/2), tiny (default 1e-6), names
+    (optional overrides).  State per sequence: S and n, stored [heads, vdim + 1, key_dim] (n is the column of a value that is
+    always 1), and m, once per column [heads, vdim + 1]."""
+
+    NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "in_gate": "i", "in_bias": "i.b", "forget_gate": "f", "forget_bias": "f.b",
+             "norm": "norm", "out": "o"}
+
+    def __init__(self, spec, runtime, position=None):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.heads, self.key_dim, self.vdim = int(p["heads"]), int(p["key_dim"]), int(p["vdim"])
+        self.gate_cap, self.eps, self.tiny = float(p["gate_cap"]), float(p["norm_eps"]), float(p.get("tiny", 1e-6))
+        self.q_scale = float(p.get("q_scale", self.key_dim ** -0.5))
+        self.names = {**self.NAMES, **dict(p.get("names", {}))}
+        refusal = state_matrix_refusal(self.key_dim, self.vdim)
+        if refusal:
+            raise ValueError(f"mlstm '{self.prefix}': {refusal}")
+        if not self.gate_cap > 0:
+            raise ValueError(f"mlstm '{self.prefix}': gate_cap must be positive, got {self.gate_cap}")
+        self.n_qk, self.n_v = self.heads * self.key_dim, self.heads * self.vdim
+
+    def tensors(self):
+        n, px, D, H = self.names, self.prefix, self.hidden, self.heads
+        return [TensorSpec(px + n["q"], (self.n_qk, D), MATRIX), TensorSpec(px + n["k"], (self.n_qk, D), MATRIX),
+                TensorSpec(px + n["v"], (self.n_v, D), MATRIX), TensorSpec(px + n["gate"], (self.n_v, D), MATRIX),
+                TensorSpec(px + n["out"], (D, self.n_v), MATRIX), TensorSpec(px + n["norm"], (self.n_v,), VECTOR, NORM_WEIGHT),
+                TensorSpec(px + n["in_gate"], (H, D), MATRIX), TensorSpec(px + n["in_bias"], (H,), VECTOR),
+                TensorSpec(px + n["forget_gate"], (H, D), MATRIX), TensorSpec(px + n["forget_bias"], (H,), VECTOR)]
+
+    def bind(self, weights):
+        n, px = self.names, self.prefix
+        # one projection for everything that reads the mixer's input: q | k | v | gate | input gate | forget gate
+        self.w_in = filled_rows([take_weight(weights, px + n[k]) for k in ("q", "k", "v", "gate", "in_gate", "forget_gate")])
+        self.w_out = weights[px + n["out"]]
+        self.norm_w, self.b_i, self.b_f = (_f32(weights, px + n[k]) for k in ("norm", "in_bias", "forget_bias"))
+
+    def kernel_modules(self):
+        return ("mlstm", "recurrent", *linear_modules(self.runtime.dtype))
+
+    def state_spec(self):
+        return (StateSpec((self.heads, self.vdim + 1, self.key_dim), torch.float32), StateSpec((self.heads, self.vdim + 1), torch.float32))
+
+    def forward(self, x, ctx, cache):
+        state, m = cache.state
+        proj = linear(x, self.w_in)
+        at = 2 * self.n_qk + 2 * self.n_v
+        raw, divisor = ops.mlstm_scan(proj, at, at + self.heads, self.b_i, self.b_f, self.gate_cap, state, m, ctx, self.heads,
+                                      self.key_dim, self.vdim, self.q_scale, self.tiny, write_state=cache.writable)
+        g = ops.gated_part_norm(raw, proj, 2 * self.n_qk + self.n_v, self.norm_w, self.heads, self.eps, gate_first=False,
+                                out_dtype=self.runtime.dtype, divisor=divisor)
+        return linear(g, self.w_out)
+
+
 register_mixer("mamba2", Mamba2Mixer)
+register_mixer("mlstm", MLSTMMixer)
 register_mixer("gated_delta_headwise", GatedDeltaHeadMixer)
 register_mixer("retention", RetentionMixer)
 register_mixer("rglru", RGLRUMixer)
