@@ -150,6 +150,27 @@ def movudra_experts_beside(width=2048, layers=6, vocab=32768):
     return {"architecture": "Movudra", "layers": [latent] * layers, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
 
 
+def tebozen_sizes(width=2048, repeats=2, window=1024, memory=(4, 256, 512), top=6, vocab=32768):
+    """A Tebozen configuration at sizes that resemble real layers: per repeat a differential attention layer (16 heads with
+    two score maps of 64 over 4 key/value heads, values of 128, 4 taps, a window of 1,024 positions), an mLSTM layer
+    (``memory``: heads, key size, value size at width 2,048) and a latent attention layer (16 heads of 128 + 64, latent 512,
+    values of 128; from the second repeat on it reads the first one's rows), each with 64 experts of 1,408 of which a token
+    uses ``top``, and a shared expert of 2,816."""
+    mlp = {"kind": "moe", "expert": {"ff": 1408}, "router": {"experts": 64, "top": top}, "shared": {"ff": 2816}}
+    heads = width // 128
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"conv": 4, "diff": 0.8, "dim": 64, "heads": heads, "kv_heads": width // 512, "vdim": 128, "scale": 64 ** -0.5,
+                     "mask": {"size": window}, "rot": {"base": 10000.0, "dims": 64}}}
+    mem = {"type": "mlstm", "mlp": mlp, "mixer": {"dim": memory[1], "gate_cap": 15.0, "heads": memory[0] * width // 2048, "vdim": memory[2]}}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"dim": 128, "heads": heads, "kv_rank": 512, "rot_dim": 64, "vdim": 128, "scale": 192 ** -0.5,
+                     "rot": {"base": 10000.0, "dims": 64}}}
+    layers = []
+    for r in range(repeats):
+        layers += [att, mem, lat if r == 0 else {**lat, "mixer": {**lat["mixer"], "kv_from": 2}}]
+    return {"architecture": "Tebozen", "embedding": {"scale": 1.0}, "layers": layers, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+
+
 def qwen3_beside(width=2048, layers=6, vocab=32768):
     """The closest model the library had, at the same width, depth and vocabulary: Qwen3 layers with 16 heads of 128
     (8 key/value heads) and a gated feed-forward of 3 x width."""
@@ -956,6 +977,138 @@ def tufadra_kernels(torch, np, peaks) -> dict:
     return out
 
 
+def tebozen_kernels(torch, np, peaks) -> dict:
+    """The Tebozen design's kernels alone at the sizes of ``tebozen_sizes``, each beside the like kernel of a model the
+    library had, with the bytes or FLOPs it must move and the share of the measured peak that this comes to: the mLSTM's
+    memory (beside retention and gated linear attention), its norm (beside the same norm without a divisor), windowed
+    differential attention with a gate per head (beside Punolix's), latent attention with a gate (beside Movudra's), the
+    router (beside Movudra's) and the experts with weights on their inputs (beside Tufadra's)."""
+    from types import SimpleNamespace
+    from questwend_b200.cache.manager import CacheManager
+    from questwend_b200.engine.engine import StepEntry, build_step_context
+    from questwend_b200.kernels import ops
+    from questwend_b200.parts.base import KVSpec
+    dev, bf = torch.device("cuda:0"), torch.bfloat16
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def timed(fn, reps=7):
+        times = []
+        for _ in range(reps + 3):
+            flush.zero_()                                         # L2 holds nothing of the last run
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            times.append(a.elapsed_time(b) * 1e3)
+        return statistics.median(times[3:])
+
+    def point(us, n_bytes=0, flops=0):
+        p = {"us": round(us, 1)}
+        if n_bytes:
+            p.update(gb_s=round(n_bytes / us / 1e3, 1), hbm_frac=round(n_bytes / (us * 1e-6) / hbm, 3))
+        if flops:
+            p.update(tflops=round(flops / us / 1e6, 1), tensor_frac=round(flops / (us * 1e-6) / tf, 3))
+        return p
+
+    out = {}
+    # ---- the recurrences, all 32-bit: read the projections' rows once, read and write the state once, write the outputs
+    for label, n_new, B in (("prefill_2048", 2048, 1), ("prefill_8192", 8192, 1), ("prefill_4x2048", 2048, 4), ("decode_b8", 1, 8), ("decode_b64", 1, 64)):
+        T = n_new * B
+        cu = torch.arange(0, T + 1, n_new, device=dev).int()
+        ctx = SimpleNamespace(cu_seqlens=cu, slots=torch.arange(B, device=dev).int(), n_seqs=B, max_new=n_new, single_token=n_new == 1)
+        for H, K, P in ((4, 256, 512), (16, 128, 128)):
+            proj = torch.randn(T, H * (2 * K + 2 * P) + 2 * H + (-2 * H) % 8, device=dev)
+            at = H * (2 * K + 2 * P)
+            bias = torch.zeros(H, device=dev)
+            state, m = torch.zeros(B, H, P + 1, K, device=dev), torch.zeros(B, H, P + 1, device=dev)
+            n_bytes = 4 * (T * H * (2 * K + 2 * P + 3) + 2 * B * H * (P + 1) * K)
+            flops = T * H * 4 * K * (P + 1)                       # the recurrence itself: an outer product and a read-out a token
+            out[f"mlstm_{H}x{K}x{P}_{label}"] = point(timed(lambda: ops.mlstm_scan(proj, at, at + H, bias, bias, 15.0, state, m, ctx, H, K, P, K ** -0.5, 1e-6)), n_bytes, flops)
+            raw, div = ops.mlstm_scan(proj, at, at + H, bias, bias, 15.0, state, m, ctx, H, K, P, K ** -0.5, 1e-6)
+            w = torch.ones(H * P, device=dev)
+            norm = lambda d: ops.gated_part_norm(raw, proj, H * (2 * K + P), w, H, 1e-5, gate_first=False, out_dtype=bf, divisor=d)
+            out[f"mlstm_norm_{H}x{P}_{label}"] = point(timed(lambda: norm(div)), T * H * P * 10)
+            out[f"gated_part_norm_{H}x{P}_{label}"] = point(timed(lambda: norm(None)), T * H * P * 10)
+            st = torch.zeros(B, H, P, K, device=dev)
+            like_bytes = 4 * (T * H * (2 * K + 2 * P) + 2 * B * H * P * K)
+            decay = torch.full((H,), 0.99, device=dev)
+            out[f"sagupel_retention_{H}x{K}x{P}_{label}"] = point(timed(lambda: ops.retention_scan(proj, None, None, 0, decay, st, ctx, H, K, P, 1.0, 1.0), reps=3), like_bytes, flops)
+            a_raw = torch.randn(T, H * K, device=dev)
+            out[f"punolix_gla_{H}x{K}x{P}_{label}"] = point(timed(lambda: ops.gla_scan(proj, a_raw, None, st, ctx, H, K, P, 1.0, 16.0), reps=3), like_bytes + 4 * T * H * K, flops)
+            del proj, state, m, st, raw, div, a_raw
+            torch.cuda.empty_cache()
+    # ---- attention
+    H, G = 16, 4
+    for label, n_new, B, prompt in (("prefill_2048", 2048, 1, 0), ("prefill_8192", 8192, 1, 0), ("decode_b8_at_4096", 1, 8, 4095)):
+        n_ctx, rows = prompt + n_new, B * n_new
+        specs = [KVSpec(G, 128, 1024, value_dim=128), KVSpec(1, 576, 0, values=False)]
+        cache = CacheManager([(sp, None, None) for sp in specs], B * n_ctx + 64 * B, B, n_ctx + 64, bf, dev)
+        slots = cache.open(B)
+        if prompt:
+            build_step_context(cache, [StepEntry(s, [0] * prompt, []) for s in slots], 10, dev)
+            for s in slots:
+                cache.advance(s, prompt)
+        u, ul = cache.unit_cache(0), cache.unit_cache(1)
+        for pool in (u.k_pool, u.v_pool, ul.k_pool):
+            pool.normal_()
+        ctx = build_step_context(cache, [StepEntry(s, [0] * n_new, []) for s in slots], 10, dev)[0]
+        table, ltable = ctx.page_tables[u.group_id], ctx.page_tables[ul.group_id]
+        gate = torch.randn(rows, 24, device=dev)
+        q = torch.randn(rows, H, 128, device=dev).to(bf)
+        run = lambda **kw: ops.maps_attention(q, u.k_pool, u.v_pool, table, ctx, 2, 0.125, lam=0.6, norm_out=True, eps=1e-5, out_scale=0.2, **kw)
+        pairs = {0: n_new * (n_new + 1) // 2, 1024: sum(min(i + 1, 1024) for i in range(n_new))}
+        for name, window, kw in (("windowed_gated_maps", 1024, {"window": 1024, "gate": gate}), ("windowed_maps", 1024, {"window": 1024}),
+                                 ("gated_maps", 0, {"gate": gate}), ("punolix_maps", 0, {}), ("punolix_maps_in_chunks", 1024, {"chunk": 1024})):
+            keys = min(window or n_ctx, n_ctx)
+            work = {"flops": H * pairs[window] * 2 * (128 + 2 * 128)} if n_new > 1 else {"n_bytes": B * G * keys * 256 * 2}
+            if n_new > 1 and name == "punolix_maps_in_chunks":
+                work = {"flops": H * (n_new // 1024) * (1024 * 1025 // 2) * 2 * (128 + 2 * 128)}
+            out[f"{name}_{label}"] = point(timed(lambda: run(**kw), reps=5), **work)
+        n_cols = (H + G) * 128 + G * 128
+        proj, qkv = torch.randn(rows, n_cols + H, device=dev), torch.randn(rows, n_cols, device=dev)
+        cs, bias = torch.ones(rows, 32, device=dev), torch.zeros(n_cols, device=dev)
+        prep = lambda x: ops.maps_prep(x, None, None, None, cs, cs, ctx, table, u.k_pool, u.v_pool, H, G, 2, 64, 128, 64, False, 1e-5)
+        out[f"maps_prep_{label}"] = point(timed(lambda: prep(qkv)), rows * n_cols * 6)
+        tail, taps = torch.zeros(B, 3, n_cols, device=dev), torch.randn(n_cols, 4, device=dev)
+        conv = lambda x: ops.short_conv(x, 0, n_cols, taps, None, tail, ctx, activation=False, in_bias=bias)
+        out[f"short_conv_beside_a_gate_{label}"] = point(timed(lambda: conv(proj)), rows * n_cols * 8)
+        out[f"punolix_short_conv_{label}"] = point(timed(lambda: conv(qkv)), rows * n_cols * 8)
+        if n_new > 1:
+            ql, kp, v = (torch.randn(rows, H * d, device=dev).to(bf) for d in (192, 128, 128))
+            lrows = torch.randn(rows, 576, device=dev).to(bf)
+            for name, kw in (("gated_latent", {"gate": gate}), ("movudra_latent", {})):
+                out[f"{name}_{label}"] = point(timed(lambda: ops.latent_prefill(ql.view(rows, H, 192), kp, lrows, v, ctx, None, 0.07, 0, H, 128, 64, 128, **kw), reps=5),
+                                               flops=H * pairs[0] * 2 * 320)
+        else:
+            qa, qr = torch.randn(H, rows, 512, device=dev), torch.randn(rows, H, 64, device=dev)
+            out[f"latent_{label}"] = point(timed(lambda: ops.latent_attention(qa, qr, ul.k_pool, ltable, ctx, None, 0.07)), B * n_ctx * 576 * 2)
+        vals = torch.randn(H, rows, 128, device=dev)
+        out[f"latent_heads_out_gated_{label}"] = point(timed(lambda: ops.latent_heads_out(vals, bf, gate)), rows * H * 128 * 6)
+        out[f"latent_heads_out_{label}"] = point(timed(lambda: ops.latent_heads_out(vals, bf)), rows * H * 128 * 6)
+        del cache, u, ul
+        torch.cuda.empty_cache()
+    # ---- the feed-forward
+    D, E, top, F, Fs = 2048, 64, 6, 1408, 2816
+    w_up, w_down = torch.randn(E, F, D, device=dev).to(bf) * 0.02, torch.randn(E, D, F, device=dev).to(bf) * 0.02
+    s_up, s_down = torch.randn(Fs, D, device=dev).to(bf) * 0.02, torch.randn(D, Fs, device=dev).to(bf) * 0.02
+    for T in (2048, 16, 8, 1):
+        x, z = torch.randn(T, D, device=dev).to(bf), torch.randn(T, E, device=dev)
+        route = lambda: ops.moe_route(z, top, scores="sigmoid")
+        out[f"router_sigmoid_{T}"] = point(timed(route), T * (E * 4 + top * 8))
+        out[f"router_movudra_{T}"] = point(timed(lambda: ops.moe_route(z, top)), T * (E * 4 + top * 8))
+        chosen, weight = route()
+        used = len(torch.unique(chosen))
+        shared = torch.randn(T, D, device=dev)
+        for name, act, kw in (("experts_weight_on_input", "relu2", {"weight_on_input": True}), ("experts_tufadra", "gelu", {})):
+            if T > 16:
+                out[f"{name}_{T}"] = point(timed(lambda: ops.moe_experts_grouped(x, w_up, w_down, chosen, weight, act, shared=shared, **kw)), flops=T * top * 4 * D * F)
+            else:
+                out[f"{name}_{T}"] = point(timed(lambda: ops.moe_experts(x, w_up, w_down, chosen, weight, act, s_up, s_down, **kw)), (used * 2 * D * F + 2 * D * Fs) * 2)
+    return out
+
+
 def reference_arm(args) -> int:
     """kishida/questwend itself, unmodified, through its own public classes (baseline/ref_bench.cpp), on the same sizes.
     Nothing of questwend_b200 is imported on this path."""
@@ -1048,9 +1201,10 @@ def main() -> int:
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--model", default="8b", choices=sorted(MODELS) + ["movudra", "roritar", "roritar-kernels", "punolix", "punolix-kernels", "sagupel", "sagupel-kernels", "tufadra", "tufadra-kernels"],
-                    help="8b: the benchmark; 0.6b, 32b: its other workloads alone; movudra, roritar, punolix, sagupel, tufadra: that design at real layer "
-                         "sizes beside Qwen3 layers of the same width and depth; roritar-kernels, punolix-kernels, sagupel-kernels, tufadra-kernels: its own kernels alone, each "
+    ap.add_argument("--model", default="8b", choices=sorted(MODELS) + ["movudra", "roritar", "roritar-kernels", "punolix", "punolix-kernels", "sagupel", "sagupel-kernels", "tufadra", "tufadra-kernels",
+                                                                               "tebozen", "tebozen-kernels"],
+                    help="8b: the benchmark; 0.6b, 32b: its other workloads alone; movudra, roritar, punolix, sagupel, tufadra, tebozen: that design at real layer "
+                         "sizes beside Qwen3 layers of the same width and depth; roritar-kernels, punolix-kernels, sagupel-kernels, tufadra-kernels, tebozen-kernels: its own kernels alone, each "
                          "beside the like kernel of a model the library had")
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the model has (named in config)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
@@ -1124,6 +1278,19 @@ def main() -> int:
         print(json.dumps({"metric": "Tufadra's kernels alone, each beside the like kernel of an earlier model", "n_gpus": 1,
                           "dtype": "bf16", "data": "synthetic: random tensors of the sizes of tufadra_sizes; L2 flushed between runs",
                           "peaks": peak_source, "points": tufadra_kernels(torch, np, peaks)}))
+        return 0
+    if args.model == "tebozen":
+        designs = (("tebozen", tebozen_sizes()), ("tebozen_memory_16x128x128_top_2", tebozen_sizes(memory=(16, 128, 128), top=2)),
+                   ("tebozen_width_1024", tebozen_sizes(width=1024)), ("tufadra_same_size", tufadra_sizes()), ("movudra_same_size", movudra_sizes()),
+                   ("punolix_same_size", punolix_sizes()), ("qwen3_same_size", qwen3_beside()))
+        print(json.dumps({"metric": "Tebozen at real layer sizes beside Tufadra, Movudra, Punolix and Qwen3 layers of equal width and depth", "n_gpus": 1,
+                          "dtype": "bf16", "data": "synthetic: seeded random weights and uniform random token ids",
+                          "peaks": peak_source, "points": movudra_workload(torch, np, peaks, steps, warmup, designs)}))
+        return 0
+    if args.model == "tebozen-kernels":
+        print(json.dumps({"metric": "Tebozen's kernels alone, each beside the like kernel of an earlier model", "n_gpus": 1,
+                          "dtype": "bf16", "data": "synthetic: random tensors of the sizes of tebozen_sizes; L2 flushed between runs",
+                          "peaks": peak_source, "points": tebozen_kernels(torch, np, peaks)}))
         return 0
     if args.model != "8b":                      # one of the other workloads alone, as a line of its own
         points = small_model_workload(torch, np, peaks) if args.model == "0.6b" else large_model_workload(torch, np, peaks)
