@@ -1,10 +1,9 @@
-// Matrix memory with exponential gates (the mLSTM of xLSTM).  Per head, token by token, with a log input gate i and a log
-// forget gate f:
-//     m_t = max(f + m_(t-1), i)                                   (m starts at 0)
-//     S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T     (K x P)
-//     n_t = e^(f + m_(t-1) - m_t) n_(t-1) + e^(i - m_t) k
-//     o_t = S_t^T q / (max(|n_t . q|, e^(-m_t)) + tiny)
-// i = cap tanh((i_raw + i_bias) / cap), f = log sigmoid(cap tanh((f_raw + f_bias) / cap)).  n is the memory of a value that
+// Matrix memory with exponential gates (the mLSTM of xLSTM).  Per head and token, with logarithms i and f of an input and a
+// forget gate, the memory S (K x P), its normaliser n (K) and a running maximum m (0 before the first token) become
+//     m' = max(m + f, i),   keep = e^(m + f - m'),   write = e^(i - m')
+//     S' = keep S + write k v^T,   n' = keep n + write k
+// and are read out as  S'^T q / (max(|n' . q|, e^-m') + tiny).  Both logarithms come from raw gates z through a cap,
+// i = cap tanh((z_i + b_i) / cap) and f = log sigmoid(cap tanh((z_f + b_f) / cap)).  n is the memory of a value that
 // is always 1, so it is kept as one more column: a head's state is [P + 1][K] floats, column by column, the last one n.
 // The running maximum is kept once per column ([P + 1] floats, all equal), so that a step of one token needs no order
 // between the warps that share a head.  Everything is 32-bit; running maxima and sums of logarithms inside a chunk are
@@ -35,7 +34,7 @@ __device__ __forceinline__ void mlstm_log_gates(MlstmRows rows, MlstmGates g, in
 // ---------------------------------------------------------------------------------
 // Gates of a step that brings several tokens.  grid (H, B), 256 threads.  A token is the map m -> max(m + f, i); maps compose
 // into maps of the same form, so the running maxima are a scan over the tokens (in 64-bit, 256 at a time).  With the rounded
-// maxima, log_decay = f + m_(t-1) - m_t telescopes exactly.  Outputs [T, H].
+// maxima, log_decay = m + f - m' telescopes exactly.  Outputs [T, H].
 // ---------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256)
 mlstm_gates_kernel(MlstmRows rows, MlstmGates gates, const float* __restrict__ m_state, const int* __restrict__ cu_seqlens,
@@ -247,15 +246,19 @@ __device__ __forceinline__ void mlstm_prefix(const float* __restrict__ log_decay
     G[2 * lane + 1] = sum;
 }
 
-// grid (chunks, H * ptiles * ktiles, B), 256 threads; a tile is 64 value columns x 64 key rows, a thread 4 x 4 of it
-template <bool VEC>
+// grid (chunks, H * ptiles * ktiles, B), 256 threads; a tile is PT (64 or 128) value columns x 64 key rows, a thread
+// PT / 16 x 4 of it; dynamic shared memory: 64 * (64 + PT) floats
+template <int PT, bool VEC>
 __global__ void __launch_bounds__(256)
 mlstm_chunk_state_kernel(MlstmRows rows, const float* __restrict__ log_decay, const float* __restrict__ write, const int* __restrict__ cu_seqlens,
                          float* __restrict__ own, float* __restrict__ totals, MlstmSizes z, int n_chunks, int ptiles, int ktiles) {
     pdl_wait();
     pdl_launch_dependents();
     constexpr int L = QWB_MLSTM_CHUNK;
-    __shared__ __align__(16) float ks[L][64], vs[L][64];
+    constexpr int CN = PT / 64;                                     // groups of four value columns a thread
+    extern __shared__ __align__(16) float cs_smem[];
+    float (*ks)[64] = reinterpret_cast<float (*)[64]>(cs_smem);
+    float (*vs)[PT] = reinterpret_cast<float (*)[PT]>(cs_smem + L * 64);
     __shared__ double G[L];
     __shared__ float coef[L];
     const int H = z.H, K = z.K, P = z.P, c = blockIdx.x, b = blockIdx.z, tid = threadIdx.x;
@@ -267,45 +270,51 @@ mlstm_chunk_state_kernel(MlstmRows rows, const float* __restrict__ log_decay, co
     if (tid < L) coef[tid] = tid < n ? expf((float)(G[L - 1] - G[tid])) * write[(size_t)(t0 + tid) * H + h] : 0.f;
     if (tid == 0 && tile == 0) totals[((size_t)b * n_chunks + c) * H + h] = expf((float)G[L - 1]);
     __syncthreads();
-    const int k0 = kt * 64, p0 = pt * 64;
+    const int k0 = kt * 64, p0 = pt * PT;
     for (int idx = tid; idx < L * 16; idx += 256) {
         const int j = idx >> 4, e = (idx & 15) * 4;
-        float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), v4 = k4;
-        if (j < n) {
-            const float* row = rows.x + (size_t)(t0 + j) * rows.ld;
-            k4 = mlstm_four<VEC>(row + (H + h) * K, k0 + e, K);
-            v4 = mlstm_four<VEC>(row + 2 * H * K + h * P, p0 + e, P);
-        }
+        float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < n) k4 = mlstm_four<VEC>(rows.x + (size_t)(t0 + j) * rows.ld + (H + h) * K, k0 + e, K);
         const float f = coef[j];
         *reinterpret_cast<float4*>(&ks[j][e]) = make_float4(k4.x * f, k4.y * f, k4.z * f, k4.w * f);
+    }
+    for (int idx = tid; idx < L * (PT / 4); idx += 256) {
+        const int j = idx / (PT / 4), e = (idx - j * (PT / 4)) * 4;
+        float4 v4 = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < n) v4 = mlstm_four<VEC>(rows.x + (size_t)(t0 + j) * rows.ld + 2 * H * K + h * P, p0 + e, P);
         *reinterpret_cast<float4*>(&vs[j][e]) = v4;
     }
     __syncthreads();
     const int kq = (tid & 15) * 4, pq = (tid >> 4) * 4;
-    float acc[4][4];
+    float acc[4 * CN][4];
 #pragma unroll
-    for (int p = 0; p < 4; ++p)
+    for (int p = 0; p < 4 * CN; ++p)
 #pragma unroll
         for (int k = 0; k < 4; ++k) acc[p][k] = 0.f;
 #pragma unroll 8
     for (int j = 0; j < L; ++j) {
         const float4 kk = *reinterpret_cast<const float4*>(&ks[j][kq]);
-        const float4 vv = *reinterpret_cast<const float4*>(&vs[j][pq]);
-        const float ka[4] = {kk.x, kk.y, kk.z, kk.w}, va[4] = {vv.x, vv.y, vv.z, vv.w};
+        const float ka[4] = {kk.x, kk.y, kk.z, kk.w};
 #pragma unroll
-        for (int p = 0; p < 4; ++p)
+        for (int g = 0; g < CN; ++g) {
+            const float4 vv = *reinterpret_cast<const float4*>(&vs[j][64 * g + pq]);
+            const float va[4] = {vv.x, vv.y, vv.z, vv.w};
 #pragma unroll
-            for (int k = 0; k < 4; ++k) acc[p][k] += va[p] * ka[k];
+            for (int p = 0; p < 4; ++p)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) acc[4 * g + p][k] += va[p] * ka[k];
+        }
     }
     float* U = own + (((size_t)b * n_chunks + c) * H + h) * (size_t)(P + 1) * K;
 #pragma unroll
-    for (int p = 0; p < 4; ++p) {
-        if (p0 + pq + p >= P) continue;
-        float* u = U + (size_t)(p0 + pq + p) * K + k0 + kq;
-        if (VEC) { if (k0 + kq < K) *reinterpret_cast<float4*>(u) = make_float4(acc[p][0], acc[p][1], acc[p][2], acc[p][3]); }
+    for (int a = 0; a < 4 * CN; ++a) {
+        const int p = p0 + 64 * (a >> 2) + pq + (a & 3);
+        if (p >= P) continue;
+        float* u = U + (size_t)p * K + k0 + kq;
+        if (VEC) { if (k0 + kq < K) *reinterpret_cast<float4*>(u) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]); }
         else {
 #pragma unroll
-            for (int k = 0; k < 4; ++k) if (k0 + kq + k < K) u[k] = acc[p][k];
+            for (int k = 0; k < 4; ++k) if (k0 + kq + k < K) u[k] = acc[a][k];
         }
     }
     if (pt == 0 && tid < 64 && k0 + tid < K) {                      // the column whose value is always 1
@@ -316,7 +325,9 @@ mlstm_chunk_state_kernel(MlstmRows rows, const float* __restrict__ log_decay, co
     }
 }
 
-// grid (ceil((P + 1) * K / 256), H, B): every element of the state runs through its sequence's chunks in order
+// grid (ceil((P + 1) * K / W / 256), H, B): every element of the state runs through its sequence's chunks in order, W (4 or 1)
+// neighbours a thread
+template <int W>
 __global__ void __launch_bounds__(256)
 mlstm_chunk_carry_kernel(const int* __restrict__ cu_seqlens, const int* __restrict__ slots, float* __restrict__ state, float* __restrict__ m_state,
                          float* own, const float* __restrict__ totals, const float* __restrict__ m_run, MlstmSizes z, int n_chunks, int write_state) {
@@ -324,27 +335,40 @@ mlstm_chunk_carry_kernel(const int* __restrict__ cu_seqlens, const int* __restri
     pdl_launch_dependents();
     constexpr int AHEAD = 8;
     const int H = z.H, K = z.K, P = z.P, h = blockIdx.y, b = blockIdx.z;
-    const int e = blockIdx.x * blockDim.x + threadIdx.x, n_el = (P + 1) * K;
+    const int e = (blockIdx.x * blockDim.x + threadIdx.x) * W, n_el = (P + 1) * K;
     const int t1 = cu_seqlens[b + 1], n_tok = t1 - cu_seqlens[b];
     if (e >= n_el || n_tok <= 0) return;
     const size_t head = (size_t)slots[b] * H + h;
-    float s = state[head * n_el + e];
+    auto load = [](const float* p, float* v) {
+        if (W == 4) { const float4 x = *reinterpret_cast<const float4*>(p); v[0] = x.x; v[W > 1 ? 1 : 0] = x.y; v[W > 2 ? 2 : 0] = x.z; v[W - 1] = x.w; }
+        else v[0] = *p;
+    };
+    auto store = [](float* p, const float* v) {
+        if (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[W > 1 ? 1 : 0], v[W > 2 ? 2 : 0], v[W - 1]);
+        else *p = v[0];
+    };
+    float s[W];
+    load(state + head * n_el + e, s);
     const int chunks = (n_tok + QWB_MLSTM_CHUNK - 1) / QWB_MLSTM_CHUNK;
     const size_t step = (size_t)H * n_el;
     float* at = own + ((size_t)b * n_chunks * H + h) * n_el + e;
     const float* total = totals + (size_t)b * n_chunks * H + h;
     for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        float u[AHEAD], d[AHEAD];
+        float u[AHEAD][W], d[AHEAD];
 #pragma unroll
         for (int a = 0; a < AHEAD; ++a)
-            if (c0 + a < chunks) { u[a] = at[(c0 + a) * step]; d[a] = total[(size_t)(c0 + a) * H]; }
+            if (c0 + a < chunks) { load(at + (c0 + a) * step, u[a]); d[a] = total[(size_t)(c0 + a) * H]; }
 #pragma unroll
         for (int a = 0; a < AHEAD; ++a)
-            if (c0 + a < chunks) { at[(c0 + a) * step] = s; s = d[a] * s + u[a]; }
+            if (c0 + a < chunks) {
+                store(at + (c0 + a) * step, s);
+#pragma unroll
+                for (int i = 0; i < W; ++i) s[i] = d[a] * s[i] + u[a][i];
+            }
     }
     if (write_state) {
-        state[head * n_el + e] = s;
-        if (e % K == 0) m_state[head * (P + 1) + e / K] = m_run[(size_t)(t1 - 1) * H + h];
+        store(state + head * n_el + e, s);
+        if (e % K == 0) m_state[head * (P + 1) + e / K] = m_run[(size_t)(t1 - 1) * H + h];     // with W = 4, K is a multiple of 4
     }
 }
 
@@ -567,19 +591,27 @@ extern "C" int qwb_mlstm_chunked(const float* x, int ld, int i_col, int f_col, c
     const MlstmGates gates{i_bias, f_bias, cap};
     if (int rc = check_mlstm("mlstm_chunked", z, rows, B)) return rc;
     const int n_chunks = (max_new + QWB_MLSTM_CHUNK - 1) / QWB_MLSTM_CHUNK;
-    const int pt = P > 64 ? 128 : 64, ptiles = (P + pt - 1) / pt, ptiles64 = (P + 63) / 64, ktiles = (K + 63) / 64;
-    if (!(cap > 0.f) || !gate_rows || !scratch || (long long)H * ptiles64 * ktiles > 65535 || (long long)(P + 1) * K > 0x7fffffffLL)
+    const int pt = P > 64 ? 128 : 64, ptiles = (P + pt - 1) / pt, ktiles = (K + 63) / 64;
+    if (!(cap > 0.f) || !gate_rows || !scratch || (long long)H * ptiles * ktiles > 65535 || (long long)(P + 1) * K > 0x7fffffffLL)
         return qwb_fail(QWB_ERR_ARG, "mlstm_chunked: cap %g, %d heads of %d x %d", (double)cap, H, K, P);
     float *log_decay = gate_rows, *write = gate_rows + (size_t)T * H, *m_run = gate_rows + 2 * (size_t)T * H;
     float* totals = scratch + (size_t)B * n_chunks * H * (P + 1) * K;
-    const bool vec = K % 4 == 0 && P % 4 == 0 && ld % 4 == 0 && mlstm_aligned(x) && mlstm_aligned(scratch) && mlstm_aligned(raw);
+    const bool vec = K % 4 == 0 && P % 4 == 0 && ld % 4 == 0 && mlstm_aligned(x) && mlstm_aligned(scratch) && mlstm_aligned(raw) && mlstm_aligned(state);
     qwb_launch(mlstm_gates_kernel, dim3(H, B), 256, 0, stream, rows, gates, (const float*)m_state, cu_seqlens, slots, log_decay, write, m_run, H, P);
     if (int rc = qwb_check_launch("mlstm_gates")) return rc;
-    const dim3 g1(n_chunks, H * ptiles64 * ktiles, B);
-    auto state_kernel = vec ? mlstm_chunk_state_kernel<true> : mlstm_chunk_state_kernel<false>;
-    qwb_launch(state_kernel, g1, 256, 0, stream, rows, (const float*)log_decay, (const float*)write, cu_seqlens, scratch, totals, z, n_chunks, ptiles64, ktiles);
+    const size_t smem1 = (size_t)QWB_MLSTM_CHUNK * (64 + pt) * sizeof(float);
+    auto state_kernel = pt == 128 ? (vec ? mlstm_chunk_state_kernel<128, true> : mlstm_chunk_state_kernel<128, false>)
+                                  : (vec ? mlstm_chunk_state_kernel<64, true> : mlstm_chunk_state_kernel<64, false>);
+    if (smem1 + 1024 > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        if (e != cudaSuccess) return qwb_fail(QWB_ERR_CUDA, "mlstm_chunked: %s", cudaGetErrorString(e));
+    }
+    qwb_launch(state_kernel, dim3(n_chunks, H * ptiles * ktiles, B), 256, smem1, stream, rows, (const float*)log_decay, (const float*)write, cu_seqlens, scratch,
+               totals, z, n_chunks, ptiles, ktiles);
     if (int rc = qwb_check_launch("mlstm_chunk_state")) return rc;
-    qwb_launch(mlstm_chunk_carry_kernel, dim3(((P + 1) * K + 255) / 256, H, B), 256, 0, stream, cu_seqlens, slots, state, m_state, scratch,
+    auto carry_kernel = vec ? mlstm_chunk_carry_kernel<4> : mlstm_chunk_carry_kernel<1>;
+    const int per_block = vec ? 1024 : 256;
+    qwb_launch(carry_kernel, dim3(((P + 1) * K + per_block - 1) / per_block, H, B), 256, 0, stream, cu_seqlens, slots, state, m_state, scratch,
                (const float*)totals, (const float*)m_run, z, n_chunks, write_state);
     if (int rc = qwb_check_launch("mlstm_chunk_carry")) return rc;
     const size_t lq = QWB_MLSTM_CHUNK + 4, lp = pt + 4;

@@ -319,9 +319,25 @@ def bench_moe(T, D, F, E, top, shared, activation, iters, dtype=torch.bfloat16) 
             "tflops": 2 * T * top * per / us / 1e6}
 
 
+def bench_mlstm(B, tokens, H, K, P, iters) -> dict:
+    """The mLSTM's matrix memory (``H`` heads of ``K`` x ``P``, 32-bit): ``B`` sequences that bring ``tokens`` new tokens each
+    (1: the kernel for single tokens; 64 and more: the chunked form; else the scan)."""
+    from types import SimpleNamespace
+    T, at = B * tokens, H * (2 * K + 2 * P)
+    proj = torch.randn(T, at + -(-2 * H // 8) * 8, device=DEV)
+    bias = torch.zeros(H, device=DEV)
+    state, m = torch.zeros(B, H, P + 1, K, device=DEV), torch.zeros(B, H, P + 1, device=DEV)
+    step = SimpleNamespace(cu_seqlens=torch.arange(0, T + 1, tokens, device=DEV).int(), slots=torch.arange(B, device=DEV).int(), n_seqs=B,
+                           max_new=tokens, single_token=tokens == 1)
+    us = _time(lambda i: ops.mlstm_scan(proj, at, at + H, bias, bias, 15.0, state, m, step, H, K, P, K ** -0.5, 1e-6), 1, iters, burst=3)
+    n_bytes = 4 * (T * H * (2 * K + 2 * P + 3) + 2 * B * H * (P + 1) * K)
+    return {"what": "mlstm", "batch": B, "tokens": tokens, "heads": H, "key": K, "value": P, "us": us, "bytes": n_bytes,
+            "gb_s": n_bytes / us / 1e3, "tflops": T * H * 4 * K * (P + 1) / us / 1e6}
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "attn_decode", "attn_prefill", "rmsnorm", "rope", "decode_shapes", "sample", "pool_attn", "maps_attn", "shaped_attn", "moe"])
+    ap.add_argument("what", choices=["gemm", "attn_decode", "attn_prefill", "rmsnorm", "rope", "decode_shapes", "sample", "pool_attn", "maps_attn", "shaped_attn", "moe", "mlstm"])
     ap.add_argument("--m", type=int, default=8)
     ap.add_argument("--n", type=int, default=24576)
     ap.add_argument("--k", type=int, default=4096)
@@ -344,7 +360,7 @@ def main() -> int:
     ap.add_argument("--runs-target", type=int, default=0, help="tensor-core decode attention: about this many runs a sequence")
     ap.add_argument("--run-pages-max", type=int, default=0, help="tensor-core decode attention: at most this many pages a run")
     ap.add_argument("--fused", action="store_true", help="decode attention with the q/k norm, rotation and cache write inside")
-    ap.add_argument("--value-dim", type=int, default=0, help="pool_attn: size of a value (default: the head size)")
+    ap.add_argument("--value-dim", type=int, default=0, help="pool_attn, mlstm: size of a value (default: the head size)")
     ap.add_argument("--window", type=int, default=1024, help="pool_attn: the window")
     ap.add_argument("--maps", type=int, default=2, help="maps_attn: score maps per head")
     ap.add_argument("--softcap", type=float, default=0.0, help="maps_attn: the cap on the scores (0: none)")
@@ -381,6 +397,8 @@ def main() -> int:
                                                 args.iters, dtype, args.attn_impl)))
     elif args.what == "moe":
         print(json.dumps(bench_moe(args.m, args.k, args.n, args.experts, args.top_k, args.shared, args.activation, args.iters, dtype)))
+    elif args.what == "mlstm":
+        print(json.dumps(bench_mlstm(args.batch, args.tokens, args.heads, args.head_dim, args.value_dim or args.head_dim, args.iters)))
     elif args.what == "sample":
         print(json.dumps(bench_sample(args.batch, args.vocab, args.temp, args.top_k, args.top_p, args.iters)))
     elif args.what == "attn_prefill":

@@ -224,8 +224,8 @@ class ScoreMapsAttention(Mixer):
     > 0, a causal mask, with ``chunk`` > 0 only the keys of the query's own block of ``chunk`` positions, counted
     from the sequence's start, and with ``window`` > 0 only the last ``window`` keys, the query's own among them).  With two maps the head's output is differential: a1 - lambda * a2 with
     lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + ``diff`` (four learned vectors of the layer), divided by its root mean
-    square over the value size (eps inside the root) and multiplied by 1 - ``diff``.  ``head_gate``: head h's output times
-    sigmoid(W_g h)_h, one number per head, in front of the output projection.  In front of the scores, in this
+    square over the value size (eps inside the root) and multiplied by 1 - ``diff``.  ``head_gate``: a sigmoid
+    gate per token and head (W_g h) on the heads' outputs, ahead of W_o.  In front of the scores, in this
     order and each optional: biases on q, k and v, a short causal convolution over time on every channel of q, k and v
     (``conv`` taps, no activation; its last inputs are per-sequence state), an RMS norm of every map of q and k with a
     weight shared by heads and maps (``qk_norm_over`` "head") or of the whole projections of q and of k with weights of

@@ -29,9 +29,9 @@ class LatentAttention(Mixer):
     c_q = RMSnorm(W_dq h); q = W_uq c_q (or q = W_q h), head by head [dim | rot_dim].  W_dkv h = [kv_rank latent, RMS-normed ->
     c | rot_dim rotated key part].  The position encoding turns neighbouring pairs of the rotated parts of q and k.
     score = (q_plain . W_uk c + q_rot . k_rot) * scale; softmax over the visible keys (and the sink); value W_uv c.
-    ``head_gate``: head h's output times sigmoid(W_g h)_h, one number per head, in front of the output projection.
-    ``shared_rows``: no W_dkv; c and the rotated key part are another layer's, as its cache holds them (the same kv_rank,
-    rot_dim and rotation); W_uk, W_uv, the queries and the rest are the layer's own."""
+    ``head_gate``: a sigmoid gate per token and head (W_g h) on the heads' outputs, ahead of W_o.  ``shared_rows``: the layer
+    has no W_dkv and writes no rows; its run reads the rows of another layer's run, whose latent and rotation have the same
+    sizes, through keys, values and queries of its own."""
 
     NAMES = {"q_down": "dq", "q_norm": "dq.norm", "q_up": "uq", "kv_down": "dkv", "kv_norm": "dkv.norm", "k_up": "uk",
              "v_up": "uv", "sink": "sink", "out": "o", "q": "q", "gate": "g"}

@@ -436,11 +436,11 @@ class RetentionMixer(Mixer):
 
 
 class MLSTMMixer(Mixer):
-    """The matrix memory of the mLSTM.  q = W_q h * ``q_scale`` and k = W_k h (heads x key_dim), v = W_v h (heads x vdim); per
-    head a log input gate i = cap tanh((W_i h + b_i) / cap) and a log forget gate f = log sigmoid(cap tanh((W_f h + b_f) / cap)),
-    cap = ``gate_cap``.  With a running maximum m from 0, m' = max(f + m, i):  S <- e^(f + m - m') S + e^(i - m') k v^T, n the
-    same with k alone, o = S^T q / (max(|n . q|, e^-m') + ``tiny``).  Each head's o is divided by its root mean square over
-    vdim, times a weight per value, times sigmoid(W_g h); then the output projection.
+    """The matrix memory of the mLSTM.  q = W_q h * ``q_scale`` and k = W_k h (heads x key_dim), v = W_v h (heads x vdim).  Per
+    head two gates as logarithms, i = c tanh((W_i h + b_i) / c) and f = log sigmoid(c tanh((W_f h + b_f) / c)) with c =
+    ``gate_cap``.  From S = 0, n = 0, m = 0, token by token: m' = max(m + f, i), S <- e^(m + f - m') S + e^(i - m') k v^T, n the
+    memory of a value of 1, and o = S^T q / (max(|n . q|, e^-m') + ``tiny``).  o is RMS-normed per head, times a weight of all
+    heads' size, times sigmoid(W_g h), and projected by W_o.
 
     params: hidden_size, heads, key_dim, vdim, gate_cap, norm_eps, q_scale (default key_dim^-1/2), tiny (default 1e-6), names
     (optional overrides).  State per sequence: S and n, stored [heads, vdim + 1, key_dim] (n is the column of a value that is

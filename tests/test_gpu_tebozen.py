@@ -172,7 +172,7 @@ def maps_oracle(q, k, v, before, maps, scale, window, lam, norm_out, eps, out_sc
 
 
 @pytest.mark.parametrize("maps, H, G, dim, vdim, window, gated", [
-    (2, 4, 2, 16, 32, 20, True), (2, 2, 1, 64, 128, 64, True), (2, 4, 1, 48, 96, 65, False), (2, 2, 2, 32, 136, 130, True), (2, 3, 1, 16, 40, 1, True),
+    (2, 4, 2, 16, 32, 20, True), (2, 2, 1, 64, 128, 64, True), (2, 6, 2, 48, 88, 65, False), (2, 2, 2, 32, 136, 130, True), (2, 3, 1, 16, 40, 1, True),
     (1, 4, 2, 32, 24, 63, True), (1, 4, 2, 64, 64, 70, False), (2, 8, 2, 80, 64, 2, True), (1, 2, 2, 160, 256, 100, True), (2, 2, 1, 128, 128, 0, True)])
 def test_windows_and_gates_of_score_maps(maps, H, G, dim, vdim, window, gated):
     """Unequal prompts that go on from cached tokens, and single tokens, over shuffled pages whose other rows hold large
